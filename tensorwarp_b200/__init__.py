@@ -1,11 +1,12 @@
-"""tensorwarp_b200 — the TW-Marlin W4A16 Q4 GEMM family for NVIDIA B200.
+"""tensorwarp_b200 — LLM inference kernels and engines for NVIDIA B200.
 
-Only what this one hot path needs: ``csrc/`` holds the sm_100a kernels and the
-C ABI (``include/twmarlin.h``), ``quantize`` mirrors the reference's host
-interface over that ABI.  Importing the package does not load the library;
-the first call does, and fails loudly if it is not built.
+``csrc/`` holds the sm_100a kernels of two libraries: the TW-Marlin W4A16 Q4 GEMM family and its decode
+step (``include/twmarlin.h``, ``include/twm_decode.h``; host mirror in ``quantize`` and ``generate``),
+and decoder models with dense 16-bit or 32-bit weights (``include/twm_dense.h``; ``dense``, ``engine``).
+``registry`` loads a model by its configuration, ``scheduler`` serves requests on it.  Importing the
+package does not load a library; the first call does, and fails loudly if it cannot.
 """
 from . import _lib  # noqa: F401
 from .build import build  # noqa: F401
 
-__all__ = ["build", "quantize"]
+__all__ = ["build", "quantize", "registry"]

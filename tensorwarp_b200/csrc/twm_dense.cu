@@ -1,0 +1,443 @@
+// twm_dense.cu — host side and C ABI of the dense-weight decoder models (include/twm_dense.h).  A library of
+// its own (libtwmdense.so): a model with 16-bit weights needs none of the 4-bit kernels.
+#include <algorithm>
+#include <cstdio>
+#include <mutex>
+
+#include "twm_dense_common.cuh"
+#include "twm_dense_decode.cuh"
+#include "twm_dense_rows.cuh"
+#include "twm_dense_simt.cuh"
+
+namespace {
+
+using namespace twm;
+using namespace twm::dense;
+
+thread_local char t_last_error[256] = "";
+thread_local int t_launches = 0;
+
+twm_status fail(const char* where, cudaError_t e)
+{
+    snprintf(t_last_error, sizeof(t_last_error), "%s: %s", where, cudaGetErrorString(e));
+    return TWM_ELAUNCH;
+}
+twm_status invalid(const char* what)
+{
+    snprintf(t_last_error, sizeof(t_last_error), "%s", what);
+    return TWM_EINVAL;
+}
+#define TRY(expr) do { const twm_status st_ = (expr); if (st_ != TWM_OK) return st_; } while (0)
+
+constexpr int kArgmaxParts = 148;
+constexpr size_t kSmemLimit = 227 * 1024;
+
+struct DeviceState { bool ready = false; twm_status status = TWM_OK; int sms = 148; };
+DeviceState g_dev[64];
+std::mutex g_mutex;
+
+twm_status device(int* sms)
+{
+    int dev = 0;
+    cudaError_t e = cudaGetDevice(&dev);
+    if (e != cudaSuccess) return fail("cudaGetDevice", e);
+    if (dev < 0 || dev >= 64) return invalid("device index");
+    std::lock_guard<std::mutex> lock(g_mutex);
+    DeviceState& st = g_dev[dev];
+    if (!st.ready) {
+        int major = 0;
+        cudaDeviceGetAttribute(&major, cudaDevAttrComputeCapabilityMajor, dev);
+        cudaDeviceGetAttribute(&st.sms, cudaDevAttrMultiProcessorCount, dev);
+        if (major != 10) {
+            snprintf(t_last_error, sizeof(t_last_error), "device %d is sm_%d*, libtwmdense holds sm_100a code only", dev, major);
+            st.status = TWM_EARCH;
+        }
+        st.ready = true;
+    }
+    if (sms) *sms = st.sms;
+    return st.status;
+}
+
+// One launch: raises the kernel's dynamic shared memory limit when needed, asks for programmatic dependent launch
+// when the caller allows it, and a cluster of `cluster` CTAs along x when > 0.
+template <typename... KArgs, typename... Args>
+twm_status launch(const char* what, void (*kernel)(KArgs...), dim3 grid, int threads, size_t smem, int flags, void* stream,
+                  int cluster, Args&&... args)
+{
+    if (smem > kSmemLimit) return invalid("a row does not fit shared memory");
+    if (smem > 48 * 1024) {
+        const cudaError_t r = cudaFuncSetAttribute((const void*)kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (r != cudaSuccess) return fail(what, r);
+    }
+    if (cluster > 8) {
+        const cudaError_t r = cudaFuncSetAttribute((const void*)kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        if (r != cudaSuccess) return fail(what, r);
+    }
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = dim3(threads);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = (cudaStream_t)stream;
+    cudaLaunchAttribute attr[2];
+    int n = 0;
+    if (flags & TWM_FLAG_PDL) {
+        attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+        attr[n++].val.programmaticStreamSerializationAllowed = 1;
+    }
+    if (cluster > 0) {
+        attr[n].id = cudaLaunchAttributeClusterDimension;
+        attr[n].val.clusterDim.x = cluster;
+        attr[n].val.clusterDim.y = 1;
+        attr[n++].val.clusterDim.z = 1;
+    }
+    cfg.attrs = attr;
+    cfg.numAttrs = n;
+    const cudaError_t e = cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...);
+    if (e != cudaSuccess) return fail(what, e);
+    ++t_launches;
+    return TWM_OK;
+}
+
+struct Sizes { int q, k, v, g, in, out; };              // columns of the fused projection, and of the mixer's output
+Sizes sizes_of(const twm_dense_layer& l)
+{
+    Sizes s;
+    s.q = l.heads * l.dim_pad;
+    s.k = l.kv_heads * l.dim_pad;
+    s.v = l.kv_heads * l.vdim_pad;
+    s.g = l.heads * l.vdim_pad;
+    s.in = s.q + s.k + s.v + s.g;
+    s.out = s.g;
+    return s;
+}
+
+twm_status check_model(const twm_dense_model* m, const twm_dense_buffers* b)
+{
+    if (!m || !b || !m->layers) return invalid("null model or buffers");
+    if (m->dtype != TWM_DENSE_F32 && m->dtype != TWM_DENSE_BF16) return invalid("dtype");
+    if (m->width < 1 || m->width_pad < m->width || m->width_pad % 16 || m->vocab < 1 || m->n_layers < 0 || m->capacity < 1)
+        return invalid("model sizes");
+    if (!m->embed || !m->head || !m->final_norm) return invalid("embedding, head or final norm missing");
+    if (!b->meta || !b->tokens || !b->want || !b->x0 || !b->x1 || !b->y || !b->a || !b->proj || !b->att || !b->act || !b->vec ||
+        !b->logits || b->max_rows < 1 || b->max_want < 1)
+        return invalid("buffers");
+    for (int i = 0; i < m->n_layers; ++i) {
+        const twm_dense_layer& l = m->layers[i];
+        if (l.heads < 1 || l.kv_heads < 1 || l.heads % l.kv_heads) return invalid("heads must be a multiple of kv_heads");
+        if (l.dim < 1 || l.vdim < 1 || l.dim_pad < l.dim || l.vdim_pad < l.vdim || l.dim_pad % 16 || l.vdim_pad % 16 || l.ff_pad % 16)
+            return invalid("head or feed-forward sizes");
+        if (l.vdim_pad > 1024) return invalid("value heads of more than 1024 columns");
+        if (l.window < 1 || l.keep_first < 0) return invalid("window");
+        if (l.bias_table && m->bias_len < m->capacity) return invalid("bias table shorter than the cache");
+        if (!l.w_in || !l.w_out || !l.k_cache || !l.v_cache || (l.shift && !l.shift_state)) return invalid("layer pointers");
+        if (l.ff_pad > 0 && (!l.w_gate_up || !l.w_down)) return invalid("feed-forward pointers");
+    }
+    return TWM_OK;
+}
+
+// ------------------------------------------------------------- operations --
+template <typename T>
+twm_status gemm(const T* a, int lda, const T* w, int ldw, void* c, int ldc, int M, int N, int K, int epi, int kernel, int flags,
+                void* stream)
+{
+    const dim3 grid((N + ST - 1) / ST, (M + ST - 1) / ST);
+    switch (epi) {
+        case TWM_EPI_STORE:
+            return launch("gemm_simt", gemm_simt_kernel<T, TWM_EPI_STORE>, grid, 256, 0, flags, stream, 0, a, lda, w, ldw, c, ldc, M, N, K);
+        case TWM_EPI_STORE_F32:
+            return launch("gemm_simt", gemm_simt_kernel<T, TWM_EPI_STORE_F32>, grid, 256, 0, flags, stream, 0, a, lda, w, ldw, c, ldc, M, N, K);
+        case TWM_EPI_GELU_GLU:
+            return launch("gemm_simt", gemm_simt_kernel<T, TWM_EPI_GELU_GLU>, grid, 256, 0, flags, stream, 0, a, lda, w, ldw, c, ldc, M, N, K);
+    }
+    return invalid("epilogue");
+}
+
+template <typename T>
+AttnArgs<T> attn_args(const twm_dense_model* m, const twm_dense_layer& l, const twm_dense_buffers* b, int rows)
+{
+    const Sizes s = sizes_of(l);
+    AttnArgs<T> g;
+    g.proj = (const T*)b->proj;
+    g.out = (T*)b->att;
+    g.k_cache = (const T*)l.k_cache;
+    g.v_cache = (const T*)l.v_cache;
+    g.bias_table = l.bias_table;
+    g.meta = b->meta;
+    g.ld = s.in;
+    g.gate_off = s.q + s.k + s.v;
+    g.heads = l.heads; g.kv_heads = l.kv_heads; g.dim_pad = l.dim_pad; g.vdim_pad = l.vdim_pad;
+    g.window = l.window; g.keep_first = l.keep_first; g.capacity = m->capacity; g.bias_len = m->bias_len; g.rows = rows;
+    g.scale = l.scale;
+    return g;
+}
+
+template <typename T>
+twm_status attention(const twm_dense_model* m, const twm_dense_layer& l, const twm_dense_buffers* b, int rows, int first_pos,
+                     int kernel, int flags, void* stream)
+{
+    const AttnArgs<T> g = attn_args<T>(m, l, b, rows);
+    const int vblock = AS_VPT * AS_THREADS;
+    return launch("attn_simt", attn_simt_kernel<T>, dim3(rows, l.heads, (l.vdim_pad + vblock - 1) / vblock), AS_THREADS,
+                  sizeof(float) * (size_t)(l.dim_pad + AS_THREADS), flags, stream, 0, g);
+}
+
+template <typename T>
+twm_status prefill(const twm_dense_model* m, const twm_dense_buffers* b, int rows, int first_pos, int n_want, float* layer_trace,
+                   int flags, void* stream)
+{
+    const int wp = m->width_pad;
+    const int rpc = rows >= 2048 ? 8 : rows >= 512 ? 4 : 2;
+    float *x = b->x0, *x_next = b->x1;
+    const float* y = nullptr;                            // the sublayer output that has yet to join the residual stream
+    const float* y_norm = nullptr;
+    bool embedded = false;
+    auto source = [&]() {
+        ResidualSource<T> s;
+        s.tokens = embedded ? nullptr : b->tokens;
+        s.embed = (const T*)m->embed;
+        s.pos_embed = (const T*)m->pos_embed;
+        s.x_in = x; s.y = y; s.y_norm = y_norm; s.eps = m->eps; s.width = m->width; s.wp = wp;
+        return s;
+    };
+    // the residual stream brought up to date, with the next sublayer's input beside it
+    auto join = [&](const float* shift, const float* state, bool want_a) {
+        const twm_status st = launch("residual_rows", residual_rows_kernel<T>, dim3((rows + rpc - 1) / rpc), ROW_THREADS,
+                                     sizeof(float) * (size_t)wp, flags, stream, 0, source(), x_next, want_a ? (T*)b->a : (T*)nullptr,
+                                     shift, state, b->meta, rows, rpc);
+        std::swap(x, x_next);
+        embedded = true;
+        y = nullptr;
+        return st;
+    };
+    auto trace = [&](int layer) -> twm_status {
+        if (!layer_trace) return TWM_OK;
+        const cudaError_t e = cudaMemcpyAsync(layer_trace + (size_t)layer * rows * wp, x, sizeof(float) * (size_t)rows * wp,
+                                              cudaMemcpyDeviceToDevice, (cudaStream_t)stream);
+        return e == cudaSuccess ? TWM_OK : fail("layer trace", e);
+    };
+    for (int i = 0; i < m->n_layers; ++i) {
+        const twm_dense_layer& l = m->layers[i];
+        const Sizes s = sizes_of(l);
+        TRY(join(l.shift, l.shift_state, true));
+        if (i > 0) TRY(trace(i - 1));
+        TRY(gemm<T>((const T*)b->a, wp, (const T*)l.w_in, wp, b->proj, s.in, rows, s.in, wp, TWM_EPI_STORE, 0, flags, stream));
+        TRY(launch("qk_norm_append", qk_norm_append_kernel<T>, dim3(rows), ROW_THREADS, 0, flags, stream, 0, (T*)b->proj, s.in,
+                   l.q_norm, l.k_norm, (T*)l.k_cache, (T*)l.v_cache, s.q, s.k, s.v, l.heads * l.dim, l.kv_heads * l.dim, m->eps,
+                   m->capacity, (const float*)x, wp, l.shift ? l.shift_state : (float*)nullptr, b->meta));
+        TRY(attention<T>(m, l, b, rows, first_pos, 0, flags, stream));
+        TRY(gemm<T>((const T*)b->att, s.out, (const T*)l.w_out, s.out, b->y, wp, rows, m->width, s.out, TWM_EPI_STORE_F32, 0, flags,
+                    stream));
+        y = b->y; y_norm = l.norm1;
+        if (l.ff_pad > 0) {
+            TRY(join(nullptr, nullptr, true));
+            TRY(gemm<T>((const T*)b->a, wp, (const T*)l.w_gate_up, wp, b->act, l.ff_pad, rows, l.ff_pad, wp, TWM_EPI_GELU_GLU, 0,
+                        flags, stream));
+            TRY(gemm<T>((const T*)b->act, l.ff_pad, (const T*)l.w_down, l.ff_pad, b->y, wp, rows, m->width, l.ff_pad,
+                        TWM_EPI_STORE_F32, 0, flags, stream));
+            y = b->y; y_norm = l.norm2;
+        }
+    }
+    if (layer_trace && m->n_layers > 0) {
+        TRY(join(nullptr, nullptr, false));
+        TRY(trace(m->n_layers - 1));
+    }
+    if (n_want > 0) {
+        TRY(launch("final_rows", final_rows_kernel<T>, dim3(n_want), ROW_THREADS, sizeof(float) * (size_t)wp, flags, stream, 0,
+                   source(), (T*)b->a, m->final_norm, (const int*)b->want, (const int*)b->meta));
+        TRY(gemm<T>((const T*)b->a, wp, (const T*)m->head, wp, b->logits, m->vocab, n_want, m->vocab, wp, TWM_EPI_STORE_F32, 0,
+                    flags, stream));
+    }
+    return TWM_OK;
+}
+
+template <typename T, int PRO, bool GATED>
+twm_status gemv(GemvArgs<T> g, int sms, int flags, void* stream)
+{
+    const int out_rows = GATED ? GV_ROWS / 2 : GV_ROWS;
+    g.rows_per_cta = std::max((g.N + sms - 1) / sms, std::min(out_rows, g.N));
+    const int grid = (g.N + g.rows_per_cta - 1) / g.rows_per_cta;
+    // a ring that leaves room for the next launch's CTA beside this one
+    const size_t act = gemv_smem_bytes<T>(g.ldw, 0);
+    const size_t room = act < 64 * 1024 ? (size_t)108 * 1024 - act : (kSmemLimit - 12 * 1024) - act;
+    if (act + 2 * GV_STAGE + 12 * 1024 > kSmemLimit) return invalid("an input row does not fit shared memory");
+    g.stages = (int)std::min<size_t>(GV_MAX_STAGES, std::max<size_t>(2, room / GV_STAGE));
+    return launch("gemv", gemv_kernel<T, PRO, GATED>, dim3(grid), GV_THREADS, gemv_smem_bytes<T>(g.ldw, g.stages), flags, stream, 0, g);
+}
+
+template <typename T>
+twm_status decode(const twm_dense_model* m, const twm_dense_buffers* b, int want_logits, int flags, void* stream, int sms)
+{
+    const int wp = m->width_pad;
+    float *x = b->x0, *x_next = b->x1;
+    const float* y = nullptr;
+    const float* y_norm = nullptr;
+    bool embedded = false;
+    int widest_in = 0, widest_out = 0;
+    for (int i = 0; i < m->n_layers; ++i) {
+        const Sizes s = sizes_of(m->layers[i]);
+        widest_in = std::max(widest_in, s.in);
+        widest_out = std::max(widest_out, s.out);
+    }
+    float* proj = b->vec;
+    float* att = proj + widest_in;
+    float* act = att + widest_out;
+    auto args = [&](const void* w, int N, int ldw, float* out) {
+        GemvArgs<T> g = {};
+        g.w = (const T*)w; g.N = N; g.ldw = ldw; g.out = out; g.meta = b->meta;
+        return g;
+    };
+    auto with_residual = [&](GemvArgs<T> g) {
+        g.src.tokens = embedded ? nullptr : b->tokens;
+        g.src.embed = (const T*)m->embed;
+        g.src.pos_embed = (const T*)m->pos_embed;
+        g.src.x_in = x; g.src.y = y; g.src.y_norm = y_norm; g.src.eps = m->eps; g.src.width = m->width; g.src.wp = wp;
+        g.x_out = x_next;
+        std::swap(x, x_next);
+        embedded = true;
+        y = nullptr;
+        return g;
+    };
+    for (int i = 0; i < m->n_layers; ++i) {
+        const twm_dense_layer& l = m->layers[i];
+        const Sizes s = sizes_of(l);
+        GemvArgs<T> g = with_residual(args(l.w_in, s.in, wp, proj));
+        g.shift = l.shift;
+        g.shift_state = l.shift_state;
+        if (l.shift) TRY((gemv<T, PRO_SHIFT, false>(g, sms, flags, stream)));
+        else TRY((gemv<T, PRO_RESIDUAL, false>(g, sms, flags, stream)));
+        AttnDecodeArgs<T> t;
+        t.proj = proj; t.out = att; t.q_norm = l.q_norm; t.k_norm = l.k_norm;
+        t.k_cache = (T*)l.k_cache; t.v_cache = (T*)l.v_cache; t.bias_table = l.bias_table; t.meta = b->meta;
+        t.heads = l.heads; t.kv_heads = l.kv_heads; t.dim = l.dim; t.dim_pad = l.dim_pad; t.vdim_pad = l.vdim_pad;
+        t.window = l.window; t.keep_first = l.keep_first; t.capacity = m->capacity; t.bias_len = m->bias_len; t.gated = 1;
+        t.scale = l.scale; t.eps = m->eps;
+        // about 64 visible keys or more per CTA; up to 8 CTAs a head, 16 (non-portable cluster) for long windows
+        const long visible = std::min<long>((long)l.window + l.keep_first, m->capacity);
+        int splits = 1;
+        while (splits < 8 && visible > 64L * splits) splits *= 2;
+        if (visible >= 4096 && l.kv_heads * 8 < sms) splits = 16;
+        TRY(launch("attn_decode", attn_decode_kernel<T>, dim3(splits, l.kv_heads), AD_THREADS,
+                   attn_decode_smem_bytes<T>(l.heads / l.kv_heads, l.dim_pad, l.vdim_pad), flags, stream, splits, t));
+        GemvArgs<T> o = args(l.w_out, m->width, s.out, b->y);
+        o.vec = att;
+        TRY((gemv<T, PRO_VEC, false>(o, sms, flags, stream)));
+        y = b->y; y_norm = l.norm1;
+        if (l.ff_pad > 0) {
+            TRY((gemv<T, PRO_RESIDUAL, true>(with_residual(args(l.w_gate_up, l.ff_pad, wp, act)), sms, flags, stream)));
+            GemvArgs<T> d = args(l.w_down, m->width, l.ff_pad, b->y);
+            d.vec = act;
+            TRY((gemv<T, PRO_VEC, false>(d, sms, flags, stream)));
+            y = b->y; y_norm = l.norm2;
+        }
+    }
+    if (want_logits) {
+        GemvArgs<T> h = with_residual(args(m->head, m->vocab, wp, b->logits));
+        h.final_norm = m->final_norm;
+        TRY((gemv<T, PRO_FINAL, false>(h, sms, flags, stream)));
+    }
+    return TWM_OK;
+}
+
+}  // namespace
+
+extern "C" {
+
+twm_status twm_dense_prefill(const twm_dense_model* m, const twm_dense_buffers* b, int rows, int first_pos, int n_want,
+                             float* layer_trace, int flags, void* stream)
+{
+    t_launches = 0;
+    TRY(check_model(m, b));
+    if (rows < 1 || rows > b->max_rows || n_want < 0 || n_want > rows || n_want > b->max_want) return invalid("rows or n_want");
+    if (first_pos < 0 || first_pos > m->capacity - rows) return invalid("the step runs past the slot's capacity");
+    TRY(device(nullptr));
+    return m->dtype == TWM_DENSE_F32 ? prefill<float>(m, b, rows, first_pos, n_want, layer_trace, flags, stream)
+                                     : prefill<bf16>(m, b, rows, first_pos, n_want, layer_trace, flags, stream);
+}
+
+twm_status twm_dense_decode(const twm_dense_model* m, const twm_dense_buffers* b, int want_logits, int flags, void* stream)
+{
+    t_launches = 0;
+    TRY(check_model(m, b));
+    int sms = 148;
+    TRY(device(&sms));
+    return m->dtype == TWM_DENSE_F32 ? decode<float>(m, b, want_logits, flags, stream, sms)
+                                     : decode<bf16>(m, b, want_logits, flags, stream, sms);
+}
+
+int twm_dense_launches(void) { return t_launches; }
+
+twm_status twm_dense_set_step(const twm_dense_buffers* b, int first_pos, int slot, int token, void* stream)
+{
+    if (!b || !b->meta || !b->tokens || first_pos < 0 || slot < 0) return invalid("set_step");
+    TRY(device(nullptr));
+    return launch("set_step", set_step_kernel, dim3(1), 1, 0, 0, stream, 0, b->meta, b->tokens, first_pos, slot, token);
+}
+
+size_t twm_dense_argmax_scratch_bytes(void) { return (size_t)kArgmaxParts * 8; }
+
+twm_status twm_dense_argmax_advance(const twm_dense_buffers* b, int vocab, int row, int* history, int history_capacity, void* scratch,
+                                    size_t scratch_bytes, int flags, void* stream)
+{
+    if (!b || vocab < 1 || row < 0 || row >= b->max_want || !scratch || (history && history_capacity < 1)) return invalid("argmax");
+    if (scratch_bytes < twm_dense_argmax_scratch_bytes()) return TWM_EWORKSPACE;
+    TRY(device(nullptr));
+    float* pval = (float*)scratch;
+    int* pidx = (int*)((char*)scratch + (size_t)kArgmaxParts * 4);
+    TRY(launch("argmax(partial)", ops::argmax_partial_kernel, dim3(kArgmaxParts), 256, 0, flags, stream, 0, pval, pidx,
+               (const float*)b->logits + (size_t)row * vocab, vocab));
+    return launch("argmax(final)", ops::argmax_final_kernel, dim3(1), 256, 0, flags, stream, 0, b->tokens, history, history_capacity,
+                  b->meta, b->meta + 2, b->meta + 3, (const float*)pval, (const int*)pidx, kArgmaxParts, vocab);
+}
+
+twm_status twm_dense_gemm(int dtype, const void* a, int lda, const void* w, int ldw, void* c, int ldc, int M, int N, int K,
+                          int epilogue, int kernel, int flags, void* stream)
+{
+    if (!a || !w || !c || M < 1 || N < 1 || K < 1 || lda < K || ldw < K || ldc < N) return invalid("gemm");
+    TRY(device(nullptr));
+    if (dtype == TWM_DENSE_F32)
+        return gemm<float>((const float*)a, lda, (const float*)w, ldw, c, ldc, M, N, K, epilogue, kernel, flags, stream);
+    if (dtype == TWM_DENSE_BF16)
+        return gemm<bf16>((const bf16*)a, lda, (const bf16*)w, ldw, c, ldc, M, N, K, epilogue, kernel, flags, stream);
+    return invalid("dtype");
+}
+
+twm_status twm_dense_attention(const twm_dense_model* m, int layer, const twm_dense_buffers* b, int rows, int first_pos, int kernel,
+                               int flags, void* stream)
+{
+    TRY(check_model(m, b));
+    if (layer < 0 || layer >= m->n_layers || rows < 1 || rows > b->max_rows || first_pos < 0 || first_pos > m->capacity - rows)
+        return invalid("attention");
+    TRY(device(nullptr));
+    return m->dtype == TWM_DENSE_F32 ? attention<float>(m, m->layers[layer], b, rows, first_pos, kernel, flags, stream)
+                                     : attention<bf16>(m, m->layers[layer], b, rows, first_pos, kernel, flags, stream);
+}
+
+twm_status twm_dense_device_error(void* stream, unsigned int* word)
+{
+    if (!word) return invalid("device_error");
+    cudaError_t e = cudaMemcpyFromSymbolAsync(word, g_error_word, sizeof(unsigned int), 0, cudaMemcpyDeviceToHost, (cudaStream_t)stream);
+    if (e == cudaSuccess) e = cudaStreamSynchronize((cudaStream_t)stream);
+    if (e == cudaSuccess && *word != 0) {
+        const unsigned int zero = 0;
+        e = cudaMemcpyToSymbol(g_error_word, &zero, sizeof(zero));
+    }
+    if (e != cudaSuccess) return fail("device_error", e);
+    return *word ? TWM_ETIMEOUT : TWM_OK;
+}
+
+const char* twm_dense_status_string(int s)
+{
+    switch (s) {
+        case TWM_OK: return "ok";
+        case TWM_EINVAL: return "invalid argument";
+        case TWM_EWORKSPACE: return "scratch missing or too small";
+        case TWM_ELAUNCH: return "CUDA launch or copy failed";
+        case TWM_EARCH: return "device is not sm_100 (B200)";
+        case TWM_ETIMEOUT: return "a bounded device-side wait expired";
+    }
+    return "unknown status";
+}
+
+const char* twm_dense_last_error(void) { return t_last_error; }
+
+}  // extern "C"

@@ -6,16 +6,19 @@ import re
 
 import pytest
 
-from tensorwarp_b200 import _lib
+from tensorwarp_b200 import _dense, _lib
 
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 
 
-def _declared_symbols():
+DENSE_HEADER = "twm_dense.h"           # declares a library of its own
+
+
+def _declared_symbols(dense=False):
     names = set()
     inc = os.path.join(ROOT, "include")
     for fn in sorted(os.listdir(inc)):
-        if fn.endswith(".h"):
+        if fn.endswith(".h") and (fn == DENSE_HEADER) == dense:
             text = open(os.path.join(inc, fn)).read()
             text = re.sub(r"/\*.*?\*/", "", text, flags=re.S)
             names.update(re.findall(r"\b(twm_[a-z0-9_]+)\s*\(", text))
@@ -28,6 +31,14 @@ def test_every_declared_symbol_is_exported_and_bound(twm_lib):
     for name in names:
         assert hasattr(twm_lib, name), f"{name} declared in twmarlin.h but not exported"
         assert name in _lib.SIGNATURES, f"{name} has no ctypes signature"
+
+
+def test_every_symbol_of_the_dense_library_is_exported_and_bound():
+    names = _declared_symbols(dense=True)
+    assert "twm_dense_prefill" in names and "twm_dense_decode" in names
+    assert set(names) == set(_dense.SIGNATURES)
+    for name in names:
+        assert hasattr(_dense.lib(), name), f"{name} declared in {DENSE_HEADER} but not exported"
 
 
 def test_version_and_status_strings(twm_lib):
