@@ -700,6 +700,183 @@ def decode_tok_s(torch, device, new_tokens: int = 64, kv_len: int = 2048):
     return out
 
 
+# ------------------------------------------------------- dense-weight decoders --
+
+# width, layers, query heads, key/value heads, head size, feed-forward, vocabulary, window, kept first keys
+BIDASUN_SIZES = {
+    "1b": dict(width=2048, layers=16, heads=16, kv_heads=4, dim=128, ff=8192, vocab=32768, window=512, keep=4),
+    "7b": dict(width=3584, layers=28, heads=28, kv_heads=4, dim=128, ff=18944, vocab=152064, window=1024, keep=4),
+    "13b-wide": dict(width=5120, layers=12, heads=40, kv_heads=8, dim=128, ff=13824, vocab=32768, window=2048, keep=4),
+}
+BIDASUN_PROMPTS = (128, 512, 2048, 8192)
+BIDASUN_CONTEXT = 2048
+
+
+def bidasun_config(size: dict, max_positions: int) -> dict:
+    mixer = {"heads": size["heads"], "kv_heads": size["kv_heads"], "dim": size["dim"], "vdim": size["dim"],
+             "scale": size["dim"] ** -0.5, "mask": {"size": size["window"], "keep_first": size["keep"]}}
+    return {"architecture": "Bidasun", "width": size["width"], "vocab": size["vocab"], "max_positions": max_positions,
+            "norm": {"eps": 1e-5},
+            "layers": [{"type": "attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": size["ff"]}}] * size["layers"]}
+
+
+def random_bidasun(torch, config: dict, device, **engine_options):
+    """An engine on random bfloat16 weights of the configuration."""
+    from tensorwarp_b200 import dense
+    from tensorwarp_b200.engine import DenseEngine
+    from tensorwarp_b200.models import bidasun
+    gen = torch.Generator(device=device).manual_seed(1)
+
+    def get(name, shape):
+        leaf = name.split(".")[-1]
+        if leaf.startswith("norm"):
+            return torch.ones(shape, device=device)
+        if leaf == "pb":
+            return torch.full(shape, -4.0, device=device)
+        if leaf in ("shift", "r1", "r2"):
+            return torch.rand(shape, generator=gen, device=device)
+        return (torch.randn(shape, generator=gen, device=device, dtype=torch.float32) * 0.02).bfloat16()
+
+    spec = bidasun.parse_config(config)
+    model = dense.DenseModel(spec, bidasun.model_tensors(spec, get), torch.bfloat16, device)
+    return DenseEngine(model, **engine_options)
+
+
+def bidasun_figures(torch, device, name: str, gbs: float, tflops: float) -> dict:
+    """Prefill and decode throughput of one size, and its products and attention one by one."""
+    import ctypes as C
+
+    from tensorwarp_b200 import _dense
+    size = BIDASUN_SIZES[name]
+    eng = random_bidasun(torch, bidasun_config(size, 8192 + 64), device, max_live=1, portion=8192)
+    lib, model = _dense.lib(), eng.model
+    w, h, g, d, ff, v, nl = (size[k] for k in ("width", "heads", "kv_heads", "dim", "ff", "vocab", "layers"))
+    matrices = nl * (w * (2 * h * d + 2 * g * d) + h * d * w + 3 * w * ff)
+    gen = torch.Generator(device=device).manual_seed(3)
+    eng._buf["tokens"].copy_(torch.randint(0, v, eng._buf["tokens"].shape, generator=gen, device=device, dtype=torch.int32))
+    eng._buf["want"].zero_()
+    torch.cuda.synchronize()
+
+    def timed(enqueue, steps, warm=3):
+        with torch.cuda.stream(eng.stream):
+            for _ in range(warm):
+                enqueue()
+            torch.cuda.synchronize()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record(eng.stream)
+            for _ in range(steps):
+                enqueue()
+            e1.record(eng.stream)
+            torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / steps
+
+    def visible(n):                                  # query-key pairs of an n-token prompt
+        full = sum(min(i + 1, size["window"]) for i in range(n))
+        return full + sum(min(max(i + 1 - size["window"], 0), size["keep"]) for i in range(n))
+
+    out = {"config": {k: size[k] for k in size}, "matrix_weights": matrices, "prefill": [], "decode": []}
+    for n in BIDASUN_PROMPTS:
+        eng._set_step(0, 0)
+        ms = timed(lambda: eng.enqueue_prefill(n, 0, 1), 5)
+        flops = 2.0 * n * matrices + nl * 4.0 * h * d * visible(n) + 2.0 * w * v
+        out["prefill"].append({"tokens": n, "ms": round(ms, 3), "tok_s": round(n / ms * 1e3), "tflops": round(flops / ms / 1e9, 1),
+                               "frac_bf16_peak": round(flops / ms / 1e9 / tflops, 3), "launches": eng.launches_per_step})
+    for ctx in (BIDASUN_CONTEXT, 8000):
+        eng._set_step(ctx, 0, 1)
+        graph = eng.capture_decode("greedy")
+        ms = timed(graph.replay, 32)
+        keys = min(ctx, size["window"] + size["keep"])
+        nbytes = 2 * (matrices + v * w) + nl * keys * 2 * g * d * 2
+        out["decode"].append({"context": ctx, "ms": round(ms, 4), "tok_s": round(1e3 / ms, 1), "bytes": nbytes,
+                              "hbm_gbs": round(nbytes / ms / 1e6, 1), "frac_hbm": round(nbytes / ms / 1e6 / gbs, 3),
+                              "launches": eng.launches_per_step})
+
+    # each product of a layer at each prompt length, over the layers' own weights in turn (larger than L2 together)
+    b, p = eng._buf, []
+    shapes = [("q|k|v|gate", "w_in", "a", "proj", 2 * h * d + 2 * g * d, w, _dense.EPI_STORE),
+              ("out", "w_out", "att", "y", w, h * d, _dense.EPI_STORE_F32),
+              ("gate_up", "w_gate_up", "a", "act", ff, w, _dense.EPI_GELU_GLU),
+              ("down", "w_down", "act", "y", w, ff, _dense.EPI_STORE_F32)]
+    for n in BIDASUN_PROMPTS:
+        row = {"tokens": n}
+        for label, wt, src, dst, cols, k, epi in shapes:
+            def enqueue():
+                for lw in model.layers:
+                    _dense.check(lib.twm_dense_gemm(_dense.TWM_DENSE_BF16, b[src].data_ptr(), b[src].shape[1], lw[wt].data_ptr(), k,
+                                                    b[dst].data_ptr(), b[dst].shape[1], n, cols, k, epi, 0, eng.flags,
+                                                    eng.stream.cuda_stream), "gemm")
+            ms = timed(enqueue, 2, 1) / nl
+            tf = 2.0 * n * k * cols * (2 if epi == _dense.EPI_GELU_GLU else 1) / ms / 1e9
+            nb = 2 * k * cols * (2 if epi == _dense.EPI_GELU_GLU else 1)
+            row[label] = {"us": round(ms * 1e3, 1), "tflops": round(tf, 1),
+                          "frac_roofline": round(max(tf / tflops, nb / ms / 1e6 / gbs), 3)}
+        eng._set_step(0, 0)
+
+        def attend():
+            for i in range(nl):
+                _dense.check(lib.twm_dense_attention(C.byref(eng._desc), i, C.byref(eng._b), n, 0, 0, eng.flags,
+                                                     eng.stream.cuda_stream), "attention")
+        ms = timed(attend, 2, 1) / nl
+        tf = 4.0 * h * d * visible(n) / ms / 1e9
+        row["attention"] = {"us": round(ms * 1e3, 1), "tflops": round(tf, 1), "frac_roofline": round(tf / tflops, 3)}
+        p.append(row)
+    out["prefill_kernels"] = p
+    out["device_error"] = _dense.device_error()
+    return out
+
+
+def q4_decode_same_size(torch, device, name: str, gbs: float) -> dict:
+    """The 4-bit decoder's step at the same width, heads, feed-forward, vocabulary and depth (its attention sees the
+    whole context)."""
+    from tensorwarp_b200 import generate as gen
+    size = BIDASUN_SIZES[name]
+    cfg = gen.TransformerConfig(hidden=size["width"], num_heads=size["heads"], num_kv_heads=size["kv_heads"], head_dim=size["dim"],
+                                ffn=size["ff"], vocab=size["vocab"], layers=size["layers"], max_seq=BIDASUN_CONTEXT + 256)
+    eng = gen.QuantizedGenerationEngine(gen.Q4Model(cfg, device=device))
+    eng.prefill_random_kv(BIDASUN_CONTEXT)
+    eng.capture()
+    eng.set_token(1)
+    torch.cuda.synchronize()
+    with torch.cuda.stream(eng.stream):
+        for _ in range(3):
+            eng.replay()
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record(eng.stream)
+        for _ in range(32):
+            eng.replay()
+        e1.record(eng.stream)
+        torch.cuda.synchronize()
+    ms = e0.elapsed_time(e1) / 32
+    nbytes = sum(algorithmic_bytes(1, n, k, GROUP) for k, n in
+                 ((cfg.hidden, cfg.q_dim + 2 * cfg.kv_dim), (cfg.q_dim, cfg.hidden), (cfg.hidden, 2 * cfg.ffn), (cfg.ffn, cfg.hidden)))
+    nbytes = cfg.layers * (nbytes + 4 * BIDASUN_CONTEXT * cfg.kv_dim) + 2 * cfg.vocab * cfg.hidden
+    return {"context": BIDASUN_CONTEXT, "ms": round(ms, 4), "tok_s": round(1e3 / ms, 1), "bytes": nbytes,
+            "hbm_gbs": round(nbytes / ms / 1e6, 1), "frac_hbm": round(nbytes / ms / 1e6 / gbs, 3), "launches": eng.launches_per_step}
+
+
+def run_bidasun(args):
+    import torch
+    torch.cuda.set_device(0)
+    device = torch.device("cuda", 0)
+    gbs, source = measured_peak_gbs()
+    tflops = 1590.0
+    path = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    if os.path.exists(path):
+        with open(path) as f:
+            tflops = float(json.load(f)["bf16_tflops"])
+    line = {"bench": "bidasun", "data": "random weights and tokens", "dtype": "bf16", "peaks": {"hbm_gbs": gbs, "bf16_tflops": tflops,
+            "source": source}, "sizes": {}}
+    with ClockSampler(0) as clocks:
+        for name in args.sizes.split(","):
+            line["sizes"][name] = bidasun_figures(torch, device, name, gbs, tflops)
+            torch.cuda.empty_cache()
+            line["sizes"][name]["q4_decode_same_size"] = q4_decode_same_size(torch, device, name, gbs)
+            torch.cuda.empty_cache()
+    line["clocks"] = clocks.summary()
+    print(json.dumps(line), flush=True)
+
+
 # ------------------------------------------------------------- tensor parallel --
 
 def run_tp(args):
@@ -1069,8 +1246,13 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-decode", action="store_true", help="skip the configs[3] decode tok/s measurement")
+    ap.add_argument("--workload", default="w4a16", choices=["w4a16", "bidasun"],
+                    help="bidasun: prefill and decode of the Bidasun decoder at a few sizes, beside the 4-bit decoder's step")
+    ap.add_argument("--sizes", default="1b,7b,13b-wide", help="--workload bidasun: which sizes")
     args = ap.parse_args()
-    if args.impl == "reference":
+    if args.workload == "bidasun":
+        run_bidasun(args)
+    elif args.impl == "reference":
         args.steps = args.steps if args.steps is not None else 5
         args.warmup = args.warmup if args.warmup is not None else 1
         args.steps = min(args.steps, 20)          # each step is about two seconds of CPU work: the run stays under a minute

@@ -3,11 +3,15 @@
 #include <algorithm>
 #include <cstdio>
 #include <mutex>
+#include <type_traits>
+#include <unordered_map>
 
+#include "twm_dense_attn.cuh"
 #include "twm_dense_common.cuh"
 #include "twm_dense_decode.cuh"
 #include "twm_dense_rows.cuh"
 #include "twm_dense_simt.cuh"
+#include "twm_dense_tc.cuh"
 
 namespace {
 
@@ -135,11 +139,134 @@ twm_status check_model(const twm_dense_model* m, const twm_dense_buffers* b)
     return TWM_OK;
 }
 
+// ------------------------------------------------------------ tensor maps --
+typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
+                                  const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
+                                  CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+EncodeTiledFn encode_tiled()
+{
+    static EncodeTiledFn fn = []() -> EncodeTiledFn {
+        void* ptr = nullptr;
+        cudaDriverEntryPointQueryResult q;
+        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &ptr, cudaEnableDefault, &q) != cudaSuccess ||
+            q != cudaDriverEntryPointSuccess)
+            return nullptr;
+        return reinterpret_cast<EncodeTiledFn>(ptr);
+    }();
+    return fn;
+}
+
+// bf16 [rows][cols] with row stride ld, boxes of 64 columns x box_rows, 128-byte swizzle, zeros outside.  A map is a
+// pure description of memory, so maps are kept by what they describe.
+struct MapKey {
+    const void* ptr; long rows, cols, ld; int box;
+    bool operator==(const MapKey& o) const { return ptr == o.ptr && rows == o.rows && cols == o.cols && ld == o.ld && box == o.box; }
+};
+struct MapHash {
+    size_t operator()(const MapKey& k) const {
+        size_t h = (size_t)k.ptr;
+        for (size_t v : {(size_t)k.rows, (size_t)k.cols, (size_t)k.ld, (size_t)k.box}) h = h * 1000003u ^ v;
+        return h;
+    }
+};
+bool rows_map(CUtensorMap* map, const void* ptr, long rows, long cols, long ld, int box_rows)
+{
+    static std::unordered_map<MapKey, CUtensorMap, MapHash> cache;
+    static std::mutex mutex;
+    const MapKey key{ptr, rows, cols, ld, box_rows};
+    std::lock_guard<std::mutex> lock(mutex);
+    auto it = cache.find(key);
+    if (it != cache.end()) { *map = it->second; return true; }
+    EncodeTiledFn enc = encode_tiled();
+    if (!enc) return false;
+    const cuuint64_t gdim[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
+    const cuuint64_t gstride[1] = {(cuuint64_t)ld * 2};
+    const cuuint32_t box[2] = {(cuuint32_t)TC_BK, (cuuint32_t)box_rows};
+    const cuuint32_t estride[2] = {1, 1};
+    if (enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(ptr), gdim, gstride, box, estride,
+            CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+            CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
+        return false;
+    if (cache.size() > 4096) cache.clear();
+    cache.emplace(key, *map);
+    return true;
+}
+
 // ------------------------------------------------------------- operations --
+// The tcgen05 product takes rows that start on 16-byte boundaries.
+bool tc_fits(const void* a, int lda, const void* w, int ldw)
+{
+    return lda % 8 == 0 && ldw % 8 == 0 && ((uintptr_t)a & 15) == 0 && ((uintptr_t)w & 15) == 0;
+}
+
+template <int BN, int EPI>
+twm_status gemm_tc_launch(const bf16* a, int lda, const bf16* w, int ldw, void* c, int ldc, int M, int N, int K, int sms, int flags,
+                          void* stream)
+{
+    constexpr bool gated = EPI == TWM_EPI_GELU_GLU;
+    constexpr int out = gated ? BN / 2 : BN;
+    TcArgs g;
+    g.c = c; g.ldc = ldc; g.M = M; g.N = N; g.K = K;
+    g.m_tiles = (M + TC_BM - 1) / TC_BM;
+    g.n_tiles = (N + out - 1) / out;
+    if (!rows_map(&g.a_map, a, M, K, lda, TC_BM) || !rows_map(&g.w_map, w, gated ? 2L * N : N, K, ldw, out))
+        return invalid("cuTensorMapEncodeTiled refused a map of the tcgen05 product");
+    return launch("gemm_tc", gemm_tc_kernel<BN, EPI>, dim3(std::min(sms, g.m_tiles * g.n_tiles)), TC_THREADS, TcCfg<BN>::SMEM_BYTES,
+                  flags, stream, 0, g);
+}
+
+// Column width of a tile: the one whose waves cost least.  Measured time of one 64-K stage of a wave of tiles:
+// 0.42, 0.25 and 0.20 us for 256, 128 and 64 columns.
+int tc_tile_width(int M, int N, bool gated, int sms)
+{
+    int best = 256;
+    long best_cost = -1;
+    for (int bn : {256, 128, 64}) {
+        const int out = gated ? bn / 2 : bn;
+        const long tiles = (long)((M + TC_BM - 1) / TC_BM) * ((N + out - 1) / out);
+        const long cost = ((tiles + sms - 1) / sms) * (bn == 256 ? 42 : bn == 128 ? 25 : 20);
+        if (best_cost < 0 || cost < best_cost) { best = bn; best_cost = cost; }
+    }
+    return best;
+}
+
+template <int EPI>
+twm_status gemm_tc(const bf16* a, int lda, const bf16* w, int ldw, void* c, int ldc, int M, int N, int K, int width, int flags,
+                   void* stream)
+{
+    int sms = 148;
+    TRY(device(&sms));
+    if (width == 0) width = tc_tile_width(M, N, EPI == TWM_EPI_GELU_GLU, sms);
+    switch (width) {
+        case 256: return gemm_tc_launch<256, EPI>(a, lda, w, ldw, c, ldc, M, N, K, sms, flags, stream);
+        case 128: return gemm_tc_launch<128, EPI>(a, lda, w, ldw, c, ldc, M, N, K, sms, flags, stream);
+        default: return gemm_tc_launch<64, EPI>(a, lda, w, ldw, c, ldc, M, N, K, sms, flags, stream);
+    }
+}
+twm_status gemm_tc_any(const float*, int, const float*, int, void*, int, int, int, int, int, int, int, void*)
+{
+    return invalid("the tcgen05 product takes bfloat16");
+}
+twm_status gemm_tc_any(const bf16* a, int lda, const bf16* w, int ldw, void* c, int ldc, int M, int N, int K, int epi, int width,
+                       int flags, void* stream)
+{
+    switch (epi) {
+        case TWM_EPI_STORE: return gemm_tc<TWM_EPI_STORE>(a, lda, w, ldw, c, ldc, M, N, K, width, flags, stream);
+        case TWM_EPI_STORE_F32: return gemm_tc<TWM_EPI_STORE_F32>(a, lda, w, ldw, c, ldc, M, N, K, width, flags, stream);
+        case TWM_EPI_GELU_GLU: return gemm_tc<TWM_EPI_GELU_GLU>(a, lda, w, ldw, c, ldc, M, N, K, width, flags, stream);
+    }
+    return invalid("epilogue");
+}
+
 template <typename T>
 twm_status gemm(const T* a, int lda, const T* w, int ldw, void* c, int ldc, int M, int N, int K, int epi, int kernel, int flags,
                 void* stream)
 {
+    const bool fits = std::is_same<T, bf16>::value && tc_fits(a, lda, w, ldw);
+    if (kernel != 0 && kernel != 1 && kernel != 2 && kernel != 64 && kernel != 128 && kernel != 256) return invalid("kernel");
+    if (kernel >= 2 && !fits) return invalid("the tcgen05 product takes bfloat16 rows on 16-byte boundaries");
+    if (kernel >= 2 || (kernel == 0 && fits))
+        return gemm_tc_any(a, lda, w, ldw, c, ldc, M, N, K, epi, kernel > 2 ? kernel : 0, flags, stream);
     const dim3 grid((N + ST - 1) / ST, (M + ST - 1) / ST);
     switch (epi) {
         case TWM_EPI_STORE:
@@ -171,11 +298,28 @@ AttnArgs<T> attn_args(const twm_dense_model* m, const twm_dense_layer& l, const 
     return g;
 }
 
+template <int DV>
+twm_status attention_mma(const AttnArgs<bf16>& g, int flags, void* stream)
+{
+    auto kernel = g.dim_pad == 128 ? attn_mma_kernel<128, DV> : g.dim_pad == 64 ? attn_mma_kernel<64, DV> : attn_mma_kernel<0, DV>;
+    return launch("attn_mma", kernel, dim3((g.rows + AM_Q - 1) / AM_Q, g.heads, (g.vdim_pad + DV - 1) / DV), AM_THREADS,
+                  attn_mma_smem_bytes<DV>(g.dim_pad), flags, stream, 0, g);
+}
+bool attention_tiles_fit(const AttnArgs<bf16>& g) { return attn_mma_smem_bytes<128>(g.dim_pad) <= kSmemLimit; }
+bool attention_tiles_fit(const AttnArgs<float>&) { return false; }
+twm_status attention_tiles(const AttnArgs<bf16>& g, int flags, void* stream)
+{
+    return g.vdim_pad <= 64 ? attention_mma<64>(g, flags, stream) : attention_mma<128>(g, flags, stream);
+}
+twm_status attention_tiles(const AttnArgs<float>&, int, void*) { return invalid("the tensor-core attention takes bfloat16"); }
+
 template <typename T>
 twm_status attention(const twm_dense_model* m, const twm_dense_layer& l, const twm_dense_buffers* b, int rows, int first_pos,
                      int kernel, int flags, void* stream)
 {
     const AttnArgs<T> g = attn_args<T>(m, l, b, rows);
+    if (kernel == 2 && !attention_tiles_fit(g)) return invalid("the tensor-core attention takes bfloat16 heads that fit shared memory");
+    if (kernel == 2 || (kernel == 0 && attention_tiles_fit(g))) return attention_tiles(g, flags, stream);
     const int vblock = AS_VPT * AS_THREADS;
     return launch("attn_simt", attn_simt_kernel<T>, dim3(rows, l.heads, (l.vdim_pad + vblock - 1) / vblock), AS_THREADS,
                   sizeof(float) * (size_t)(l.dim_pad + AS_THREADS), flags, stream, 0, g);
@@ -254,13 +398,13 @@ template <typename T, int PRO, bool GATED>
 twm_status gemv(GemvArgs<T> g, int sms, int flags, void* stream)
 {
     const int out_rows = GATED ? GV_ROWS / 2 : GV_ROWS;
-    g.rows_per_cta = std::max((g.N + sms - 1) / sms, std::min(out_rows, g.N));
-    const int grid = (g.N + g.rows_per_cta - 1) / g.rows_per_cta;
-    // a ring that leaves room for the next launch's CTA beside this one
-    const size_t act = gemv_smem_bytes<T>(g.ldw, 0);
-    const size_t room = act < 64 * 1024 ? (size_t)108 * 1024 - act : (kSmemLimit - 12 * 1024) - act;
-    if (act + 2 * GV_STAGE + 12 * 1024 > kSmemLimit) return invalid("an input row does not fit shared memory");
-    g.stages = (int)std::min<size_t>(GV_MAX_STAGES, std::max<size_t>(2, room / GV_STAGE));
+    const int grid = std::min(sms, (g.N + out_rows - 1) / out_rows);
+    g.rounds = g.N / (grid * out_rows);
+    const int left = g.N - g.rounds * grid * out_rows;
+    g.last_rows = (left + grid - 1) / grid;
+    const size_t act = gemv_smem_bytes<T>(g.ldw, 0), limit = kSmemLimit - 8 * 1024;      // static shared memory beside it
+    if (act + 2 * GV_STAGE > limit) return invalid("an input row does not fit shared memory");
+    g.stages = (int)std::min<size_t>(GV_MAX_STAGES, (limit - act) / GV_STAGE);
     return launch("gemv", gemv_kernel<T, PRO, GATED>, dim3(grid), GV_THREADS, gemv_smem_bytes<T>(g.ldw, g.stages), flags, stream, 0, g);
 }
 
@@ -311,11 +455,11 @@ twm_status decode(const twm_dense_model* m, const twm_dense_buffers* b, int want
         t.heads = l.heads; t.kv_heads = l.kv_heads; t.dim = l.dim; t.dim_pad = l.dim_pad; t.vdim_pad = l.vdim_pad;
         t.window = l.window; t.keep_first = l.keep_first; t.capacity = m->capacity; t.bias_len = m->bias_len; t.gated = 1;
         t.scale = l.scale; t.eps = m->eps;
-        // about 64 visible keys or more per CTA; up to 8 CTAs a head, 16 (non-portable cluster) for long windows
+        // about 64 visible keys per CTA, up to 16 CTAs a head (a cluster; more than 8 is the non-portable size), and no
+        // more CTAs than one wave
         const long visible = std::min<long>((long)l.window + l.keep_first, m->capacity);
         int splits = 1;
-        while (splits < 8 && visible > 64L * splits) splits *= 2;
-        if (visible >= 4096 && l.kv_heads * 8 < sms) splits = 16;
+        while (splits < 16 && visible > 64L * splits && l.kv_heads * splits * 2 <= sms) splits *= 2;
         TRY(launch("attn_decode", attn_decode_kernel<T>, dim3(splits, l.kv_heads), AD_THREADS,
                    attn_decode_smem_bytes<T>(l.heads / l.kv_heads, l.dim_pad, l.vdim_pad), flags, stream, splits, t));
         GemvArgs<T> o = args(l.w_out, m->width, s.out, b->y);

@@ -70,6 +70,14 @@ __device__ __forceinline__ float group_sum(float v, float* red, int threads, int
 }
 __device__ __forceinline__ float inv_rms(float sumsq, int n, float eps) { return 1.0f / sqrtf(sumsq / (float)n + eps); }
 
+// True in one lane of a converged warp.  Code under it is known to run in one thread, which the tensor-core and TMA
+// instructions (uniform operands) issue faster from than from a lane-number test.
+__device__ __forceinline__ bool elect_one() {
+    uint32_t p;
+    asm volatile("{\n\t.reg .pred p;\n\telect.sync _|p, 0xffffffff;\n\tselp.u32 %0, 1, 0, p;\n\t}" : "=r"(p));
+    return p != 0;
+}
+
 // Which keys the query at position p sees: [0, sinks) and [lo, p].
 __device__ __forceinline__ void visible_range(int p, int window, int keep_first, int& sinks, int& lo) {
     lo = window > p ? 0 : p - window + 1;               // p - j < window

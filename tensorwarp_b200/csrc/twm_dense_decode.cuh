@@ -1,10 +1,13 @@
 // twm_dense_decode.cuh — one decoded token of a dense model: the streaming matrix-vector product and
 // the split-key attention.
 //
-// gemv_kernel: y = W a for one token, HBM-bound.  A CTA owns a run of W's rows.  One warp streams them
-// with 1-D bulk copies into a shared-memory ring, eight row pieces of 2 KB a stage, and starts
-// before the preceding kernel has finished (weights are constants); eight warps multiply: warps 0-3 the
-// stage's rows 0-3, a quarter of the piece each, warps 4-7 the rows 4-7.  The steps between two products
+// gemv_kernel: y = W a for one token, HBM-bound.  The CTAs (one per SM) take W's rows eight at a time in
+// turn, so that together they read one contiguous window of it; what is left after the last full round is
+// shared out evenly.  One thread streams them with 1-D bulk copies into a shared-memory ring, eight row
+// pieces of 2 KB a stage, and starts before the preceding kernel has finished (weights are constants);
+// eight warps multiply: warps 0-3 the stage's rows 0-3, a quarter of the piece each, warps 4-7 the rows 4-7.
+// A CTA asks for more than half an SM's shared memory: with two to an SM, those of the next launch would
+// gather on the SMs that happen to be free.  The steps between two products
 // are its prologue: every CTA makes the product's input row itself, from the residual stream and the
 // sublayer output that joins it (norm, add, token shift or final norm), in FP32, and rounds it once.
 // The epilogue of the gate/up product applies the gated activation, so no launch stands between products
@@ -25,7 +28,7 @@ constexpr int GV_THREADS = GV_CONSUMERS + 32;
 constexpr int GV_ROWS = 8;                  // rows per stage
 constexpr int GV_PIECE = 2048;              // bytes of a row per stage
 constexpr int GV_STAGE = GV_ROWS * GV_PIECE;
-constexpr int GV_MAX_STAGES = 8;
+constexpr int GV_MAX_STAGES = 9;
 constexpr int GV_FLUSH = 16;                // row groups between two cross-warp sums
 
 template <typename T>
@@ -33,7 +36,8 @@ struct GemvArgs {
     const T* w;                 // [N (gated: N gate rows, then N up rows)][ldw]
     int N, ldw;                 // ldw = K: padded, a multiple of 16 bytes
     float* out;                 // [N]
-    int rows_per_cta, stages;
+    int rounds, last_rows;      // full rounds of row groups over the grid, then rows per CTA of what is left (0 = none)
+    int stages;
     const float* vec;           // PRO_VEC: the input row, f32 [ldw]
     ResidualSource<T> src;      // otherwise: row 0 of the residual stream
     float* x_out;               // the residual row after the add, written by CTA 0
@@ -64,8 +68,11 @@ gemv_kernel(const GemvArgs<T> g)
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     constexpr int OUT_ROWS = GATED ? GV_ROWS / 2 : GV_ROWS;         // outputs per row group
-    const int n_begin = blockIdx.x * g.rows_per_cta, n_end = min(g.N, n_begin + g.rows_per_cta);
-    const int groups = (n_end - n_begin + OUT_ROWS - 1) / OUT_ROWS;
+    const int last_first = g.rounds * (int)gridDim.x * OUT_ROWS + (int)blockIdx.x * g.last_rows;
+    const int last_valid = max(0, min(g.last_rows, g.N - last_first));
+    const int groups = g.rounds + (last_valid > 0 ? 1 : 0);
+    auto group_first = [&](int gi) { return gi < g.rounds ? (gi * (int)gridDim.x + (int)blockIdx.x) * OUT_ROWS : last_first; };
+    auto group_rows = [&](int gi) { return gi < g.rounds ? OUT_ROWS : last_valid; };
     const int row_bytes = g.ldw * (int)sizeof(T);
     const int chunks = (row_bytes + GV_PIECE - 1) / GV_PIECE;
     const int iters = groups * chunks;
@@ -80,23 +87,27 @@ gemv_kernel(const GemvArgs<T> g)
 
     if (warp == GV_CONSUMERS / 32) {
         // ------------------------------------------------------------ producer --
-        int slot = 0, c = 0, gi = 0;
-        uint32_t phase = 1;                                          // a fresh barrier passes a wait for the phase before
-        for (int it = 0; it < iters; ++it) {
-            if (it >= g.stages && !mbar_wait_bounded(&empty[slot], phase, abort_flag)) break;
-            const int bytes = min(GV_PIECE, row_bytes - c * GV_PIECE);
-            const int o0 = n_begin + gi * OUT_ROWS;
-            const int valid = min(OUT_ROWS, n_end - o0);             // outputs of this group
-            if (lane == 0) mbar_arrive_expect_tx(&full[slot], (uint32_t)bytes * (uint32_t)(GATED ? 2 * valid : valid));
-            __syncwarp();
-            if (lane < GV_ROWS && (GATED ? (lane & 3) : lane) < valid) {
-                const int row = GATED ? (lane < 4 ? o0 + lane : g.N + o0 + lane - 4) : o0 + lane;
-                bulk_g2s(ring + (size_t)slot * GV_STAGE + lane * GV_PIECE,
-                         reinterpret_cast<const uint8_t*>(g.w) + (size_t)row * row_bytes + (size_t)c * GV_PIECE, (uint32_t)bytes,
-                         &full[slot]);
+        if (elect_one()) {
+            int slot = 0, c = 0, gi = 0;
+            uint32_t phase = 0;
+            for (int it = 0; it < iters; ++it) {
+                if (it >= g.stages && !mbar_wait_bounded(&empty[slot], phase, abort_flag)) break;
+                const int bytes = min(GV_PIECE, row_bytes - c * GV_PIECE);
+                const int o0 = group_first(gi), valid = group_rows(gi);      // outputs of this group
+                mbar_arrive_expect_tx(&full[slot], (uint32_t)bytes * (uint32_t)(GATED ? 2 * valid : valid));
+                uint8_t* dst = ring + (size_t)slot * GV_STAGE;
+                const uint8_t* src = reinterpret_cast<const uint8_t*>(g.w) + (size_t)o0 * row_bytes + (size_t)c * GV_PIECE;
+#pragma unroll
+                for (int r = 0; r < OUT_ROWS; ++r) {
+                    if (r < valid) {
+                        bulk_g2s(dst + r * GV_PIECE, src + (size_t)r * row_bytes, (uint32_t)bytes, &full[slot]);
+                        if (GATED)
+                            bulk_g2s(dst + (r + OUT_ROWS) * GV_PIECE, src + (size_t)(g.N + r) * row_bytes, (uint32_t)bytes, &full[slot]);
+                    }
+                }
+                if (++c == chunks) { c = 0; ++gi; }
+                if (++slot == g.stages) { slot = 0; if (it >= g.stages) phase ^= 1u; }
             }
-            if (++c == chunks) { c = 0; ++gi; }
-            if (++slot == g.stages) { slot = 0; if (it >= g.stages) phase ^= 1u; else phase = 0; }
         }
         return;
     }
@@ -108,22 +119,15 @@ gemv_kernel(const GemvArgs<T> g)
     } else {
         const int pos = g.meta[0];
         const int tok = g.src.tokens != nullptr ? g.src.tokens[0] : 0;
-        const float ir = g.src.row_inv_rms(0, red, GV_CONSUMERS, 1);
         const int wp = g.src.wp, nvec = wp >> 2;
-        float fr = 1.0f;
-        if (PRO == PRO_FINAL) {
-            float ss = 0.0f;
-            for (int i = tid; i < nvec; i += GV_CONSUMERS) ss += ops::sumsq4(g.src.at(0, pos, tok, i, ir));
-            fr = inv_rms(group_sum(ss, red, GV_CONSUMERS, 1), g.src.width, g.src.eps);
-        }
         const bool writer = blockIdx.x == 0;
         float* st = PRO == PRO_SHIFT ? g.shift_state + (size_t)g.meta[1] * 2 * wp : nullptr;
-        for (int i = tid; i < nvec; i += GV_CONSUMERS) {
-            const float4 x = g.src.at(0, pos, tok, i, ir);
+        const float* st_before = PRO == PRO_SHIFT && pos > 0 ? st + (size_t)((pos - 1) & 1) * wp : nullptr;
+        float fr = 1.0f;
+        // element i of the residual row x; before = the state's, for the token shift
+        auto finish = [&](int i, const float4 x, const float4 before) {
             float4 h = x;
             if (PRO == PRO_SHIFT) {
-                const float4 before = pos > 0 ? reinterpret_cast<const float4*>(st + (size_t)((pos - 1) & 1) * wp)[i]
-                                              : make_float4(0.f, 0.f, 0.f, 0.f);
                 h = shift4(x, before, __ldg(reinterpret_cast<const float4*>(g.shift) + i));
                 if (writer) reinterpret_cast<float4*>(st + (size_t)(pos & 1) * wp)[i] = x;      // the other half of the pair
             }
@@ -133,6 +137,49 @@ gemv_kernel(const GemvArgs<T> g)
             }
             if (writer && g.x_out != nullptr) reinterpret_cast<float4*>(g.x_out)[i] = x;
             store4<T>(as + i * 4, h);
+        };
+        auto state_at = [&](int i) {
+            return st_before != nullptr ? reinterpret_cast<const float4*>(st_before)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+        };
+        constexpr int PER = 4;
+        if (nvec <= PER * GV_CONSUMERS && g.src.tokens == nullptr && g.src.y != nullptr && g.src.y_norm != nullptr) {
+            // rows of up to 4096: everything is requested before the first use
+            const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+            float4 x[PER], y[PER], before[PER];
+#pragma unroll
+            for (int j = 0; j < PER; ++j) {
+                const int i = tid + j * GV_CONSUMERS;
+                const bool in = i < nvec;
+                y[j] = in ? reinterpret_cast<const float4*>(g.src.y)[i] : zero;
+                x[j] = in ? reinterpret_cast<const float4*>(g.src.x_in)[i] : zero;
+                before[j] = PRO == PRO_SHIFT && in ? state_at(i) : zero;
+            }
+            float ss = 0.0f;
+#pragma unroll
+            for (int j = 0; j < PER; ++j) ss += ops::sumsq4(y[j]);
+            const float ir = inv_rms(group_sum(ss, red, GV_CONSUMERS, 1), g.src.width, g.src.eps);
+            ss = 0.0f;
+#pragma unroll
+            for (int j = 0; j < PER; ++j) {
+                const int i = tid + j * GV_CONSUMERS;
+                if (i < nvec) {
+                    const float4 n = __ldg(reinterpret_cast<const float4*>(g.src.y_norm) + i);
+                    x[j].x += y[j].x * ir * n.x; x[j].y += y[j].y * ir * n.y; x[j].z += y[j].z * ir * n.z; x[j].w += y[j].w * ir * n.w;
+                }
+                ss += ops::sumsq4(x[j]);
+            }
+            if (PRO == PRO_FINAL) fr = inv_rms(group_sum(ss, red, GV_CONSUMERS, 1), g.src.width, g.src.eps);
+#pragma unroll
+            for (int j = 0; j < PER; ++j)
+                if (tid + j * GV_CONSUMERS < nvec) finish(tid + j * GV_CONSUMERS, x[j], before[j]);
+        } else {
+            const float ir = g.src.row_inv_rms(0, red, GV_CONSUMERS, 1);
+            if (PRO == PRO_FINAL) {
+                float ss = 0.0f;
+                for (int i = tid; i < nvec; i += GV_CONSUMERS) ss += ops::sumsq4(g.src.at(0, pos, tok, i, ir));
+                fr = inv_rms(group_sum(ss, red, GV_CONSUMERS, 1), g.src.width, g.src.eps);
+            }
+            for (int i = tid; i < nvec; i += GV_CONSUMERS) finish(i, g.src.at(0, pos, tok, i, ir), state_at(i));
         }
     }
     named_bar_sync(1, GV_CONSUMERS);
@@ -178,16 +225,15 @@ gemv_kernel(const GemvArgs<T> g)
         if ((lane & 7) == 0) part[buf][at][warp][lane >> 3] = v;
         if (at == GV_FLUSH - 1 || gi == groups - 1) {
             named_bar_sync(1, GV_CONSUMERS);
-            const int o = tid;                                       // output within this flush
-            const int first = n_begin + (gi - at) * OUT_ROWS;
-            if (o < (at + 1) * OUT_ROWS && first + o < n_end && *abort_flag == 0) {
-                const int grp = o / OUT_ROWS, row = o % OUT_ROWS;
+            const int grp = tid / OUT_ROWS, row = tid % OUT_ROWS;    // one output per thread
+            const int gg = gi - at + grp;
+            if (grp <= at && row < group_rows(gg) && *abort_flag == 0) {
                 auto sum = [&](int stage_row) {
                     const float(*p)[4] = &part[buf][grp][(stage_row >> 2) * 4];
                     const int r = stage_row & 3;
                     return ((p[0][r] + p[1][r]) + (p[2][r] + p[3][r]));
                 };
-                g.out[first + o] = GATED ? gelu_tanh(sum(row)) * sum(row + 4) : sum(row);
+                g.out[group_first(gg) + row] = GATED ? gelu_tanh(sum(row)) * sum(row + 4) : sum(row);
             }
         }
     }
@@ -196,8 +242,10 @@ gemv_kernel(const GemvArgs<T> g)
 // One query of every head over the slot's cache.  CTA = (share of the visible keys, key/value head); the CTAs of a head
 // are one cluster and add their partial outputs through distributed shared memory (the weights are not
 // normalised, so a partial is a plain sum).  Takes the projection row as the product leaves it: the RMS norms of
-// the whole q and k rows are taken here, the CTA with the newest key appends it and its value.
-constexpr int AD_THREADS = 256, AD_CHUNK = 256, AD_HB = 4;       // keys per pass, query heads per pass
+// the whole q and k rows are taken here, the CTA with the newest key appends it and its value.  A share of keys and
+// values is on its way into shared memory (cp.async) while the norms are taken; then a thread takes one
+// (key, query head) score at a time, and four value columns of one query head over the share's keys.
+constexpr int AD_THREADS = 256, AD_CHUNK = 128;       // keys in shared memory at a time
 
 template <typename T>
 struct AttnDecodeArgs {
@@ -215,8 +263,8 @@ struct AttnDecodeArgs {
 
 template <typename T>
 __host__ inline size_t attn_decode_smem_bytes(int group, int dim_pad, int vdim_pad) {
-    return sizeof(float) * ((size_t)group * dim_pad + AD_HB * AD_CHUNK + (size_t)group * vdim_pad +
-                            (size_t)AD_THREADS * AD_HB * Vec<T>::N);
+    return sizeof(float) * ((size_t)group * dim_pad + (size_t)group * AD_CHUNK + (size_t)group * vdim_pad) +
+           (size_t)AD_CHUNK * (dim_pad * sizeof(T) + 16 + vdim_pad * sizeof(T));
 }
 
 __device__ __forceinline__ float ld_cluster_f32(uint32_t addr) {
@@ -235,10 +283,12 @@ attn_decode_kernel(const AttnDecodeArgs<T> g)
     __shared__ float red[32];
     const int group = g.heads / g.kv_heads;
     float* qs = ad_smem;                                   // [group][dim_pad], normalised and scaled
-    float* ws = qs + group * g.dim_pad;                    // [AD_HB][AD_CHUNK]
-    float* os = ws + AD_HB * AD_CHUNK;                     // [group][vdim_pad]: this CTA's share of the output
-    float* sums = os + group * g.vdim_pad;                 // [key group][AD_HB][vdim_pad]
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    float* ws = qs + group * g.dim_pad;                    // [group][AD_CHUNK]
+    float* os = ws + group * AD_CHUNK;                     // [group][vdim_pad]: this CTA's share of the output
+    const int krow = g.dim_pad * (int)sizeof(T) + 16, vrow = g.vdim_pad * (int)sizeof(T);
+    uint8_t* ks = reinterpret_cast<uint8_t*>(os + group * g.vdim_pad);       // rows padded: a lane per key reads distinct banks
+    uint8_t* vs = ks + AD_CHUNK * krow;
+    const int tid = threadIdx.x;
     const int kvh = blockIdx.y, splits = gridDim.x, rank = blockIdx.x;
     const int kd = g.kv_heads * g.dim_pad, vd = g.kv_heads * g.vdim_pad, q_n = g.heads * g.dim_pad;
     pdl_wait_prior_grids();
@@ -251,116 +301,118 @@ attn_decode_kernel(const AttnDecodeArgs<T> g)
     const int per = (total + splits - 1) / splits;
     const int t_begin = min(total, rank * per), t_end = min(total, t_begin + per);
 
+    auto key_of = [&](int t) { return t < sinks ? t : lo + (t - sinks); };
+    const int kp = g.dim_pad / V::N, vp = g.vdim_pad / V::N;       // 16-byte pieces of a key and of a value row
+    const bool newest = t_begin < t_end && t_end == total && p < g.capacity;      // this CTA's share ends with key p
+    // the share's rows, all but the newest one, which is not in the cache yet
+    auto load_share = [&](int t0, int n) {
+        for (int i = tid; i < n * kp; i += AD_THREADS) {
+            const int r = i / kp, c = i - r * kp, j = key_of(t0 + r);
+            if (j < p) ops::att_cp_async16(smem_u32(ks + r * krow + c * 16), kc + (size_t)j * kd + c * V::N, 16);
+        }
+        for (int i = tid; i < n * vp; i += AD_THREADS) {
+            const int r = i / vp, c = i - r * vp, j = key_of(t0 + r);
+            if (j < p) ops::att_cp_async16(smem_u32(vs + r * vrow + c * 16), vc + (size_t)j * vd + c * V::N, 16);
+        }
+        ops::att_cp_async_commit();
+    };
+    load_share(t_begin, min(AD_CHUNK, t_end - t_begin));
+
     // norms of the whole rows
     float qr = 1.0f, kr = 1.0f;
     auto row_sq = [&](const float* v, int n) {
         float ss = 0.0f;
+#pragma unroll 4
         for (int i = tid; i < (n >> 2); i += AD_THREADS) ss += ops::sumsq4(reinterpret_cast<const float4*>(v)[i]);
         return group_sum(ss, red, AD_THREADS, 1);
     };
     if (g.q_norm != nullptr) qr = inv_rms(row_sq(g.proj, q_n), g.heads * g.dim, g.eps);
-    const bool newest = t_begin < t_end && t_end == total && p < g.capacity;      // this CTA's share ends with key p
-    if (newest) {
-        if (g.k_norm != nullptr) kr = inv_rms(row_sq(g.proj + q_n, kd), g.kv_heads * g.dim, g.eps);
-        for (int d = tid; d < g.dim_pad; d += AD_THREADS) {
-            float k = g.proj[q_n + kvh * g.dim_pad + d];
-            if (g.k_norm != nullptr) k *= kr * g.k_norm[kvh * g.dim_pad + d];
-            kc[(size_t)p * kd + d] = from_f32<T>(k);
-        }
-        for (int d = tid; d < g.vdim_pad; d += AD_THREADS)
-            vc[(size_t)p * vd + d] = from_f32<T>(g.proj[q_n + kd + kvh * g.vdim_pad + d]);
-    }
+    if (newest && g.k_norm != nullptr) kr = inv_rms(row_sq(g.proj + q_n, kd), g.kv_heads * g.dim, g.eps);
     for (int i = tid; i < group * g.dim_pad; i += AD_THREADS) {
         const int e = kvh * group * g.dim_pad + i;
         float q = g.proj[e];
         if (g.q_norm != nullptr) q *= qr * g.q_norm[e];
         qs[i] = q * g.scale;
     }
-    __syncthreads();
+    for (int i = tid; i < group * g.vdim_pad; i += AD_THREADS) os[i] = 0.0f;
 
-    const int kp = g.dim_pad / V::N, vp = g.vdim_pad / V::N;       // 16-byte pieces of a key and of a value row
-    const int kgroups = AD_THREADS / vp, piece = tid % vp, kg = tid / vp;
-    auto key_of = [&](int t) { return t < sinks ? t : lo + (t - sinks); };
-    for (int h0 = 0; h0 < group; h0 += AD_HB) {
-        const int nh = min(AD_HB, group - h0);
-        float acc[AD_HB][V::N];
+    for (int t0 = t_begin; t0 < t_end; t0 += AD_CHUNK) {
+        const int n = min(AD_CHUNK, t_end - t0);
+        if (t0 > t_begin) {
+            __syncthreads();                                       // the chunk before has been used
+            load_share(t0, n);
+        }
+        if (newest && t0 + n == t_end) {                           // the new row: into the cache and beside the others
+            for (int d = tid; d < g.dim_pad; d += AD_THREADS) {
+                float k = g.proj[q_n + kvh * g.dim_pad + d];
+                if (g.k_norm != nullptr) k *= kr * g.k_norm[kvh * g.dim_pad + d];
+                const T kt = from_f32<T>(k);
+                kc[(size_t)p * kd + d] = kt;
+                reinterpret_cast<T*>(ks + (n - 1) * krow)[d] = kt;
+            }
+            for (int d = tid; d < g.vdim_pad; d += AD_THREADS) {
+                const T vt = from_f32<T>(g.proj[q_n + kd + kvh * g.vdim_pad + d]);
+                vc[(size_t)p * vd + d] = vt;
+                reinterpret_cast<T*>(vs + (n - 1) * vrow)[d] = vt;
+            }
+        }
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        const int nr = (n + 31) & ~31;
+        for (int i = tid; i < group * nr; i += AD_THREADS) {
+            const int h = i / nr, tt = i - h * nr;                 // a warp's lanes: consecutive keys of one head
+            if (tt >= n) continue;
+            float bias = 0.0f;
+            if (g.bias_table != nullptr) bias = __ldg(g.bias_table + (size_t)(kvh * group + h) * g.bias_len + (p - key_of(t0 + tt)));
+            const uint8_t* kr_s = ks + tt * krow;
+            const float* q = qs + h * g.dim_pad;
+            float s0 = 0.0f, s1 = 0.0f;
+#pragma unroll 4
+            for (int c = 0; c < kp; ++c) {
+                float kf[V::N];
+                V::unpack(lds128(kr_s + c * 16), kf);
 #pragma unroll
-        for (int h = 0; h < AD_HB; ++h)
-#pragma unroll
-            for (int e = 0; e < V::N; ++e) acc[h][e] = 0.0f;
-        for (int t0 = t_begin; t0 < t_end; t0 += AD_CHUNK) {
-            const int n = min(AD_CHUNK, t_end - t0);
-            // scores: eight lanes per key, 32 keys per pass of the CTA
-            const int sub = lane & 7;
-            for (int k0 = 0; k0 < n; k0 += 32) {
-                const int tt = k0 + warp * 4 + (lane >> 3);
-                const bool in = tt < n;
-                const int j = key_of(t0 + (in ? tt : 0));
-                float s[AD_HB] = {0.f, 0.f, 0.f, 0.f};
-                for (int c = sub; c < kp; c += 8) {
-                    float kf[V::N];
-                    V::unpack(*reinterpret_cast<const uint4*>(kc + (size_t)j * kd + c * V::N), kf);
-#pragma unroll
-                    for (int h = 0; h < AD_HB; ++h) {
-                        if (h < nh) {
-                            const float* q = qs + (h0 + h) * g.dim_pad + c * V::N;
-#pragma unroll
-                            for (int e = 0; e < V::N; ++e) s[h] = fmaf(kf[e], q[e], s[h]);
-                        }
-                    }
-                }
-#pragma unroll
-                for (int h = 0; h < AD_HB; ++h) {
-                    s[h] += __shfl_xor_sync(0xffffffffu, s[h], 4);
-                    s[h] += __shfl_xor_sync(0xffffffffu, s[h], 2);
-                    s[h] += __shfl_xor_sync(0xffffffffu, s[h], 1);
-                }
-                if (in && sub < nh) {
-                    float sc = s[0];
-                    if (sub == 1) sc = s[1];
-                    if (sub == 2) sc = s[2];
-                    if (sub == 3) sc = s[3];
-                    if (g.bias_table != nullptr) sc += g.bias_table[(size_t)(kvh * group + h0 + sub) * g.bias_len + (p - j)];
-                    ws[sub * AD_CHUNK + tt] = sigmoid_f32(sc);
+                for (int e = 0; e < V::N; e += 4) {
+                    const float4 qv = *reinterpret_cast<const float4*>(q + c * V::N + e);
+                    s0 = fmaf(kf[e], qv.x, fmaf(kf[e + 1], qv.y, s0));
+                    s1 = fmaf(kf[e + 2], qv.z, fmaf(kf[e + 3], qv.w, s1));
                 }
             }
-            __syncthreads();
-            if (kg < kgroups) {
-#pragma unroll 2
-                for (int tt = kg; tt < n; tt += kgroups) {
-                    float vf[V::N];
-                    V::unpack(*reinterpret_cast<const uint4*>(vc + (size_t)key_of(t0 + tt) * vd + piece * V::N), vf);
-#pragma unroll
-                    for (int h = 0; h < AD_HB; ++h) {
-                        const float w = h < nh ? ws[h * AD_CHUNK + tt] : 0.0f;
-#pragma unroll
-                        for (int e = 0; e < V::N; ++e) acc[h][e] = fmaf(w, vf[e], acc[h][e]);
-                    }
-                }
+            ws[h * AD_CHUNK + tt] = sigmoid_f32(s0 + s1 + bias);
+        }
+        __syncthreads();
+        const int quads = g.vdim_pad / 4;
+        for (int i = tid; i < group * quads; i += AD_THREADS) {
+            const int h = i / quads, c = (i - h * quads) * 4;
+            float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
+            const float* w = ws + h * AD_CHUNK;
+            const uint8_t* v0 = vs + c * sizeof(T);
+#pragma unroll 8
+            for (int tt = 0; tt < n; ++tt) {
+                const float4 vf = load4(reinterpret_cast<const T*>(v0 + (size_t)tt * vrow));
+                const float wt = w[tt];
+                o0 = fmaf(wt, vf.x, o0); o1 = fmaf(wt, vf.y, o1); o2 = fmaf(wt, vf.z, o2); o3 = fmaf(wt, vf.w, o3);
             }
-            __syncthreads();                                        // ws is written again
+            float4* o = reinterpret_cast<float4*>(os + h * g.vdim_pad + c);      // this thread's own columns
+            const float4 before = *o;
+            *o = make_float4(before.x + o0, before.y + o1, before.z + o2, before.w + o3);
         }
-        if (kg < kgroups) {
-#pragma unroll
-            for (int h = 0; h < AD_HB; ++h)
-#pragma unroll
-                for (int e = 0; e < V::N; ++e) sums[(kg * AD_HB + h) * g.vdim_pad + piece * V::N + e] = acc[h][e];
-        }
-        __syncthreads();
-        for (int i = tid; i < nh * g.vdim_pad; i += AD_THREADS) {
-            float o = 0.0f;
-            for (int k = 0; k < kgroups; ++k) o += sums[k * AD_HB * g.vdim_pad + i];
-            os[h0 * g.vdim_pad + i] = o;
-        }
-        __syncthreads();
     }
+    __syncthreads();
     cluster_sync_all();
     for (int i = rank * AD_THREADS + tid; i < group * g.vdim_pad; i += splits * AD_THREADS) {
+        const int e = kvh * group * g.vdim_pad + i;
+        const float gate = g.gated ? g.proj[q_n + kd + vd + e] : 0.0f;
         float o = 0.0f;
         const uint32_t at = smem_u32(os + i);
-        for (int s = 0; s < splits; ++s) o += ld_cluster_f32(mapa_shared(at, s));
-        const int e = kvh * group * g.vdim_pad + i;
-        if (g.gated) o *= sigmoid_f32(g.proj[q_n + kd + vd + e]);
+        for (int s0 = 0; s0 < splits; s0 += 8) {                    // eight ranks' loads in flight, added in rank order
+            float part[8];
+#pragma unroll
+            for (int s = 0; s < 8; ++s) part[s] = s0 + s < splits ? ld_cluster_f32(mapa_shared(at, s0 + s)) : 0.0f;
+#pragma unroll
+            for (int s = 0; s < 8; ++s) o += part[s];
+        }
+        if (g.gated) o *= sigmoid_f32(gate);
         g.out[e] = o;
     }
     cluster_sync_all();                                             // nobody leaves while its shared memory may be read

@@ -66,6 +66,14 @@ __device__ __forceinline__ void store4<bf16>(bf16* dst, const float4 v) {
     *reinterpret_cast<uint2*>(dst) = o;
 }
 
+// four consecutive elements as floats
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const bf16* p) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16),
+                       __uint_as_float(v.y & 0xffff0000u));
+}
+
 // x + (before - x) * mix
 __device__ __forceinline__ float4 shift4(const float4 x, const float4 before, const float4 mix) {
     return make_float4(fmaf(before.x - x.x, mix.x, x.x), fmaf(before.y - x.y, mix.y, x.y), fmaf(before.z - x.z, mix.z, x.z),
