@@ -72,9 +72,10 @@ def attention_mixer(x, w, pre, m, eps):
     k = rms_norm(h @ w[pre + "mix.k"].T, w[pre + "mix.k.norm"], eps)
     v = h @ w[pre + "mix.v"].T
     n = x.shape[0]
+    mask = m.get("mask") or {"size": n, "keep_first": 0}
     o = sigmoid_attention(q.reshape(n, m["heads"], m["dim"]), k.reshape(n, m["kv_heads"], m["dim"]),
                           v.reshape(n, m["kv_heads"], m["vdim"]), m["scale"], w[pre + "mix.r1"], w[pre + "mix.r2"],
-                          w[pre + "mix.pb"], visible(n, m["mask"]["size"], m["mask"]["keep_first"]))
+                          w[pre + "mix.pb"], visible(n, mask["size"], mask["keep_first"]))
     o = o.reshape(n, -1) * sigmoid(h @ w[pre + "mix.g"].T)
     return o @ w[pre + "mix.o"].T
 

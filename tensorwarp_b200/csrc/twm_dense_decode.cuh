@@ -245,7 +245,7 @@ gemv_kernel(const GemvArgs<T> g)
 // the whole q and k rows are taken here, the CTA with the newest key appends it and its value.  A share of keys and
 // values is on its way into shared memory (cp.async) while the norms are taken; then a thread takes one
 // (key, query head) score at a time, and four value columns of one query head over the share's keys.
-constexpr int AD_THREADS = 256, AD_CHUNK = 128;       // keys in shared memory at a time
+constexpr int AD_THREADS = 256, AD_MAX_CHUNK = 128;   // keys in shared memory at a time, at most
 
 template <typename T>
 struct AttnDecodeArgs {
@@ -258,13 +258,14 @@ struct AttnDecodeArgs {
     const float* bias_table;
     const int* meta;
     int heads, kv_heads, dim, dim_pad, vdim_pad, window, keep_first, capacity, bias_len, gated;
+    int chunk;                  // keys in shared memory at a time, a multiple of 4
     float scale, eps;
 };
 
 template <typename T>
-__host__ inline size_t attn_decode_smem_bytes(int group, int dim_pad, int vdim_pad) {
-    return sizeof(float) * ((size_t)group * dim_pad + (size_t)group * AD_CHUNK + (size_t)group * vdim_pad) +
-           (size_t)AD_CHUNK * (dim_pad * sizeof(T) + 16 + vdim_pad * sizeof(T));
+__host__ inline size_t attn_decode_smem_bytes(int group, int dim_pad, int vdim_pad, int chunk) {
+    return sizeof(float) * ((size_t)group * dim_pad + (size_t)group * chunk + (size_t)group * vdim_pad) +
+           (size_t)chunk * (dim_pad * sizeof(T) + 16 + vdim_pad * sizeof(T));
 }
 
 __device__ __forceinline__ float ld_cluster_f32(uint32_t addr) {
@@ -283,11 +284,11 @@ attn_decode_kernel(const AttnDecodeArgs<T> g)
     __shared__ float red[32];
     const int group = g.heads / g.kv_heads;
     float* qs = ad_smem;                                   // [group][dim_pad], normalised and scaled
-    float* ws = qs + group * g.dim_pad;                    // [group][AD_CHUNK]
-    float* os = ws + group * AD_CHUNK;                     // [group][vdim_pad]: this CTA's share of the output
+    float* ws = qs + group * g.dim_pad;                    // [group][chunk]
+    float* os = ws + group * g.chunk;                     // [group][vdim_pad]: this CTA's share of the output
     const int krow = g.dim_pad * (int)sizeof(T) + 16, vrow = g.vdim_pad * (int)sizeof(T);
     uint8_t* ks = reinterpret_cast<uint8_t*>(os + group * g.vdim_pad);       // rows padded: a lane per key reads distinct banks
-    uint8_t* vs = ks + AD_CHUNK * krow;
+    uint8_t* vs = ks + g.chunk * krow;
     const int tid = threadIdx.x;
     const int kvh = blockIdx.y, splits = gridDim.x, rank = blockIdx.x;
     const int kd = g.kv_heads * g.dim_pad, vd = g.kv_heads * g.vdim_pad, q_n = g.heads * g.dim_pad;
@@ -316,7 +317,7 @@ attn_decode_kernel(const AttnDecodeArgs<T> g)
         }
         ops::att_cp_async_commit();
     };
-    load_share(t_begin, min(AD_CHUNK, t_end - t_begin));
+    load_share(t_begin, min(g.chunk, t_end - t_begin));
 
     // norms of the whole rows
     float qr = 1.0f, kr = 1.0f;
@@ -336,8 +337,8 @@ attn_decode_kernel(const AttnDecodeArgs<T> g)
     }
     for (int i = tid; i < group * g.vdim_pad; i += AD_THREADS) os[i] = 0.0f;
 
-    for (int t0 = t_begin; t0 < t_end; t0 += AD_CHUNK) {
-        const int n = min(AD_CHUNK, t_end - t0);
+    for (int t0 = t_begin; t0 < t_end; t0 += g.chunk) {
+        const int n = min(g.chunk, t_end - t0);
         if (t0 > t_begin) {
             __syncthreads();                                       // the chunk before has been used
             load_share(t0, n);
@@ -378,14 +379,14 @@ attn_decode_kernel(const AttnDecodeArgs<T> g)
                     s1 = fmaf(kf[e + 2], qv.z, fmaf(kf[e + 3], qv.w, s1));
                 }
             }
-            ws[h * AD_CHUNK + tt] = sigmoid_f32(s0 + s1 + bias);
+            ws[h * g.chunk + tt] = sigmoid_f32(s0 + s1 + bias);
         }
         __syncthreads();
         const int quads = g.vdim_pad / 4;
         for (int i = tid; i < group * quads; i += AD_THREADS) {
             const int h = i / quads, c = (i - h * quads) * 4;
             float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
-            const float* w = ws + h * AD_CHUNK;
+            const float* w = ws + h * g.chunk;
             const uint8_t* v0 = vs + c * sizeof(T);
 #pragma unroll 8
             for (int tt = 0; tt < n; ++tt) {
