@@ -54,6 +54,7 @@ typedef struct twm_dense_model {
     int width, width_pad, vocab, n_layers;
     int bias_len;                /* entries per head of the bias tables; > every distance that can occur */
     int capacity;                /* tokens per slot */
+    int slots;
     float eps;
     const void* embed;           /* [vocab][width_pad] */
     const void* pos_embed;       /* [>= capacity][width_pad] or NULL */
@@ -113,7 +114,7 @@ twm_status twm_dense_gemm(int dtype, const void* a, int lda, const void* w, int 
                           int epilogue, int kernel, int flags, void* stream);
 /* Attention of `rows` queries at positions meta[0] ... over the slot's cache (already holding their keys and values);
  * proj rows as the fused projection leaves them (q normalised in place, gate = last block).  kernel: 0 = by size,
- * 1 = one query per CTA, 2 = tensor-core tiles. */
+ * 1 = one query per CTA, 2 = warp-level tensor-core tiles, 3 = tcgen05 tiles. */
 twm_status twm_dense_attention(const twm_dense_model* m, int layer, const twm_dense_buffers* b, int rows, int first_pos,
                                int kernel, int flags, void* stream);
 

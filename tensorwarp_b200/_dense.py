@@ -23,7 +23,7 @@ class Layer(C.Structure):
 class Model(C.Structure):
     """``twm_dense_model``."""
     _fields_ = [("dtype", C.c_int), ("width", C.c_int), ("width_pad", C.c_int), ("vocab", C.c_int), ("n_layers", C.c_int),
-                ("bias_len", C.c_int), ("capacity", C.c_int), ("eps", C.c_float), ("embed", C.c_void_p), ("pos_embed", C.c_void_p),
+                ("bias_len", C.c_int), ("capacity", C.c_int), ("slots", C.c_int), ("eps", C.c_float), ("embed", C.c_void_p), ("pos_embed", C.c_void_p),
                 ("head", C.c_void_p), ("final_norm", C.c_void_p), ("layers", C.POINTER(Layer))]
 
 

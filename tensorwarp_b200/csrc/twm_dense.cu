@@ -7,6 +7,7 @@
 #include <unordered_map>
 
 #include "twm_dense_attn.cuh"
+#include "twm_dense_attn_tc.cuh"
 #include "twm_dense_common.cuh"
 #include "twm_dense_decode.cuh"
 #include "twm_dense_rows.cuh"
@@ -119,7 +120,7 @@ twm_status check_model(const twm_dense_model* m, const twm_dense_buffers* b)
 {
     if (!m || !b || !m->layers) return invalid("null model or buffers");
     if (m->dtype != TWM_DENSE_F32 && m->dtype != TWM_DENSE_BF16) return invalid("dtype");
-    if (m->width < 1 || m->width_pad < m->width || m->width_pad % 16 || m->vocab < 1 || m->n_layers < 0 || m->capacity < 1)
+    if (m->width < 1 || m->width_pad < m->width || m->width_pad % 16 || m->vocab < 1 || m->n_layers < 0 || m->capacity < 1 || m->slots < 1)
         return invalid("model sizes");
     if (!m->embed || !m->head || !m->final_norm) return invalid("embedding, head or final norm missing");
     if (!b->meta || !b->tokens || !b->want || !b->x0 || !b->x1 || !b->y || !b->a || !b->proj || !b->att || !b->act || !b->vec ||
@@ -156,40 +157,53 @@ EncodeTiledFn encode_tiled()
     return fn;
 }
 
-// bf16 [rows][cols] with row stride ld, boxes of 64 columns x box_rows, 128-byte swizzle, zeros outside.  A map is a
-// pure description of memory, so maps are kept by what they describe.
+// A bf16 tensor of up to four dimensions (innermost first; strides in elements), boxes of 64 x box[1] x ..., 128-byte
+// swizzle, zeros outside.  A map is a pure description of memory, so maps are kept by what they describe.
 struct MapKey {
-    const void* ptr; long rows, cols, ld; int box;
-    bool operator==(const MapKey& o) const { return ptr == o.ptr && rows == o.rows && cols == o.cols && ld == o.ld && box == o.box; }
+    const void* ptr;
+    int rank;
+    long dim[4], stride[4], box[4];
+    bool operator==(const MapKey& o) const {
+        return ptr == o.ptr && rank == o.rank && std::equal(dim, dim + 4, o.dim) && std::equal(stride, stride + 4, o.stride) &&
+               std::equal(box, box + 4, o.box);
+    }
 };
 struct MapHash {
     size_t operator()(const MapKey& k) const {
-        size_t h = (size_t)k.ptr;
-        for (size_t v : {(size_t)k.rows, (size_t)k.cols, (size_t)k.ld, (size_t)k.box}) h = h * 1000003u ^ v;
+        size_t h = (size_t)k.ptr + (size_t)k.rank;
+        for (int i = 0; i < 4; ++i)
+            for (long v : {k.dim[i], k.stride[i], k.box[i]}) h = h * 1000003u ^ (size_t)v;
         return h;
     }
 };
-bool rows_map(CUtensorMap* map, const void* ptr, long rows, long cols, long ld, int box_rows)
+bool swizzled_map(CUtensorMap* map, const MapKey& key)
 {
     static std::unordered_map<MapKey, CUtensorMap, MapHash> cache;
     static std::mutex mutex;
-    const MapKey key{ptr, rows, cols, ld, box_rows};
     std::lock_guard<std::mutex> lock(mutex);
     auto it = cache.find(key);
     if (it != cache.end()) { *map = it->second; return true; }
     EncodeTiledFn enc = encode_tiled();
     if (!enc) return false;
-    const cuuint64_t gdim[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
-    const cuuint64_t gstride[1] = {(cuuint64_t)ld * 2};
-    const cuuint32_t box[2] = {(cuuint32_t)TC_BK, (cuuint32_t)box_rows};
-    const cuuint32_t estride[2] = {1, 1};
-    if (enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(ptr), gdim, gstride, box, estride,
+    cuuint64_t gdim[4], gstride[3];
+    cuuint32_t box[4], estride[4] = {1, 1, 1, 1};
+    for (int i = 0; i < key.rank; ++i) {
+        gdim[i] = (cuuint64_t)key.dim[i];
+        box[i] = (cuuint32_t)key.box[i];
+        if (i > 0) gstride[i - 1] = (cuuint64_t)key.stride[i] * 2;
+    }
+    if (enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, (cuuint32_t)key.rank, const_cast<void*>(key.ptr), gdim, gstride, box, estride,
             CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
         return false;
-    if (cache.size() > 4096) cache.clear();
+    if (cache.size() > 8192) cache.clear();
     cache.emplace(key, *map);
     return true;
+}
+// [rows][cols] with row stride ld, boxes of 64 columns x box_rows
+bool rows_map(CUtensorMap* map, const void* ptr, long rows, long cols, long ld, int box_rows)
+{
+    return swizzled_map(map, MapKey{ptr, 2, {cols, rows, 0, 0}, {1, ld, 0, 0}, {TC_BK, box_rows, 0, 0}});
 }
 
 // ------------------------------------------------------------- operations --
@@ -313,11 +327,37 @@ twm_status attention_tiles(const AttnArgs<bf16>& g, int flags, void* stream)
 }
 twm_status attention_tiles(const AttnArgs<float>&, int, void*) { return invalid("the tensor-core attention takes bfloat16"); }
 
+// The tcgen05 attention: heads of up to 128 columns.
+bool attention_tc_fits(const AttnArgs<bf16>& g)
+{
+    return g.dim_pad <= 128 && g.vdim_pad <= 128 && ((uintptr_t)g.proj & 15) == 0 && ((uintptr_t)g.k_cache & 15) == 0 &&
+           ((uintptr_t)g.v_cache & 15) == 0;
+}
+bool attention_tc_fits(const AttnArgs<float>&) { return false; }
+twm_status attention_tc(const AttnArgs<bf16>& g, int end, int slots, int flags, void* stream)
+{
+    AttnTcArgs t;
+    t.a = g;
+    auto cache_map = [&](CUtensorMap* map, const bf16* base, int pad) {
+        const long row = (long)g.kv_heads * pad;
+        return swizzled_map(map, MapKey{base, 4, {pad, g.kv_heads, end, slots}, {1, pad, row, row * g.capacity}, {64, 1, AT_K, 1}});
+    };
+    if (!swizzled_map(&t.q_map, MapKey{g.proj, 3, {g.dim_pad, g.heads, g.rows, 0}, {1, g.dim_pad, g.ld, 0}, {64, 1, AT_Q, 0}}) ||
+        !cache_map(&t.k_map, g.k_cache, g.dim_pad) || !cache_map(&t.v_map, g.v_cache, g.vdim_pad))
+        return invalid("cuTensorMapEncodeTiled refused a map of the tcgen05 attention");
+    return launch("attn_tc", attn_tc_kernel, dim3((g.rows + AT_Q - 1) / AT_Q, g.heads), AT_THREADS, sizeof(AttnTcSmem) + 1024, flags,
+                  stream, 0, t);
+}
+twm_status attention_tc(const AttnArgs<float>&, int, int, int, void*) { return invalid("the tcgen05 attention takes bfloat16"); }
+
 template <typename T>
 twm_status attention(const twm_dense_model* m, const twm_dense_layer& l, const twm_dense_buffers* b, int rows, int first_pos,
                      int kernel, int flags, void* stream)
 {
     const AttnArgs<T> g = attn_args<T>(m, l, b, rows);
+    if (kernel < 0 || kernel > 3) return invalid("kernel");
+    if (kernel == 3 && !attention_tc_fits(g)) return invalid("the tcgen05 attention takes bfloat16 heads of up to 128 columns");
+    if (kernel == 3 || (kernel == 0 && attention_tc_fits(g))) return attention_tc(g, first_pos + rows, m->slots, flags, stream);
     if (kernel == 2 && !attention_tiles_fit(g)) return invalid("the tensor-core attention takes bfloat16 heads that fit shared memory");
     if (kernel == 2 || (kernel == 0 && attention_tiles_fit(g))) return attention_tiles(g, flags, stream);
     const int vblock = AS_VPT * AS_THREADS;

@@ -167,7 +167,7 @@ class DenseModel:
         d = _dense.Model()
         d.dtype = _dense.TWM_DENSE_F32 if self.dtype == torch.float32 else _dense.TWM_DENSE_BF16
         d.width, d.width_pad, d.vocab, d.n_layers = self.spec.width, self.width_pad, self.spec.vocab, n
-        d.bias_len, d.capacity, d.eps = self.spec.max_positions, state.capacity, self.spec.eps
+        d.bias_len, d.capacity, d.slots, d.eps = self.spec.max_positions, state.capacity, state.slots, self.spec.eps
         d.embed, d.head, d.final_norm = self.embed.data_ptr(), self.head.data_ptr(), self.final_norm.data_ptr()
         d.pos_embed = self.pos.data_ptr() if self.pos is not None else None
         d.layers = array

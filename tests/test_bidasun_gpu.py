@@ -191,13 +191,15 @@ def _lone_layer(dtype, heads, kv_heads, dim, vdim, window, keep):
     return DenseEngine(dense.DenseModel(spec, bidasun.model_tensors(spec, lambda n, s: t[n]), dtype), portion=512), cases.as_float64(t)
 
 
-@pytest.mark.parametrize("dtype,kernel", [(torch.float32, 1), (torch.bfloat16, 1), (torch.bfloat16, 2)])
+@pytest.mark.parametrize("dtype,kernel", [(torch.float32, 1), (torch.bfloat16, 1), (torch.bfloat16, 2), (torch.bfloat16, 3)])
 @pytest.mark.parametrize("heads,kv_heads,dim,vdim,window,keep", [(4, 2, 64, 64, 100, 3), (3, 1, 128, 128, 64, 64), (2, 2, 32, 144, 65, 130),
                                                                  (8, 2, 80, 48, 1, 1), (2, 1, 64, 128, 300, 0), (2, 2, 128, 64, 600, 5)])
 @pytest.mark.parametrize("first,rows", [(0, 330), (70, 5), (191, 130), (320, 64)])
 def test_attention_one_key_stands_out(dtype, kernel, heads, kv_heads, dim, vdim, window, keep, first, rows):
     """All scores far below zero but for one key, whose value is its own: a query's output shows whether it sees
     that key, and with what weight, for keys inside and outside the window, among the kept ones and at tile borders."""
+    if kernel == 3 and max(dim, vdim) > 128:
+        pytest.skip("the tcgen05 attention takes heads of up to 128 columns")
     eng, w = _lone_layer(dtype, heads, kv_heads, dim, vdim, window, keep)
     n = first + rows
     rng = np.random.default_rng(n + window)
