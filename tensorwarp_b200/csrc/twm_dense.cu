@@ -370,7 +370,6 @@ twm_status prefill(const twm_dense_model* m, const twm_dense_buffers* b, int row
                    int flags, void* stream)
 {
     const int wp = m->width_pad;
-    const int rpc = rows >= 2048 ? 8 : rows >= 512 ? 4 : 2;
     float *x = b->x0, *x_next = b->x1;
     const float* y = nullptr;                            // the sublayer output that has yet to join the residual stream
     const float* y_norm = nullptr;
@@ -385,9 +384,14 @@ twm_status prefill(const twm_dense_model* m, const twm_dense_buffers* b, int row
     };
     // the residual stream brought up to date, with the next sublayer's input beside it
     auto join = [&](const float* shift, const float* state, bool want_a) {
-        const twm_status st = launch("residual_rows", residual_rows_kernel<T>, dim3((rows + rpc - 1) / rpc), ROW_THREADS,
-                                     sizeof(float) * (size_t)wp, flags, stream, 0, source(), x_next, want_a ? (T*)b->a : (T*)nullptr,
-                                     shift, state, b->meta, rows, rpc);
+        // rows per CTA: enough CTAs to fill the machine several times; a shifted run computes one row more than it has
+        const int rpc = shift ? (rows >= 4096 ? 8 : rows >= 1024 ? 4 : rows >= 256 ? 2 : 1) : 1;
+        const int per = (wp / 4 + ROW_THREADS - 1) / ROW_THREADS;
+        auto kernel = per <= 1 ? residual_rows_kernel<T, 1> : per <= 2 ? residual_rows_kernel<T, 2> :
+                      per <= 4 ? residual_rows_kernel<T, 4> : per <= 8 ? residual_rows_kernel<T, 8> : residual_rows_kernel<T, 0>;
+        const twm_status st = launch("residual_rows", kernel, dim3((rows + rpc - 1) / rpc), ROW_THREADS,
+                                     per <= 8 ? 0 : sizeof(float) * (size_t)wp, flags, stream, 0, source(), x_next,
+                                     want_a ? (T*)b->a : (T*)nullptr, shift, state, b->meta, rows, rpc);
         std::swap(x, x_next);
         embedded = true;
         y = nullptr;

@@ -81,47 +81,93 @@ __device__ __forceinline__ float4 shift4(const float4 x, const float4 before, co
 }
 
 // x_out = residual row; a = T(x_out), or T(token shift of x_out).  A CTA walks `rows_per_cta` consecutive rows and
-// keeps the row before in shared memory; its first row's predecessor is computed again (or comes from the state).
-template <typename T>
+// keeps the row before; its first row's predecessor is computed again (or comes from the state).  PER > 0: a
+// thread's share of a row is PER vectors, held in registers, every load issued before the first use; PER = 0: rows
+// of any length, in shared memory.
+template <typename T, int PER>
 __global__ void __launch_bounds__(ROW_THREADS)
 residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __restrict__ a, const float* __restrict__ shift,
                      const float* __restrict__ shift_state, const int* __restrict__ meta, int rows, int rows_per_cta)
 {
     pdl_launch_dependents();
-    extern __shared__ __align__(16) float row_smem[];       // [wp]: the residual row before
+    extern __shared__ __align__(16) float row_smem[];       // PER = 0: [wp], the residual row before
     __shared__ float red[32];
     pdl_wait_prior_grids();
     const int wp = src.wp, nvec = wp >> 2;
     const int r0 = blockIdx.x * rows_per_cta, r1 = min(rows, r0 + rows_per_cta);
     const int pos0 = meta[0];
-    if (shift != nullptr) {
-        if (r0 == 0) {
-            const float* st = shift_state + ((size_t)meta[1] * 2 + ((pos0 - 1) & 1)) * wp;
-            for (int i = threadIdx.x; i < nvec; i += ROW_THREADS)
-                reinterpret_cast<float4*>(row_smem)[i] =
-                    pos0 > 0 ? reinterpret_cast<const float4*>(st)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
-        } else {
-            const int r = r0 - 1;
+    const float* st = shift != nullptr && r0 == 0 && pos0 > 0
+                          ? shift_state + ((size_t)meta[1] * 2 + ((pos0 - 1) & 1)) * wp : nullptr;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    if constexpr (PER > 0) {
+        float4 before[PER];
+#pragma unroll
+        for (int j = 0; j < PER; ++j) {
+            const int i = threadIdx.x + j * ROW_THREADS;
+            before[j] = st != nullptr && i < nvec ? reinterpret_cast<const float4*>(st)[i] : zero;
+        }
+        for (int r = (shift != nullptr && r0 > 0) ? r0 - 1 : r0; r < r1; ++r) {
+            float4 x[PER], y[PER];
+            const int tok = src.tokens != nullptr ? src.tokens[r] : 0;
+            ResidualSource<T> plain = src;                  // the row without what joins it
+            plain.y = nullptr;
+#pragma unroll
+            for (int j = 0; j < PER; ++j) {
+                const int i = threadIdx.x + j * ROW_THREADS;
+                y[j] = src.y != nullptr && i < nvec ? reinterpret_cast<const float4*>(src.y + (size_t)r * wp)[i] : zero;
+                x[j] = i < nvec ? plain.at(r, pos0 + r, tok, i, 1.0f) : zero;
+            }
+            float ir = 1.0f;
+            if (src.y != nullptr && src.y_norm != nullptr) {
+                float ss = 0.0f;
+#pragma unroll
+                for (int j = 0; j < PER; ++j) ss += ops::sumsq4(y[j]);
+                ir = inv_rms(group_sum(ss, red, ROW_THREADS, 1), src.width, src.eps);
+            }
+#pragma unroll
+            for (int j = 0; j < PER; ++j) {
+                const int i = threadIdx.x + j * ROW_THREADS;
+                if (i >= nvec) continue;
+                float4 n = make_float4(1.f, 1.f, 1.f, 1.f);
+                if (src.y_norm != nullptr) n = __ldg(reinterpret_cast<const float4*>(src.y_norm) + i);
+                x[j].x += y[j].x * ir * n.x; x[j].y += y[j].y * ir * n.y; x[j].z += y[j].z * ir * n.z; x[j].w += y[j].w * ir * n.w;
+                if (r >= r0) {
+                    reinterpret_cast<float4*>(x_out + (size_t)r * wp)[i] = x[j];
+                    float4 h = x[j];
+                    if (shift != nullptr) h = shift4(x[j], before[j], __ldg(reinterpret_cast<const float4*>(shift) + i));
+                    if (a != nullptr) store4<T>(a + (size_t)r * wp + i * 4, h);
+                }
+                before[j] = x[j];
+            }
+        }
+    } else {
+        if (shift != nullptr) {
+            if (r0 == 0) {
+                for (int i = threadIdx.x; i < nvec; i += ROW_THREADS)
+                    reinterpret_cast<float4*>(row_smem)[i] = st != nullptr ? reinterpret_cast<const float4*>(st)[i] : zero;
+            } else {
+                const int r = r0 - 1;
+                const int tok = src.tokens != nullptr ? src.tokens[r] : 0;
+                const float ir = src.row_inv_rms(r, red, ROW_THREADS, 1);
+                for (int i = threadIdx.x; i < nvec; i += ROW_THREADS)
+                    reinterpret_cast<float4*>(row_smem)[i] = src.at(r, pos0 + r, tok, i, ir);
+            }
+        }
+        for (int r = r0; r < r1; ++r) {
             const int tok = src.tokens != nullptr ? src.tokens[r] : 0;
             const float ir = src.row_inv_rms(r, red, ROW_THREADS, 1);
-            for (int i = threadIdx.x; i < nvec; i += ROW_THREADS)
-                reinterpret_cast<float4*>(row_smem)[i] = src.at(r, pos0 + r, tok, i, ir);
-        }
-    }
-    for (int r = r0; r < r1; ++r) {
-        const int tok = src.tokens != nullptr ? src.tokens[r] : 0;
-        const float ir = src.row_inv_rms(r, red, ROW_THREADS, 1);
-        // every thread reads and replaces its own elements of row_smem: no barrier needed between rows
-        for (int i = threadIdx.x; i < nvec; i += ROW_THREADS) {
-            const float4 x = src.at(r, pos0 + r, tok, i, ir);
-            reinterpret_cast<float4*>(x_out + (size_t)r * wp)[i] = x;
-            float4 h = x;
-            if (shift != nullptr) {
-                float4* before = reinterpret_cast<float4*>(row_smem) + i;
-                h = shift4(x, *before, __ldg(reinterpret_cast<const float4*>(shift) + i));
-                *before = x;
+            // every thread reads and replaces its own elements of row_smem: no barrier needed between rows
+            for (int i = threadIdx.x; i < nvec; i += ROW_THREADS) {
+                const float4 x = src.at(r, pos0 + r, tok, i, ir);
+                reinterpret_cast<float4*>(x_out + (size_t)r * wp)[i] = x;
+                float4 h = x;
+                if (shift != nullptr) {
+                    float4* before = reinterpret_cast<float4*>(row_smem) + i;
+                    h = shift4(x, *before, __ldg(reinterpret_cast<const float4*>(shift) + i));
+                    *before = x;
+                }
+                if (a != nullptr) store4<T>(a + (size_t)r * wp + i * 4, h);
             }
-            if (a != nullptr) store4<T>(a + (size_t)r * wp + i * 4, h);
         }
     }
 }
@@ -169,39 +215,73 @@ qk_norm_append_kernel(T* __restrict__ proj, int ld, const float* __restrict__ q_
     using V = Vec<T>;
     const int r = blockIdx.x, p = meta[0] + r, slot = meta[1];
     T* row = proj + (size_t)r * ld;
-    auto sum_sq = [&](const T* base, int n) {
-        float ss = 0.0f;
-        for (int i = threadIdx.x; i < n / V::N; i += ROW_THREADS) {
-            float f[V::N];
-            V::unpack(reinterpret_cast<const uint4*>(base)[i], f);
+    const bool cached = p < capacity;
+    T* k_dst = k_cache + ((size_t)slot * capacity + p) * k_n;
+    T* v_dst = v_cache + ((size_t)slot * capacity + p) * v_n;
+    auto sum_sq = [&](const uint4& raw) {
+        float f[V::N], ss = 0.0f;
+        V::unpack(raw, f);
 #pragma unroll
-            for (int j = 0; j < V::N; ++j) ss = fmaf(f[j], f[j], ss);
-        }
+        for (int j = 0; j < V::N; ++j) ss = fmaf(f[j], f[j], ss);
         return ss;
     };
-    auto scale_row = [&](const T* base, T* dst, int n, float ir, const float* g) {
-        for (int i = threadIdx.x; i < n / V::N; i += ROW_THREADS) {
-            uint4 raw = reinterpret_cast<const uint4*>(base)[i];
-            if (g != nullptr) {
-                float f[V::N];
-                V::unpack(raw, f);
+    auto scaled = [&](const uint4& raw, float ir, const float* g, int i) {
+        float f[V::N];
+        V::unpack(raw, f);
 #pragma unroll
-                for (int j = 0; j < V::N; ++j) f[j] *= ir * __ldg(g + i * V::N + j);
-                raw = V::pack(f);
-            }
-            reinterpret_cast<uint4*>(dst)[i] = raw;
+        for (int j = 0; j < V::N; j += 4) {
+            const float4 n = __ldg(reinterpret_cast<const float4*>(g + i * V::N + j));
+            f[j] *= ir * n.x; f[j + 1] *= ir * n.y; f[j + 2] *= ir * n.z; f[j + 3] *= ir * n.w;
         }
+        return V::pack(f);
     };
-    if (q_norm != nullptr) {
-        const float ir = inv_rms(group_sum(sum_sq(row, q_n), red, ROW_THREADS, 1), q_true, eps);
-        scale_row(row, row, q_n, ir, q_norm);
+    const uint4* q_row = reinterpret_cast<const uint4*>(row);
+    const uint4* k_row = reinterpret_cast<const uint4*>(row + q_n);
+    const uint4* v_row = reinterpret_cast<const uint4*>(row + q_n + k_n);
+    // a thread's first pieces stay in registers between the sum and the scaling; longer rows read the rest again
+    constexpr int QP = 4, KP = 2;
+    uint4 q[QP], k[KP];
+    float qs = 0.0f, ks = 0.0f;
+#pragma unroll
+    for (int j = 0; j < QP; ++j) {
+        const int i = threadIdx.x + j * ROW_THREADS;
+        q[j] = q_norm != nullptr && i < q_n / V::N ? q_row[i] : make_uint4(0, 0, 0, 0);
     }
-    if (p < capacity) {
-        const size_t at = (size_t)slot * capacity + p;
-        float ir = 1.0f;
-        if (k_norm != nullptr) ir = inv_rms(group_sum(sum_sq(row + q_n, k_n), red, ROW_THREADS, 1), k_true, eps);
-        scale_row(row + q_n, k_cache + at * k_n, k_n, ir, k_norm);
-        scale_row(row + q_n + k_n, v_cache + at * v_n, v_n, 1.0f, nullptr);
+#pragma unroll
+    for (int j = 0; j < KP; ++j) {
+        const int i = threadIdx.x + j * ROW_THREADS;
+        k[j] = i < k_n / V::N ? k_row[i] : make_uint4(0, 0, 0, 0);
+    }
+    if (cached)
+        for (int i = threadIdx.x; i < v_n / V::N; i += ROW_THREADS) reinterpret_cast<uint4*>(v_dst)[i] = v_row[i];
+    if (q_norm != nullptr) {
+#pragma unroll
+        for (int j = 0; j < QP; ++j) qs += sum_sq(q[j]);
+        for (int i = threadIdx.x + QP * ROW_THREADS; i < q_n / V::N; i += ROW_THREADS) qs += sum_sq(q_row[i]);
+        const float ir = inv_rms(group_sum(qs, red, ROW_THREADS, 1), q_true, eps);
+#pragma unroll
+        for (int j = 0; j < QP; ++j) {
+            const int i = threadIdx.x + j * ROW_THREADS;
+            if (i < q_n / V::N) reinterpret_cast<uint4*>(row)[i] = scaled(q[j], ir, q_norm, i);
+        }
+        for (int i = threadIdx.x + QP * ROW_THREADS; i < q_n / V::N; i += ROW_THREADS)
+            reinterpret_cast<uint4*>(row)[i] = scaled(q_row[i], ir, q_norm, i);
+    }
+    float kir = 1.0f;
+    if (k_norm != nullptr) {
+#pragma unroll
+        for (int j = 0; j < KP; ++j) ks += sum_sq(k[j]);
+        for (int i = threadIdx.x + KP * ROW_THREADS; i < k_n / V::N; i += ROW_THREADS) ks += sum_sq(k_row[i]);
+        kir = inv_rms(group_sum(ks, red, ROW_THREADS, 1), k_true, eps);
+    }
+    if (cached) {
+#pragma unroll
+        for (int j = 0; j < KP; ++j) {
+            const int i = threadIdx.x + j * ROW_THREADS;
+            if (i < k_n / V::N) reinterpret_cast<uint4*>(k_dst)[i] = k_norm != nullptr ? scaled(k[j], kir, k_norm, i) : k[j];
+        }
+        for (int i = threadIdx.x + KP * ROW_THREADS; i < k_n / V::N; i += ROW_THREADS)
+            reinterpret_cast<uint4*>(k_dst)[i] = k_norm != nullptr ? scaled(k_row[i], kir, k_norm, i) : k_row[i];
     }
     if (shift_state != nullptr && r == gridDim.x - 1) {
         float* st = shift_state + ((size_t)slot * 2 + (p & 1)) * wp;
