@@ -109,7 +109,7 @@ twm_status twm_dense_argmax_advance(const twm_dense_buffers* b, int vocab, int r
 enum { TWM_EPI_STORE = 0, TWM_EPI_STORE_F32 = 1, TWM_EPI_GELU_GLU = 2 };
 /* C[M][N] = A[M][K] . W[N][K]^T with FP32 accumulation.  GELU_GLU: W is [N | N][K] (gate, up), C = gelu_tanh(gate) * up.
  * C has the input type except for STORE_F32.  kernel: 0 = chosen by size, 1 = plain tiles, 2 = tcgen05, 64/128/256 = tcgen05 with
- * tiles of that many columns. */
+ * tiles of that many columns, 512 = tiles of 256 x 256 on a pair of SMs. */
 twm_status twm_dense_gemm(int dtype, const void* a, int lda, const void* w, int ldw, void* c, int ldc, int M, int N, int K,
                           int epilogue, int kernel, int flags, void* stream);
 /* Attention of `rows` queries at positions meta[0] ... over the slot's cache (already holding their keys and values);

@@ -13,6 +13,7 @@
 #include "twm_dense_rows.cuh"
 #include "twm_dense_simt.cuh"
 #include "twm_dense_tc.cuh"
+#include "twm_dense_tc2.cuh"
 
 namespace {
 
@@ -229,18 +230,38 @@ twm_status gemm_tc_launch(const bf16* a, int lda, const bf16* w, int ldw, void* 
                   flags, stream, 0, g);
 }
 
-// Column width of a tile: the one whose waves cost least.  Measured time of one 64-K stage of a wave of tiles:
-// 0.42, 0.25 and 0.20 us for 256, 128 and 64 columns.
-int tc_tile_width(int M, int N, bool gated, int sms)
+template <int EPI>
+twm_status gemm_tc2_launch(const bf16* a, int lda, const bf16* w, int ldw, void* c, int ldc, int M, int N, int K, int sms, int flags,
+                           void* stream)
+{
+    constexpr bool gated = EPI == TWM_EPI_GELU_GLU;
+    constexpr int out = gated ? T2_BN / 2 : T2_BN;
+    TcArgs g;
+    g.c = c; g.ldc = ldc; g.M = M; g.N = N; g.K = K;
+    g.m_tiles = (M + 2 * TC_BM - 1) / (2 * TC_BM);
+    g.n_tiles = (N + out - 1) / out;
+    if (!rows_map(&g.a_map, a, M, K, lda, TC_BM) || !rows_map(&g.w_map, w, gated ? 2L * N : N, K, ldw, TC_BM))
+        return invalid("cuTensorMapEncodeTiled refused a map of the paired tcgen05 product");
+    return launch("gemm_tc2", gemm_tc2_kernel<EPI>, dim3(2 * std::min(sms / 2, g.m_tiles * g.n_tiles)), TC_THREADS, T2_SMEM_BYTES, flags,
+                  stream, 2, g);
+}
+
+// Tile: the one whose waves cost least.  Measured time of one 64-K stage of a wave: 0.42, 0.25 and 0.20 us for tiles of
+// 128 rows x 256, 128 and 64 columns; 0.33 us for 256 x 256 on a pair of SMs (returned as 512).
+int tc_tile_choice(int M, int N, bool gated, int sms)
 {
     int best = 256;
     long best_cost = -1;
-    for (int bn : {256, 128, 64}) {
+    auto consider = [&](int choice, int rows, int bn, long units, int cost) {
         const int out = gated ? bn / 2 : bn;
-        const long tiles = (long)((M + TC_BM - 1) / TC_BM) * ((N + out - 1) / out);
-        const long cost = ((tiles + sms - 1) / sms) * (bn == 256 ? 42 : bn == 128 ? 25 : 20);
-        if (best_cost < 0 || cost < best_cost) { best = bn; best_cost = cost; }
-    }
+        const long tiles = (long)((M + rows - 1) / rows) * ((N + out - 1) / out);
+        const long c = ((tiles + units - 1) / units) * cost;
+        if (best_cost < 0 || c < best_cost) { best = choice; best_cost = c; }
+    };
+    consider(512, 256, 256, sms / 2, 33);
+    consider(256, 128, 256, sms, 42);
+    consider(128, 128, 128, sms, 25);
+    consider(64, 128, 64, sms, 20);
     return best;
 }
 
@@ -250,8 +271,9 @@ twm_status gemm_tc(const bf16* a, int lda, const bf16* w, int ldw, void* c, int 
 {
     int sms = 148;
     TRY(device(&sms));
-    if (width == 0) width = tc_tile_width(M, N, EPI == TWM_EPI_GELU_GLU, sms);
+    if (width == 0) width = tc_tile_choice(M, N, EPI == TWM_EPI_GELU_GLU, sms);
     switch (width) {
+        case 512: return gemm_tc2_launch<EPI>(a, lda, w, ldw, c, ldc, M, N, K, sms, flags, stream);
         case 256: return gemm_tc_launch<256, EPI>(a, lda, w, ldw, c, ldc, M, N, K, sms, flags, stream);
         case 128: return gemm_tc_launch<128, EPI>(a, lda, w, ldw, c, ldc, M, N, K, sms, flags, stream);
         default: return gemm_tc_launch<64, EPI>(a, lda, w, ldw, c, ldc, M, N, K, sms, flags, stream);
@@ -277,7 +299,7 @@ twm_status gemm(const T* a, int lda, const T* w, int ldw, void* c, int ldc, int 
                 void* stream)
 {
     const bool fits = std::is_same<T, bf16>::value && tc_fits(a, lda, w, ldw);
-    if (kernel != 0 && kernel != 1 && kernel != 2 && kernel != 64 && kernel != 128 && kernel != 256) return invalid("kernel");
+    if (kernel != 0 && kernel != 1 && kernel != 2 && kernel != 64 && kernel != 128 && kernel != 256 && kernel != 512) return invalid("kernel");
     if (kernel >= 2 && !fits) return invalid("the tcgen05 product takes bfloat16 rows on 16-byte boundaries");
     if (kernel >= 2 || (kernel == 0 && fits))
         return gemm_tc_any(a, lda, w, ldw, c, ldc, M, N, K, epi, kernel > 2 ? kernel : 0, flags, stream);

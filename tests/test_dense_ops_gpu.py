@@ -32,7 +32,7 @@ def gelu_tanh(z):
                                    (300, 1000, 336), (700, 2064, 128), (1024, 4096, 1024), (2100, 1530, 640)])
 @pytest.mark.parametrize("epi", [_dense.EPI_STORE, _dense.EPI_STORE_F32, _dense.EPI_GELU_GLU])
 @pytest.mark.parametrize("dtype,kernel", [(torch.float32, 1), (torch.bfloat16, 1), (torch.bfloat16, 2), (torch.bfloat16, 64),
-                                          (torch.bfloat16, 128), (torch.bfloat16, 256)])
+                                          (torch.bfloat16, 128), (torch.bfloat16, 256), (torch.bfloat16, 512)])
 def test_gemm(m, n, k, epi, dtype, kernel):
     gen = torch.Generator(device="cuda").manual_seed(m * 7 + n)
     a = torch.randn((m, k), generator=gen, device="cuda").to(dtype)
