@@ -527,7 +527,8 @@ twm_status decode(const twm_dense_model* m, const twm_dense_buffers* b, int want
         int splits = 1;
         while (splits < 16 && visible > 64L * splits && l.kv_heads * splits * 2 <= sms) splits *= 2;
         // a chunk of keys and values that leaves room for a product's CTA on the same SM, where heads are not too wide
-        auto bytes = [&](int chunk) { return attn_decode_smem_bytes<T>(l.heads / l.kv_heads, l.dim_pad, l.vdim_pad, chunk); };
+        auto bytes = [&](int chunk) { return attn_decode_smem_bytes<T>(l.heads / l.kv_heads, l.dim_pad, l.vdim_pad, chunk, splits); };
+        t.parts = attn_decode_parts(l.heads / l.kv_heads, l.vdim_pad);
         t.chunk = AD_MAX_CHUNK;
         while (t.chunk > 8 && bytes(t.chunk) > 80 * 1024) t.chunk /= 2;
         TRY(launch("attn_decode", attn_decode_kernel<T>, dim3(splits, l.kv_heads), AD_THREADS, bytes(t.chunk), flags, stream, splits, t));

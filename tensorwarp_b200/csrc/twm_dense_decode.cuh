@@ -240,12 +240,13 @@ gemv_kernel(const GemvArgs<T> g)
 }
 
 // One query of every head over the slot's cache.  CTA = (share of the visible keys, key/value head); the CTAs of a head
-// are one cluster and add their partial outputs through distributed shared memory (the weights are not
-// normalised, so a partial is a plain sum).  Takes the projection row as the product leaves it: the RMS norms of
-// the whole q and k rows are taken here, the CTA with the newest key appends it and its value.  A share of keys and
-// values is on its way into shared memory (cp.async) while the norms are taken; then a thread takes one
-// (key, query head) score at a time, and four value columns of one query head over the share's keys.
-constexpr int AD_THREADS = 256, AD_MAX_CHUNK = 128;   // keys in shared memory at a time, at most
+// are one cluster: each pushes its partial output, which is a plain sum because the weights are not normalised,
+// into the shared memory of the CTA that owns the columns, and after one cluster barrier the owners add up in rank
+// order, apply the gate and store.  Takes the projection row as the product leaves it: the RMS norms of the whole q
+// and k rows are taken here, the CTA with the newest key appends it and its value.  A share of keys and values is on
+// its way into shared memory (cp.async) while the norms are taken; then a thread takes one (key, query head) score at
+// a time, and four value columns of one query head over a part of the share's keys.
+constexpr int AD_THREADS = 512, AD_MAX_CHUNK = 128;   // keys in shared memory at a time, at most
 
 template <typename T>
 struct AttnDecodeArgs {
@@ -258,20 +259,22 @@ struct AttnDecodeArgs {
     const float* bias_table;
     const int* meta;
     int heads, kv_heads, dim, dim_pad, vdim_pad, window, keep_first, capacity, bias_len, gated;
-    int chunk;                  // keys in shared memory at a time, a multiple of 4
+    int chunk;                  // keys in shared memory at a time, a multiple of 8
+    int parts;                  // threads that share the keys of one output column quad
     float scale, eps;
 };
 
-template <typename T>
-__host__ inline size_t attn_decode_smem_bytes(int group, int dim_pad, int vdim_pad, int chunk) {
-    return sizeof(float) * ((size_t)group * dim_pad + (size_t)group * chunk + (size_t)group * vdim_pad) +
-           (size_t)chunk * (dim_pad * sizeof(T) + 16 + vdim_pad * sizeof(T));
+// threads per column quad: as many as the CTA has, up to four
+__host__ inline int attn_decode_parts(int group, int vdim_pad) {
+    const int n = AD_THREADS / (group * (vdim_pad / 4));
+    return n < 1 ? 1 : n > 4 ? 4 : n;
 }
-
-__device__ __forceinline__ float ld_cluster_f32(uint32_t addr) {
-    float v;
-    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr) : "memory");
-    return v;
+template <typename T>
+__host__ inline size_t attn_decode_smem_bytes(int group, int dim_pad, int vdim_pad, int chunk, int splits) {
+    const int slice = (group * vdim_pad + splits - 1) / splits;
+    return sizeof(float) * ((size_t)group * dim_pad + (size_t)group * chunk +
+                            (size_t)group * vdim_pad * attn_decode_parts(group, vdim_pad) + (((size_t)slice * splits + 3) & ~(size_t)3)) +
+           (size_t)chunk * (dim_pad * sizeof(T) + 16 + vdim_pad * sizeof(T));
 }
 
 template <typename T>
@@ -280,22 +283,48 @@ attn_decode_kernel(const AttnDecodeArgs<T> g)
 {
     using V = Vec<T>;
     pdl_launch_dependents();
+    asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");      // waited for before the first push
     extern __shared__ __align__(16) float ad_smem[];
     __shared__ float red[32];
-    const int group = g.heads / g.kv_heads;
+    const int group = g.heads / g.kv_heads, splits = gridDim.x, rank = blockIdx.x;
+    const int columns = group * g.vdim_pad, slice = (columns + splits - 1) / splits;       // a CTA owns `slice` output columns
     float* qs = ad_smem;                                   // [group][dim_pad], normalised and scaled
     float* ws = qs + group * g.dim_pad;                    // [group][chunk]
-    float* os = ws + group * g.chunk;                     // [group][vdim_pad]: this CTA's share of the output
+    float* os = ws + group * g.chunk;                      // [parts][group][vdim_pad]: this CTA's share of the output
+    float* recv = os + g.parts * columns;                  // [splits][slice]: what the cluster pushed here
     const int krow = g.dim_pad * (int)sizeof(T) + 16, vrow = g.vdim_pad * (int)sizeof(T);
-    uint8_t* ks = reinterpret_cast<uint8_t*>(os + group * g.vdim_pad);       // rows padded: a lane per key reads distinct banks
+    uint8_t* ks = reinterpret_cast<uint8_t*>(recv + ((slice * splits + 3) & ~3));       // rows padded: a lane per key reads distinct banks
     uint8_t* vs = ks + g.chunk * krow;
     const int tid = threadIdx.x;
-    const int kvh = blockIdx.y, splits = gridDim.x, rank = blockIdx.x;
+    const int kvh = blockIdx.y;
     const int kd = g.kv_heads * g.dim_pad, vd = g.kv_heads * g.vdim_pad, q_n = g.heads * g.dim_pad;
+    const int kp = g.dim_pad / V::N, vp = g.vdim_pad / V::N;       // 16-byte pieces of a key and of a value row
+    const int krow0 = tid / kp, kcol0 = tid - krow0 * kp, vrow0 = tid / vp, vcol0 = tid - vrow0 * vp;
+    const int kstep = AD_THREADS / kp, kwrap = AD_THREADS - kstep * kp, vstep = AD_THREADS / vp, vwrap = AD_THREADS - vstep * vp;
+    constexpr int QV = 2;                                  // a thread's first q elements and norm weights, ahead of the sum
+    float nq[QV];
+#pragma unroll
+    for (int j = 0; j < QV; ++j) {
+        const int i = tid + j * AD_THREADS;
+        nq[j] = g.q_norm != nullptr && i < group * g.dim_pad ? __ldg(g.q_norm + kvh * group * g.dim_pad + i) : 1.0f;
+    }
     pdl_wait_prior_grids();
-    const int p = g.meta[0];
-    T* kc = g.k_cache + (size_t)g.meta[1] * g.capacity * kd + kvh * g.dim_pad;
-    T* vc = g.v_cache + (size_t)g.meta[1] * g.capacity * vd + kvh * g.vdim_pad;
+    const int p = g.meta[0], slot = g.meta[1];
+    float q[QV];
+#pragma unroll
+    for (int j = 0; j < QV; ++j) {
+        const int i = tid + j * AD_THREADS;
+        q[j] = i < group * g.dim_pad ? g.proj[kvh * group * g.dim_pad + i] : 0.0f;
+    }
+    const int own = min(slice, columns - rank * slice);    // may be <= 0
+    const float gate = g.gated && tid < own ? g.proj[q_n + kd + vd + kvh * columns + rank * slice + tid] : 0.0f;
+    float qss = 0.0f;
+    if (g.q_norm != nullptr) {
+#pragma unroll 4
+        for (int i = tid; i < (q_n >> 2); i += AD_THREADS) qss += ops::sumsq4(reinterpret_cast<const float4*>(g.proj)[i]);
+    }
+    T* kc = g.k_cache + (size_t)slot * g.capacity * kd + kvh * g.dim_pad;
+    T* vc = g.v_cache + (size_t)slot * g.capacity * vd + kvh * g.vdim_pad;
     int sinks, lo;
     visible_range(p, g.window, g.keep_first, sinks, lo);
     const int total = sinks + (p - lo + 1);
@@ -303,39 +332,43 @@ attn_decode_kernel(const AttnDecodeArgs<T> g)
     const int t_begin = min(total, rank * per), t_end = min(total, t_begin + per);
 
     auto key_of = [&](int t) { return t < sinks ? t : lo + (t - sinks); };
-    const int kp = g.dim_pad / V::N, vp = g.vdim_pad / V::N;       // 16-byte pieces of a key and of a value row
     const bool newest = t_begin < t_end && t_end == total && p < g.capacity;      // this CTA's share ends with key p
     // the share's rows, all but the newest one, which is not in the cache yet
     auto load_share = [&](int t0, int n) {
-        for (int i = tid; i < n * kp; i += AD_THREADS) {
-            const int r = i / kp, c = i - r * kp, j = key_of(t0 + r);
+        for (int r = krow0, c = kcol0; r < n;) {
+            const int j = key_of(t0 + r);
             if (j < p) ops::att_cp_async16(smem_u32(ks + r * krow + c * 16), kc + (size_t)j * kd + c * V::N, 16);
+            r += kstep; c += kwrap;
+            if (c >= kp) { c -= kp; ++r; }
         }
-        for (int i = tid; i < n * vp; i += AD_THREADS) {
-            const int r = i / vp, c = i - r * vp, j = key_of(t0 + r);
+        for (int r = vrow0, c = vcol0; r < n;) {
+            const int j = key_of(t0 + r);
             if (j < p) ops::att_cp_async16(smem_u32(vs + r * vrow + c * 16), vc + (size_t)j * vd + c * V::N, 16);
+            r += vstep; c += vwrap;
+            if (c >= vp) { c -= vp; ++r; }
         }
         ops::att_cp_async_commit();
     };
     load_share(t_begin, min(g.chunk, t_end - t_begin));
 
     // norms of the whole rows
-    float qr = 1.0f, kr = 1.0f;
-    auto row_sq = [&](const float* v, int n) {
-        float ss = 0.0f;
-#pragma unroll 4
-        for (int i = tid; i < (n >> 2); i += AD_THREADS) ss += ops::sumsq4(reinterpret_cast<const float4*>(v)[i]);
-        return group_sum(ss, red, AD_THREADS, 1);
-    };
-    if (g.q_norm != nullptr) qr = inv_rms(row_sq(g.proj, q_n), g.heads * g.dim, g.eps);
-    if (newest && g.k_norm != nullptr) kr = inv_rms(row_sq(g.proj + q_n, kd), g.kv_heads * g.dim, g.eps);
-    for (int i = tid; i < group * g.dim_pad; i += AD_THREADS) {
-        const int e = kvh * group * g.dim_pad + i;
-        float q = g.proj[e];
-        if (g.q_norm != nullptr) q *= qr * g.q_norm[e];
-        qs[i] = q * g.scale;
+    float kr = 1.0f;
+    const float qr = g.q_norm != nullptr ? inv_rms(group_sum(qss, red, AD_THREADS, 1), g.heads * g.dim, g.eps) : 1.0f;
+    if (newest && g.k_norm != nullptr) {
+        float kss = 0.0f;
+        for (int i = tid; i < (kd >> 2); i += AD_THREADS) kss += ops::sumsq4(reinterpret_cast<const float4*>(g.proj + q_n)[i]);
+        kr = inv_rms(group_sum(kss, red, AD_THREADS, 1), g.kv_heads * g.dim, g.eps);
     }
-    for (int i = tid; i < group * g.vdim_pad; i += AD_THREADS) os[i] = 0.0f;
+#pragma unroll
+    for (int j = 0; j < QV; ++j) {
+        const int i = tid + j * AD_THREADS;
+        if (i < group * g.dim_pad) qs[i] = q[j] * (g.q_norm != nullptr ? qr * nq[j] : 1.0f) * g.scale;
+    }
+    for (int i = tid + QV * AD_THREADS; i < group * g.dim_pad; i += AD_THREADS) {
+        const int e = kvh * group * g.dim_pad + i;
+        qs[i] = g.proj[e] * (g.q_norm != nullptr ? qr * g.q_norm[e] : 1.0f) * g.scale;
+    }
+    for (int i = tid; i < g.parts * columns; i += AD_THREADS) os[i] = 0.0f;
 
     for (int t0 = t_begin; t0 < t_end; t0 += g.chunk) {
         const int n = min(g.chunk, t_end - t0);
@@ -357,16 +390,16 @@ attn_decode_kernel(const AttnDecodeArgs<T> g)
                 reinterpret_cast<T*>(vs + (n - 1) * vrow)[d] = vt;
             }
         }
+        const int nr = (n + 31) & ~31;
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
-        const int nr = (n + 31) & ~31;
         for (int i = tid; i < group * nr; i += AD_THREADS) {
             const int h = i / nr, tt = i - h * nr;                 // a warp's lanes: consecutive keys of one head
             if (tt >= n) continue;
             float bias = 0.0f;
             if (g.bias_table != nullptr) bias = __ldg(g.bias_table + (size_t)(kvh * group + h) * g.bias_len + (p - key_of(t0 + tt)));
             const uint8_t* kr_s = ks + tt * krow;
-            const float* q = qs + h * g.dim_pad;
+            const float* qh = qs + h * g.dim_pad;
             float s0 = 0.0f, s1 = 0.0f;
 #pragma unroll 4
             for (int c = 0; c < kp; ++c) {
@@ -374,7 +407,7 @@ attn_decode_kernel(const AttnDecodeArgs<T> g)
                 V::unpack(lds128(kr_s + c * 16), kf);
 #pragma unroll
                 for (int e = 0; e < V::N; e += 4) {
-                    const float4 qv = *reinterpret_cast<const float4*>(q + c * V::N + e);
+                    const float4 qv = *reinterpret_cast<const float4*>(qh + c * V::N + e);
                     s0 = fmaf(kf[e], qv.x, fmaf(kf[e + 1], qv.y, s0));
                     s1 = fmaf(kf[e + 2], qv.z, fmaf(kf[e + 3], qv.w, s1));
                 }
@@ -382,41 +415,41 @@ attn_decode_kernel(const AttnDecodeArgs<T> g)
             ws[h * g.chunk + tt] = sigmoid_f32(s0 + s1 + bias);
         }
         __syncthreads();
-        const int quads = g.vdim_pad / 4;
-        for (int i = tid; i < group * quads; i += AD_THREADS) {
-            const int h = i / quads, c = (i - h * quads) * 4;
+        const int quads = g.vdim_pad / 4, items = group * quads;
+        for (int i = tid; i < items * g.parts; i += AD_THREADS) {
+            const int part = i / items, item = i - part * items;
+            const int h = item / quads, c = (item - h * quads) * 4;
             float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
             const float* w = ws + h * g.chunk;
             const uint8_t* v0 = vs + c * sizeof(T);
 #pragma unroll 8
-            for (int tt = 0; tt < n; ++tt) {
+            for (int tt = part; tt < n; tt += g.parts) {
                 const float4 vf = load4(reinterpret_cast<const T*>(v0 + (size_t)tt * vrow));
                 const float wt = w[tt];
                 o0 = fmaf(wt, vf.x, o0); o1 = fmaf(wt, vf.y, o1); o2 = fmaf(wt, vf.z, o2); o3 = fmaf(wt, vf.w, o3);
             }
-            float4* o = reinterpret_cast<float4*>(os + h * g.vdim_pad + c);      // this thread's own columns
+            float4* o = reinterpret_cast<float4*>(os + part * columns + h * g.vdim_pad + c);     // this thread's own columns
             const float4 before = *o;
             *o = make_float4(before.x + o0, before.y + o1, before.z + o2, before.w + o3);
         }
     }
+    asm volatile("barrier.cluster.wait.aligned;" ::: "memory");    // every CTA of the cluster has started
     __syncthreads();
+    for (int i = tid; i < columns; i += AD_THREADS) {
+        float o = os[i];
+        for (int part = 1; part < g.parts; ++part) o += os[part * columns + i];
+        const int owner = i / slice;
+        st_cluster_f32(mapa_shared(smem_u32(recv + rank * slice + i - owner * slice), owner), o);
+    }
     cluster_sync_all();
-    for (int i = rank * AD_THREADS + tid; i < group * g.vdim_pad; i += splits * AD_THREADS) {
-        const int e = kvh * group * g.vdim_pad + i;
-        const float gate = g.gated ? g.proj[q_n + kd + vd + e] : 0.0f;
+    for (int i = tid; i < own; i += AD_THREADS) {
         float o = 0.0f;
-        const uint32_t at = smem_u32(os + i);
-        for (int s0 = 0; s0 < splits; s0 += 8) {                    // eight ranks' loads in flight, added in rank order
-            float part[8];
-#pragma unroll
-            for (int s = 0; s < 8; ++s) part[s] = s0 + s < splits ? ld_cluster_f32(mapa_shared(at, s0 + s)) : 0.0f;
-#pragma unroll
-            for (int s = 0; s < 8; ++s) o += part[s];
-        }
-        if (g.gated) o *= sigmoid_f32(gate);
+#pragma unroll 8
+        for (int s = 0; s < splits; ++s) o += recv[s * slice + i];
+        const int e = kvh * columns + rank * slice + i;
+        if (g.gated) o *= sigmoid_f32(i < AD_THREADS ? gate : g.proj[q_n + kd + vd + e]);
         g.out[e] = o;
     }
-    cluster_sync_all();                                             // nobody leaves while its shared memory may be read
 }
 
 }  // namespace dense
