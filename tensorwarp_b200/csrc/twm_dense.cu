@@ -158,26 +158,28 @@ EncodeTiledFn encode_tiled()
     return fn;
 }
 
-// A bf16 tensor of up to four dimensions (innermost first; strides in elements), boxes of 64 x box[1] x ..., 128-byte
-// swizzle, zeros outside.  A map is a pure description of memory, so maps are kept by what they describe.
+// A tensor of up to four dimensions (innermost first; strides in elements), zeros outside.  A map is a pure description
+// of memory, so maps are kept by what they describe.
+enum MapKind { MAP_BF16_SWIZZLED = 0, MAP_WORDS = 1 };      // bfloat16 in 128-byte swizzled boxes; 64-bit words as they are
 struct MapKey {
+    MapKind kind;
     const void* ptr;
     int rank;
     long dim[4], stride[4], box[4];
     bool operator==(const MapKey& o) const {
-        return ptr == o.ptr && rank == o.rank && std::equal(dim, dim + 4, o.dim) && std::equal(stride, stride + 4, o.stride) &&
+        return kind == o.kind && ptr == o.ptr && rank == o.rank && std::equal(dim, dim + 4, o.dim) && std::equal(stride, stride + 4, o.stride) &&
                std::equal(box, box + 4, o.box);
     }
 };
 struct MapHash {
     size_t operator()(const MapKey& k) const {
-        size_t h = (size_t)k.ptr + (size_t)k.rank;
+        size_t h = (size_t)k.ptr + (size_t)k.rank + 16 * (size_t)k.kind;
         for (int i = 0; i < 4; ++i)
             for (long v : {k.dim[i], k.stride[i], k.box[i]}) h = h * 1000003u ^ (size_t)v;
         return h;
     }
 };
-bool swizzled_map(CUtensorMap* map, const MapKey& key)
+bool tensor_map(CUtensorMap* map, const MapKey& key)
 {
     static std::unordered_map<MapKey, CUtensorMap, MapHash> cache;
     static std::mutex mutex;
@@ -191,10 +193,11 @@ bool swizzled_map(CUtensorMap* map, const MapKey& key)
     for (int i = 0; i < key.rank; ++i) {
         gdim[i] = (cuuint64_t)key.dim[i];
         box[i] = (cuuint32_t)key.box[i];
-        if (i > 0) gstride[i - 1] = (cuuint64_t)key.stride[i] * 2;
+        if (i > 0) gstride[i - 1] = (cuuint64_t)key.stride[i] * (key.kind == MAP_WORDS ? 8 : 2);
     }
-    if (enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, (cuuint32_t)key.rank, const_cast<void*>(key.ptr), gdim, gstride, box, estride,
-            CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+    const bool words = key.kind == MAP_WORDS;
+    if (enc(map, words ? CU_TENSOR_MAP_DATA_TYPE_UINT64 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, (cuuint32_t)key.rank, const_cast<void*>(key.ptr), gdim, gstride, box, estride,
+            CU_TENSOR_MAP_INTERLEAVE_NONE, words ? CU_TENSOR_MAP_SWIZZLE_NONE : CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
         return false;
     if (cache.size() > 8192) cache.clear();
@@ -204,7 +207,13 @@ bool swizzled_map(CUtensorMap* map, const MapKey& key)
 // [rows][cols] with row stride ld, boxes of 64 columns x box_rows
 bool rows_map(CUtensorMap* map, const void* ptr, long rows, long cols, long ld, int box_rows)
 {
-    return swizzled_map(map, MapKey{ptr, 2, {cols, rows, 0, 0}, {1, ld, 0, 0}, {TC_BK, box_rows, 0, 0}});
+    return tensor_map(map, MapKey{MAP_BF16_SWIZZLED, ptr, 2, {cols, rows, 0, 0}, {1, ld, 0, 0}, {TC_BK, box_rows, 0, 0}});
+}
+
+// [rows][words] of 64-bit words, boxes of box_words x box_rows
+bool word_rows_map(CUtensorMap* map, const void* ptr, long rows, long words, int box_words, int box_rows)
+{
+    return tensor_map(map, MapKey{MAP_WORDS, ptr, 2, {words, rows, 0, 0}, {1, words, 0, 0}, {box_words, box_rows, 0, 0}});
 }
 
 // ------------------------------------------------------------- operations --
@@ -362,9 +371,9 @@ twm_status attention_tc(const AttnArgs<bf16>& g, int end, int slots, int flags, 
     t.a = g;
     auto cache_map = [&](CUtensorMap* map, const bf16* base, int pad) {
         const long row = (long)g.kv_heads * pad;
-        return swizzled_map(map, MapKey{base, 4, {pad, g.kv_heads, end, slots}, {1, pad, row, row * g.capacity}, {64, 1, AT_K, 1}});
+        return tensor_map(map, MapKey{MAP_BF16_SWIZZLED, base, 4, {pad, g.kv_heads, end, slots}, {1, pad, row, row * g.capacity}, {64, 1, AT_K, 1}});
     };
-    if (!swizzled_map(&t.q_map, MapKey{g.proj, 3, {g.dim_pad, g.heads, g.rows, 0}, {1, g.dim_pad, g.ld, 0}, {64, 1, AT_Q, 0}}) ||
+    if (!tensor_map(&t.q_map, MapKey{MAP_BF16_SWIZZLED, g.proj, 3, {g.dim_pad, g.heads, g.rows, 0}, {1, g.dim_pad, g.ld, 0}, {64, 1, AT_Q, 0}}) ||
         !cache_map(&t.k_map, g.k_cache, g.dim_pad) || !cache_map(&t.v_map, g.v_cache, g.vdim_pad))
         return invalid("cuTensorMapEncodeTiled refused a map of the tcgen05 attention");
     return launch("attn_tc", attn_tc_kernel, dim3((g.rows + AT_Q - 1) / AT_Q, g.heads), AT_THREADS, sizeof(AttnTcSmem) + 1024, flags,
@@ -463,11 +472,16 @@ twm_status prefill(const twm_dense_model* m, const twm_dense_buffers* b, int row
 template <typename T, int PRO, bool GATED>
 twm_status gemv(GemvArgs<T> g, int sms, int flags, void* stream)
 {
-    const int out_rows = GATED ? GV_ROWS / 2 : GV_ROWS;
-    const int grid = std::min(sms, (g.N + out_rows - 1) / out_rows);
-    g.rounds = g.N / (grid * out_rows);
-    const int left = g.N - g.rounds * grid * out_rows;
+    const int rows = GV_ROWS / 2, stream_rows = GATED ? g.N : (g.N + 1) / 2;      // of each of the two streams
+    const int grid = std::min(sms, (stream_rows + rows - 1) / rows);
+    g.rounds = stream_rows / (grid * rows);
+    // a full round of an undivided product's second stream must exist in it too: an odd row count leaves its last row out
+    while (!GATED && g.rounds > 0 && g.rounds * grid * rows > g.N - stream_rows) --g.rounds;
+    const int left = stream_rows - g.rounds * grid * rows;
     g.last_rows = (left + grid - 1) / grid;
+    const long words = (long)g.ldw * sizeof(T) / 8;
+    if (!word_rows_map(&g.w_map, g.w, GATED ? 2L * g.N : g.N, words, GV_PIECE / 8, rows))
+        return invalid("cuTensorMapEncodeTiled refused a map of the decode product");
     const size_t act = gemv_smem_bytes<T>(g.ldw, 0), limit = kSmemLimit - 8 * 1024;      // static shared memory beside it
     if (act + 2 * GV_STAGE > limit) return invalid("an input row does not fit shared memory");
     g.stages = (int)std::min<size_t>(GV_MAX_STAGES, (limit - act) / GV_STAGE);

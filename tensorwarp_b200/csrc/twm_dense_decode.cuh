@@ -1,10 +1,13 @@
 // twm_dense_decode.cuh — one decoded token of a dense model: the streaming matrix-vector product and
 // the split-key attention.
 //
-// gemv_kernel: y = W a for one token, HBM-bound.  The CTAs (one per SM) take W's rows eight at a time in
-// turn, so that together they read one contiguous window of it; what is left after the last full round is
-// shared out evenly.  One thread streams them with 1-D bulk copies into a shared-memory ring, eight row
-// pieces of 2 KB a stage, and starts before the preceding kernel has finished (weights are constants);
+// gemv_kernel: y = W a for one token, HBM-bound.  W is read as two streams of rows (gate and up rows of a
+// gated product, otherwise its two halves).  The CTAs (one per SM) take four rows of each at a time in
+// turn, so that together they read two contiguous windows; what is left after the last full round is
+// shared out evenly.  One thread streams them into a shared-memory ring,
+// eight row pieces of 2 KB a stage: two tiled TMA loads (a copy per row piece would keep that thread busier
+// than the memory), and one bulk copy per row in the last, partial round.  It starts before the preceding
+// kernel has finished (weights are constants);
 // eight warps multiply: warps 0-3 the stage's rows 0-3, a quarter of the piece each, warps 4-7 the rows 4-7.
 // A CTA asks for more than half an SM's shared memory: with two to an SM, those of the next launch would
 // gather on the SMs that happen to be free.  The steps between two products
@@ -45,6 +48,7 @@ struct GemvArgs {
     float* shift_state;
     const float* final_norm;
     const int* meta;
+    alignas(64) CUtensorMap w_map;      // W's rows as 64-bit words, boxes of 256 words x 4 rows
 };
 
 template <typename T>
@@ -54,7 +58,7 @@ __host__ __device__ inline size_t gemv_smem_bytes(int ldw, int stages) {
 
 template <typename T, int PRO, bool GATED>
 __global__ void __launch_bounds__(GV_THREADS, 1)
-gemv_kernel(const GemvArgs<T> g)
+gemv_kernel(const __grid_constant__ GemvArgs<T> g)
 {
     using V = Vec<T>;
     extern __shared__ __align__(128) uint8_t gemv_smem[];
@@ -67,12 +71,14 @@ gemv_kernel(const GemvArgs<T> g)
     volatile int* abort_flag = &abort_s;
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    constexpr int OUT_ROWS = GATED ? GV_ROWS / 2 : GV_ROWS;         // outputs per row group
+    constexpr int OUT_ROWS = GV_ROWS / 2;                            // rows of each stream per row group
+    const int stream = GATED ? g.N : (g.N + 1) / 2;                  // rows of a stream; the second one may be a row shorter
     const int last_first = g.rounds * (int)gridDim.x * OUT_ROWS + (int)blockIdx.x * g.last_rows;
-    const int last_valid = max(0, min(g.last_rows, g.N - last_first));
+    const int last_valid = max(0, min(g.last_rows, stream - last_first));
     const int groups = g.rounds + (last_valid > 0 ? 1 : 0);
     auto group_first = [&](int gi) { return gi < g.rounds ? (gi * (int)gridDim.x + (int)blockIdx.x) * OUT_ROWS : last_first; };
     auto group_rows = [&](int gi) { return gi < g.rounds ? OUT_ROWS : last_valid; };
+    auto second_rows = [&](int gi) { return GATED ? group_rows(gi) : min(group_rows(gi), g.N - stream - group_first(gi)); };
     const int row_bytes = g.ldw * (int)sizeof(T);
     const int chunks = (row_bytes + GV_PIECE - 1) / GV_PIECE;
     const int iters = groups * chunks;
@@ -92,18 +98,20 @@ gemv_kernel(const GemvArgs<T> g)
             uint32_t phase = 0;
             for (int it = 0; it < iters; ++it) {
                 if (it >= g.stages && !mbar_wait_bounded(&empty[slot], phase, abort_flag)) break;
-                const int bytes = min(GV_PIECE, row_bytes - c * GV_PIECE);
-                const int o0 = group_first(gi), valid = group_rows(gi);      // outputs of this group
-                mbar_arrive_expect_tx(&full[slot], (uint32_t)bytes * (uint32_t)(GATED ? 2 * valid : valid));
                 uint8_t* dst = ring + (size_t)slot * GV_STAGE;
-                const uint8_t* src = reinterpret_cast<const uint8_t*>(g.w) + (size_t)o0 * row_bytes + (size_t)c * GV_PIECE;
-#pragma unroll
-                for (int r = 0; r < OUT_ROWS; ++r) {
-                    if (r < valid) {
+                const int o0 = group_first(gi);
+                if (gi < g.rounds) {
+                    mbar_arrive_expect_tx(&full[slot], GV_STAGE);
+                    tma_load_2d(dst, &g.w_map, c * (GV_PIECE / 8), o0, &full[slot]);
+                    tma_load_2d(dst + OUT_ROWS * GV_PIECE, &g.w_map, c * (GV_PIECE / 8), stream + o0, &full[slot]);
+                } else {
+                    const int bytes = min(GV_PIECE, row_bytes - c * GV_PIECE), valid = group_rows(gi), second = second_rows(gi);
+                    mbar_arrive_expect_tx(&full[slot], (uint32_t)bytes * (uint32_t)(valid + second));
+                    const uint8_t* src = reinterpret_cast<const uint8_t*>(g.w) + (size_t)o0 * row_bytes + (size_t)c * GV_PIECE;
+                    for (int r = 0; r < valid; ++r)
                         bulk_g2s(dst + r * GV_PIECE, src + (size_t)r * row_bytes, (uint32_t)bytes, &full[slot]);
-                        if (GATED)
-                            bulk_g2s(dst + (r + OUT_ROWS) * GV_PIECE, src + (size_t)(g.N + r) * row_bytes, (uint32_t)bytes, &full[slot]);
-                    }
+                    for (int r = 0; r < second; ++r)
+                        bulk_g2s(dst + (r + OUT_ROWS) * GV_PIECE, src + (size_t)(stream + r) * row_bytes, (uint32_t)bytes, &full[slot]);
                 }
                 if (++c == chunks) { c = 0; ++gi; }
                 if (++slot == g.stages) { slot = 0; if (it >= g.stages) phase ^= 1u; }
@@ -225,15 +233,16 @@ gemv_kernel(const GemvArgs<T> g)
         if ((lane & 7) == 0) part[buf][at][warp][lane >> 3] = v;
         if (at == GV_FLUSH - 1 || gi == groups - 1) {
             named_bar_sync(1, GV_CONSUMERS);
-            const int grp = tid / OUT_ROWS, row = tid % OUT_ROWS;    // one output per thread
+            const int grp = tid / GV_ROWS, row = tid % OUT_ROWS, which = (tid / OUT_ROWS) & 1;     // one row of one stream per thread
             const int gg = gi - at + grp;
-            if (grp <= at && row < group_rows(gg) && *abort_flag == 0) {
+            if (grp <= at && (GATED ? which == 0 && row < group_rows(gg) : row < (which ? second_rows(gg) : group_rows(gg))) &&
+                *abort_flag == 0) {
                 auto sum = [&](int stage_row) {
                     const float(*p)[4] = &part[buf][grp][(stage_row >> 2) * 4];
                     const int r = stage_row & 3;
                     return ((p[0][r] + p[1][r]) + (p[2][r] + p[3][r]));
                 };
-                g.out[group_first(gg) + row] = GATED ? gelu_tanh(sum(row)) * sum(row + 4) : sum(row);
+                g.out[group_first(gg) + row + (GATED ? 0 : which * stream)] = GATED ? gelu_tanh(sum(row)) * sum(row + 4) : sum(row + 4 * which);
             }
         }
     }
