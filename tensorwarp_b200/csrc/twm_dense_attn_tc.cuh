@@ -72,6 +72,9 @@ attn_tc_kernel(const __grid_constant__ AttnTcArgs args)
     constexpr float LOG2E = 1.4426950408889634f;
 
     if (tid == 0) {
+        prefetch_map(&args.q_map);
+        prefetch_map(&args.k_map);
+        prefetch_map(&args.v_map);
         for (uint64_t* bar : {&sm.q_full, &sm.k_full, &sm.k_empty, &sm.v_full, &sm.v_empty, &sm.s_full, &sm.o_full}) mbar_init(bar, 1);
         mbar_init(&sm.p_full, AT_SOFT / 32);
         sm.abort_flag = 0;

@@ -78,6 +78,11 @@ __device__ __forceinline__ bool elect_one() {
     return p != 0;
 }
 
+// Ask for a tensor map (kernel-parameter space) ahead of the first load that uses it.
+__device__ __forceinline__ void prefetch_map(const CUtensorMap* map) {
+    asm volatile("prefetch.tensormap [%0];" ::"l"(reinterpret_cast<uint64_t>(map)) : "memory");
+}
+
 // Which keys the query at position p sees: [0, sinks) and [lo, p].
 __device__ __forceinline__ void visible_range(int p, int window, int keep_first, int& sinks, int& lo) {
     lo = window > p ? 0 : p - window + 1;               // p - j < window

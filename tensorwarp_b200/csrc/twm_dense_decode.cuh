@@ -6,7 +6,8 @@
 // turn, so that together they read two contiguous windows; what is left after the last full round is
 // shared out evenly.  One thread streams them into a shared-memory ring,
 // eight row pieces of 2 KB a stage: two tiled TMA loads (a copy per row piece would keep that thread busier
-// than the memory), and one bulk copy per row in the last, partial round.  It starts before the preceding
+// than the memory), and one bulk copy per row for the first ring-full, which need not wait for the tensor
+// map, and in the last, partial round.  It starts before the preceding
 // kernel has finished (weights are constants);
 // eight warps multiply: warps 0-3 the stage's rows 0-3, a quarter of the piece each, warps 4-7 the rows 4-7.
 // A CTA asks for more than half an SM's shared memory: with two to an SM, those of the next launch would
@@ -84,6 +85,7 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
     const int iters = groups * chunks;
 
     if (tid == 0) {
+        prefetch_map(&g.w_map);
         for (int s = 0; s < g.stages; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], GV_CONSUMERS / 32); }
         abort_s = 0;
         mbar_fence_init();
@@ -100,7 +102,7 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
                 if (it >= g.stages && !mbar_wait_bounded(&empty[slot], phase, abort_flag)) break;
                 uint8_t* dst = ring + (size_t)slot * GV_STAGE;
                 const int o0 = group_first(gi);
-                if (gi < g.rounds) {
+                if (gi < g.rounds && it >= g.stages) {
                     mbar_arrive_expect_tx(&full[slot], GV_STAGE);
                     tma_load_2d(dst, &g.w_map, c * (GV_PIECE / 8), o0, &full[slot]);
                     tma_load_2d(dst + OUT_ROWS * GV_PIECE, &g.w_map, c * (GV_PIECE / 8), stream + o0, &full[slot]);

@@ -58,6 +58,8 @@ gemm_tc2_kernel(const __grid_constant__ TcArgs g)
     const int k_steps = (g.K + TC_BK - 1) / TC_BK;
 
     if (tid == 0) {
+        prefetch_map(&g.a_map);
+        prefetch_map(&g.w_map);
         for (int s = 0; s < T2_STAGES; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); }
         for (int i = 0; i < 2; ++i) { mbar_init(&acc_full[i], 1); mbar_init(&acc_empty[i], 8); }
         abort_s = 0;
