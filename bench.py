@@ -755,9 +755,14 @@ def bidasun_figures(torch, device, name: str, gbs: float, tflops: float) -> dict
     gen = torch.Generator(device=device).manual_seed(3)
     eng._buf["tokens"].copy_(torch.randint(0, v, eng._buf["tokens"].shape, generator=gen, device=device, dtype=torch.int32))
     eng._buf["want"].zero_()
+    # real operands: products of zeros draw little power and run at clocks that no workload sees
+    for t in [eng._buf[k] for k in ("a", "proj", "att", "act")] + eng.state.k + eng.state.v:
+        t.normal_(generator=gen)
     torch.cuda.synchronize()
 
     def timed(enqueue, steps, warm=3):
+        torch.cuda.synchronize()
+        time.sleep(0.5)          # directly after long prompts everything reads slower for a while
         with torch.cuda.stream(eng.stream):
             for _ in range(warm):
                 enqueue()
@@ -775,7 +780,6 @@ def bidasun_figures(torch, device, name: str, gbs: float, tflops: float) -> dict
         return full + sum(min(max(i + 1 - size["window"], 0), size["keep"]) for i in range(n))
 
     out = {"config": {k: size[k] for k in size}, "matrix_weights": matrices, "prefill": [], "decode": []}
-    # decoding before this size's prompts, as the 4-bit decoder's step is timed
     for ctx in (BIDASUN_CONTEXT, 8000):
         eng._set_step(ctx, 0, 1)
         graph = eng.capture_decode("greedy")
@@ -785,13 +789,6 @@ def bidasun_figures(torch, device, name: str, gbs: float, tflops: float) -> dict
         out["decode"].append({"context": ctx, "ms": round(ms, 4), "tok_s": round(1e3 / ms, 1), "bytes": nbytes,
                               "hbm_gbs": round(nbytes / ms / 1e6, 1), "frac_hbm": round(nbytes / ms / 1e6 / gbs, 3),
                               "launches": eng.launches_per_step})
-    for n in BIDASUN_PROMPTS:
-        eng._set_step(0, 0)
-        ms = timed(lambda: eng.enqueue_prefill(n, 0, 1), 5)
-        flops = 2.0 * n * matrices + nl * 4.0 * h * d * visible(n) + 2.0 * w * v
-        out["prefill"].append({"tokens": n, "ms": round(ms, 3), "tok_s": round(n / ms * 1e3), "tflops": round(flops / ms / 1e9, 1),
-                               "frac_bf16_peak": round(flops / ms / 1e9 / tflops, 3), "launches": eng.launches_per_step})
-
     # each product of a layer at each prompt length, over the layers' own weights in turn (larger than L2 together)
     b, p = eng._buf, []
     shapes = [("q|k|v|gate", "w_in", "a", "proj", 2 * h * d + 2 * g * d, w, _dense.EPI_STORE),
@@ -806,7 +803,7 @@ def bidasun_figures(torch, device, name: str, gbs: float, tflops: float) -> dict
                     _dense.check(lib.twm_dense_gemm(_dense.TWM_DENSE_BF16, b[src].data_ptr(), b[src].shape[1], lw[wt].data_ptr(), k,
                                                     b[dst].data_ptr(), b[dst].shape[1], n, cols, k, epi, 0, eng.flags,
                                                     eng.stream.cuda_stream), "gemm")
-            ms = timed(enqueue, 2, 1) / nl
+            ms = timed(enqueue, 4, 2) / nl
             tf = 2.0 * n * k * cols * (2 if epi == _dense.EPI_GELU_GLU else 1) / ms / 1e9
             nb = 2 * k * cols * (2 if epi == _dense.EPI_GELU_GLU else 1)
             row[label] = {"us": round(ms * 1e3, 1), "tflops": round(tf, 1),
@@ -817,11 +814,17 @@ def bidasun_figures(torch, device, name: str, gbs: float, tflops: float) -> dict
             for i in range(nl):
                 _dense.check(lib.twm_dense_attention(C.byref(eng._desc), i, C.byref(eng._b), n, 0, 0, eng.flags,
                                                      eng.stream.cuda_stream), "attention")
-        ms = timed(attend, 2, 1) / nl
+        ms = timed(attend, 4, 2) / nl
         tf = 4.0 * h * d * visible(n) / ms / 1e9
         row["attention"] = {"us": round(ms * 1e3, 1), "tflops": round(tf, 1), "frac_roofline": round(tf / tflops, 3)}
         p.append(row)
     out["prefill_kernels"] = p
+    for n in BIDASUN_PROMPTS:
+        eng._set_step(0, 0)
+        ms = timed(lambda: eng.enqueue_prefill(n, 0, 1), 5)
+        flops = 2.0 * n * matrices + nl * 4.0 * h * d * visible(n) + 2.0 * w * v
+        out["prefill"].append({"tokens": n, "ms": round(ms, 3), "tok_s": round(n / ms * 1e3), "tflops": round(flops / ms / 1e9, 1),
+                               "frac_bf16_peak": round(flops / ms / 1e9 / tflops, 3), "launches": eng.launches_per_step})
     out["device_error"] = _dense.device_error()
     return out
 
@@ -838,6 +841,7 @@ def q4_decode_same_size(torch, device, name: str, gbs: float) -> dict:
     eng.capture()
     eng.set_token(1)
     torch.cuda.synchronize()
+    time.sleep(0.5)
     with torch.cuda.stream(eng.stream):
         for _ in range(20):
             eng.replay()
