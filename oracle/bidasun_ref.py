@@ -15,7 +15,7 @@ import numpy as np
 
 
 def rms_norm(x, w, eps):
-    """x / sqrt(mean(x^2) + eps) * w over the last axis."""
+    """The last axis scaled to unit root mean square, eps under the root, then weighted."""
     return x / np.sqrt(np.mean(x * x, axis=-1, keepdims=True) + x.dtype.type(eps)) * w
 
 
