@@ -53,7 +53,7 @@ def main(argv=None) -> int:
     t.add_argument("--model", required=True)
     t.add_argument("--dtype", choices=["bfloat16", "float32"], required=True)
     t.add_argument("--out", required=True, help="folder for <step>.f32")
-    t.add_argument("--max-tokens", type=int, required=True, help="most tokens that live requests hold at any time")
+    t.add_argument("--max-tokens", type=int, required=True, help="room for this many tokens per sequence")
     t.set_defaults(run=_trace)
     m = sub.add_parser("models", help="list the architectures")
     m.set_defaults(run=_models)

@@ -1,7 +1,7 @@
 """Checkpoints: a folder with ``config.json`` and ``model.safetensors``.
 
-A safetensors file is an 8-byte little-endian header length, that many bytes of JSON (name -> dtype,
-shape, data_offsets relative to the end of the header), and the data.
+Layout of the latter: the header's size as a 64-bit little-endian integer, the header (a JSON object that
+gives dtype, shape and byte range of every tensor, counted from the header's end), then the raw tensors.
 """
 from __future__ import annotations
 
