@@ -45,6 +45,13 @@ class SafetensorsFile:
     def names(self) -> Iterable[str]:
         return self._entries.keys()
 
+    def shape(self, name: str) -> Tuple[int, ...]:
+        """The shape of the tensor `name`, for sizes that the configuration does not give."""
+        e = self._entries.get(name)
+        if e is None:
+            raise CheckpointError(f"{self.path}: tensor {name!r} is missing")
+        return tuple(e["shape"])
+
     def get(self, name: str, shape: Tuple[int, ...]) -> torch.Tensor:
         """The tensor `name`, which must have the given shape."""
         e = self._entries.get(name)

@@ -56,6 +56,12 @@ __device__ __forceinline__ float gelu_tanh(float z) {
     return 0.5f * z * (1.0f + tanhf(u));
 }
 __device__ __forceinline__ float sigmoid_f32(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float silu_f32(float z) { return z * sigmoid_f32(z); }
+__device__ __forceinline__ float log_sigmoid_f32(float z) { return fminf(z, 0.0f) - log1pf(expf(-fabsf(z))); }
+__device__ __forceinline__ float squared_relu(float z) { const float p = fmaxf(z, 0.0f); return p * p; }
+// what a product's epilogue does to a single sum
+template <int EPI>
+__device__ __forceinline__ float epilogue_value(float v) { return EPI == TWM_EPI_RELU2 ? squared_relu(v) : v; }
 
 // Sum over the `threads` threads (a multiple of 32, all taking part) that share named barrier `bar`; `red` holds 32
 // floats.  Every thread gets the sum, added in warp order.

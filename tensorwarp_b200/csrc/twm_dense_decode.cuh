@@ -16,8 +16,14 @@
 // sublayer output that joins it (norm, add, token shift or final norm), in FP32, and rounds it once.
 // The epilogue of the gate/up product applies the gated activation, so no launch stands between products
 // but the attention.
+//
+// Routed products (experts) differ in where a row comes from.  ROUTE_ROWS (up): the `top` chosen experts' rows, one
+// expert after the other, are one long list of rows; the first warp makes the choice from the router's logits.
+// ROUTE_COLUMNS (down): a row is the chosen experts' rows side by side, and the input is their activations side by
+// side, each times its expert's weight; so the sum over experts is part of the product.
 #pragma once
 
+#include "twm_dense_moe.cuh"
 #include "twm_dense_rows.cuh"
 #include "twm_dense_simt.cuh"
 #include "twm_gemm_tc.cuh"
@@ -25,7 +31,8 @@
 namespace twm {
 namespace dense {
 
-enum { PRO_VEC = 0, PRO_RESIDUAL = 1, PRO_SHIFT = 2, PRO_FINAL = 3 };
+enum { PRO_VEC = 0, PRO_RESIDUAL = 1, PRO_SHIFT = 2, PRO_NORM = 3 };
+enum { ROUTE_NONE = 0, ROUTE_ROWS = 1, ROUTE_COLUMNS = 2 };
 
 constexpr int GV_CONSUMERS = 256;
 constexpr int GV_THREADS = GV_CONSUMERS + 32;
@@ -47,22 +54,33 @@ struct GemvArgs {
     float* x_out;               // the residual row after the add, written by CTA 0
     const float* shift;
     float* shift_state;
-    const float* final_norm;
+    const float* pre_norm;      // PRO_NORM: the input row is rms_norm(residual row) * pre_norm
     const int* meta;
+    // routed: W is [experts][expert_rows][ldw].  ROUTE_ROWS: N = top * expert_rows, the choice is made from `logits` and left
+    // in ids and weights.  ROUTE_COLUMNS: N = expert_rows, vec is [top][ldw].
+    RouterArgs router;
+    int expert_rows;
+    const float* logits;
+    int* ids;
+    float* weights;
     alignas(64) CUtensorMap w_map;      // W's rows as 64-bit words, boxes of 256 words x 4 rows
 };
 
-template <typename T>
-__host__ __device__ inline size_t gemv_smem_bytes(int ldw, int stages) {
-    return (size_t)stages * GV_STAGE + (((size_t)ldw * sizeof(T) + 127) & ~(size_t)127);
+// row pieces of one expert's row: each expert's input starts on a piece of its own
+__host__ __device__ inline int gemv_pieces(size_t row_bytes) { return (int)((row_bytes + GV_PIECE - 1) / GV_PIECE); }
+__host__ __device__ inline size_t gemv_smem_bytes(size_t row_bytes, int parts, int stages) {
+    return (size_t)stages * GV_STAGE + (parts > 1 ? (size_t)parts * gemv_pieces(row_bytes) * GV_PIECE : ((row_bytes + 127) & ~(size_t)127));
 }
 
-template <typename T, int PRO, bool GATED>
+template <typename T, int PRO, int EPI, int ROUTE>
 __global__ void __launch_bounds__(GV_THREADS, 1)
 gemv_kernel(const __grid_constant__ GemvArgs<T> g)
 {
     using V = Vec<T>;
+    constexpr bool GATED = EPI == TWM_EPI_GELU_GLU;
     extern __shared__ __align__(128) uint8_t gemv_smem[];
+    __shared__ float route_s[ROUTE == ROUTE_ROWS ? 2 * MOE_MAX_EXPERTS : 1];
+    __shared__ int ids_s[ROUTE != ROUTE_NONE ? MOE_MAX_TOP : 1];
     uint8_t* ring = gemv_smem;
     T* as = reinterpret_cast<T*>(gemv_smem + (size_t)g.stages * GV_STAGE);
     __shared__ __align__(8) uint64_t full[GV_MAX_STAGES], empty[GV_MAX_STAGES];
@@ -81,7 +99,14 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
     auto group_rows = [&](int gi) { return gi < g.rounds ? OUT_ROWS : last_valid; };
     auto second_rows = [&](int gi) { return GATED ? group_rows(gi) : min(group_rows(gi), g.N - stream - group_first(gi)); };
     const int row_bytes = g.ldw * (int)sizeof(T);
-    const int chunks = (row_bytes + GV_PIECE - 1) / GV_PIECE;
+    const int pieces = (row_bytes + GV_PIECE - 1) / GV_PIECE;        // of one row as it lies in memory
+    const int chunks = ROUTE == ROUTE_COLUMNS ? pieces * g.router.top : pieces;
+    // where row o of the list lies, its chunk's expert given
+    auto physical = [&](int o, int slot) {
+        if (ROUTE == ROUTE_ROWS) return ids_s[o / g.expert_rows] * g.expert_rows + o % g.expert_rows;
+        if (ROUTE == ROUTE_COLUMNS) return ids_s[slot] * g.expert_rows + o;
+        return o;
+    };
     const int iters = groups * chunks;
 
     if (tid == 0) {
@@ -95,6 +120,7 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
 
     if (warp == GV_CONSUMERS / 32) {
         // ------------------------------------------------------------ producer --
+        if (ROUTE != ROUTE_NONE) named_bar_sync(2, 64);              // the choice is in ids_s
         if (elect_one()) {
             int slot = 0, c = 0, gi = 0;
             uint32_t phase = 0;
@@ -102,18 +128,21 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
                 if (it >= g.stages && !mbar_wait_bounded(&empty[slot], phase, abort_flag)) break;
                 uint8_t* dst = ring + (size_t)slot * GV_STAGE;
                 const int o0 = group_first(gi);
+                const int part = ROUTE == ROUTE_COLUMNS ? c / pieces : 0, piece = c - part * pieces;
+                // a full group's four rows lie together: an expert's rows are a multiple of 16
                 if (gi < g.rounds && it >= g.stages) {
                     mbar_arrive_expect_tx(&full[slot], GV_STAGE);
-                    tma_load_2d(dst, &g.w_map, c * (GV_PIECE / 8), o0, &full[slot]);
-                    tma_load_2d(dst + OUT_ROWS * GV_PIECE, &g.w_map, c * (GV_PIECE / 8), stream + o0, &full[slot]);
+                    tma_load_2d(dst, &g.w_map, piece * (GV_PIECE / 8), physical(o0, part), &full[slot]);
+                    tma_load_2d(dst + OUT_ROWS * GV_PIECE, &g.w_map, piece * (GV_PIECE / 8), physical(stream + o0, part), &full[slot]);
                 } else {
-                    const int bytes = min(GV_PIECE, row_bytes - c * GV_PIECE), valid = group_rows(gi), second = second_rows(gi);
+                    const int bytes = min(GV_PIECE, row_bytes - piece * GV_PIECE), valid = group_rows(gi), second = second_rows(gi);
                     mbar_arrive_expect_tx(&full[slot], (uint32_t)bytes * (uint32_t)(valid + second));
-                    const uint8_t* src = reinterpret_cast<const uint8_t*>(g.w) + (size_t)o0 * row_bytes + (size_t)c * GV_PIECE;
+                    const uint8_t* src = reinterpret_cast<const uint8_t*>(g.w) + (size_t)piece * GV_PIECE;
                     for (int r = 0; r < valid; ++r)
-                        bulk_g2s(dst + r * GV_PIECE, src + (size_t)r * row_bytes, (uint32_t)bytes, &full[slot]);
+                        bulk_g2s(dst + r * GV_PIECE, src + (size_t)physical(o0 + r, part) * row_bytes, (uint32_t)bytes, &full[slot]);
                     for (int r = 0; r < second; ++r)
-                        bulk_g2s(dst + (r + OUT_ROWS) * GV_PIECE, src + (size_t)(stream + r) * row_bytes, (uint32_t)bytes, &full[slot]);
+                        bulk_g2s(dst + (r + OUT_ROWS) * GV_PIECE, src + (size_t)physical(stream + o0 + r, part) * row_bytes, (uint32_t)bytes,
+                                 &full[slot]);
                 }
                 if (++c == chunks) { c = 0; ++gi; }
                 if (++slot == g.stages) { slot = 0; if (it >= g.stages) phase ^= 1u; }
@@ -124,7 +153,28 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
 
     // ------------------------------------------------------- prologue (256 threads) --
     pdl_wait_prior_grids();
-    if (PRO == PRO_VEC) {
+    if (ROUTE != ROUTE_NONE && warp == 0) {
+        int id = 0;
+        if (ROUTE == ROUTE_ROWS) {
+            float weight;
+            route_warp(g.logits, g.router, route_s, route_s + MOE_MAX_EXPERTS, lane, id, weight);
+            if (blockIdx.x == 0 && lane < g.router.top) { g.ids[lane] = id; g.weights[lane] = weight; }
+        } else if (lane < g.router.top) {
+            id = g.ids[lane];
+        }
+        if (lane < g.router.top) ids_s[lane] = id;
+        named_bar_sync(2, 64);
+    }
+    if (ROUTE == ROUTE_COLUMNS) {
+        for (int s = 0; s < g.router.top; ++s) {
+            const float ws = g.weights[s];
+            T* dst = as + (size_t)s * pieces * (GV_PIECE / sizeof(T));
+            for (int i = tid; i < (g.ldw >> 2); i += GV_CONSUMERS) {
+                const float4 v = reinterpret_cast<const float4*>(g.vec + (size_t)s * g.ldw)[i];
+                store4<T>(dst + i * 4, make_float4(v.x * ws, v.y * ws, v.z * ws, v.w * ws));
+            }
+        }
+    } else if (PRO == PRO_VEC) {
         for (int i = tid; i < (g.ldw >> 2); i += GV_CONSUMERS) store4<T>(as + i * 4, reinterpret_cast<const float4*>(g.vec)[i]);
     } else {
         const int pos = g.meta[0];
@@ -141,10 +191,7 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
                 h = shift4(x, before, __ldg(reinterpret_cast<const float4*>(g.shift) + i));
                 if (writer) reinterpret_cast<float4*>(st + (size_t)(pos & 1) * wp)[i] = x;      // the other half of the pair
             }
-            if (PRO == PRO_FINAL) {
-                const float4 n = __ldg(reinterpret_cast<const float4*>(g.final_norm) + i);
-                h = make_float4(x.x * fr * n.x, x.y * fr * n.y, x.z * fr * n.z, x.w * fr * n.w);
-            }
+            if (PRO == PRO_NORM) h = scale4(x, fr, __ldg(reinterpret_cast<const float4*>(g.pre_norm) + i));
             if (writer && g.x_out != nullptr) reinterpret_cast<float4*>(g.x_out)[i] = x;
             store4<T>(as + i * 4, h);
         };
@@ -152,7 +199,7 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
             return st_before != nullptr ? reinterpret_cast<const float4*>(st_before)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
         };
         constexpr int PER = 4;
-        if (nvec <= PER * GV_CONSUMERS && g.src.tokens == nullptr && g.src.y != nullptr && g.src.y_norm != nullptr) {
+        if (nvec <= PER * GV_CONSUMERS && g.src.tokens == nullptr) {
             // rows of up to 4096: everything is requested before the first use
             const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
             float4 x[PER], y[PER], before[PER];
@@ -160,31 +207,39 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
             for (int j = 0; j < PER; ++j) {
                 const int i = tid + j * GV_CONSUMERS;
                 const bool in = i < nvec;
-                y[j] = in ? reinterpret_cast<const float4*>(g.src.y)[i] : zero;
+                y[j] = in && g.src.y != nullptr ? reinterpret_cast<const float4*>(g.src.y)[i] : zero;
                 x[j] = in ? reinterpret_cast<const float4*>(g.src.x_in)[i] : zero;
                 before[j] = PRO == PRO_SHIFT && in ? state_at(i) : zero;
             }
-            float ss = 0.0f;
+            float ss = 0.0f, ir = 1.0f;
+            const bool normed = g.src.y != nullptr && g.src.y_norm != nullptr;
+            if (normed) {
 #pragma unroll
-            for (int j = 0; j < PER; ++j) ss += ops::sumsq4(y[j]);
-            const float ir = inv_rms(group_sum(ss, red, GV_CONSUMERS, 1), g.src.width, g.src.eps);
+                for (int j = 0; j < PER; ++j) ss += ops::sumsq4(y[j]);
+                ir = inv_rms(group_sum(ss, red, GV_CONSUMERS, 1), g.src.width, g.src.eps);
+            }
             ss = 0.0f;
 #pragma unroll
             for (int j = 0; j < PER; ++j) {
                 const int i = tid + j * GV_CONSUMERS;
                 if (i < nvec) {
-                    const float4 n = __ldg(reinterpret_cast<const float4*>(g.src.y_norm) + i);
+                    float4 n = make_float4(1.f, 1.f, 1.f, 1.f);
+                    if (normed) n = __ldg(reinterpret_cast<const float4*>(g.src.y_norm) + i);
                     x[j].x += y[j].x * ir * n.x; x[j].y += y[j].y * ir * n.y; x[j].z += y[j].z * ir * n.z; x[j].w += y[j].w * ir * n.w;
+                    if (g.src.step != nullptr) {
+                        const float4 t = __ldg(reinterpret_cast<const float4*>(g.src.step) + i);
+                        x[j].x += t.x; x[j].y += t.y; x[j].z += t.z; x[j].w += t.w;
+                    }
                 }
                 ss += ops::sumsq4(x[j]);
             }
-            if (PRO == PRO_FINAL) fr = inv_rms(group_sum(ss, red, GV_CONSUMERS, 1), g.src.width, g.src.eps);
+            if (PRO == PRO_NORM) fr = inv_rms(group_sum(ss, red, GV_CONSUMERS, 1), g.src.width, g.src.eps);
 #pragma unroll
             for (int j = 0; j < PER; ++j)
                 if (tid + j * GV_CONSUMERS < nvec) finish(tid + j * GV_CONSUMERS, x[j], before[j]);
         } else {
             const float ir = g.src.row_inv_rms(0, red, GV_CONSUMERS, 1);
-            if (PRO == PRO_FINAL) {
+            if (PRO == PRO_NORM) {
                 float ss = 0.0f;
                 for (int i = tid; i < nvec; i += GV_CONSUMERS) ss += ops::sumsq4(g.src.at(0, pos, tok, i, ir));
                 fr = inv_rms(group_sum(ss, red, GV_CONSUMERS, 1), g.src.width, g.src.eps);
@@ -202,9 +257,12 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
     bool ok = true;
     for (int gi = 0; gi < groups; ++gi) {
         float acc[4] = {0.f, 0.f, 0.f, 0.f};
+        int piece = 0;
         for (int c = 0; c < chunks; ++c) {
             ok = tc::wait_uniform(&full[slot], phase, abort_flag) && ok;
-            if (ok && c * GV_PIECE + off < row_bytes) {
+            const bool in = piece * GV_PIECE + off < row_bytes;
+            if (++piece == pieces) piece = 0;
+            if (ok && in) {
                 float af[V::N];
                 V::unpack(lds128(reinterpret_cast<const uint8_t*>(as) + (size_t)c * GV_PIECE + off), af);
                 const uint8_t* st = ring + (size_t)slot * GV_STAGE + half * 4 * GV_PIECE + off;
@@ -244,7 +302,8 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
                     const int r = stage_row & 3;
                     return ((p[0][r] + p[1][r]) + (p[2][r] + p[3][r]));
                 };
-                g.out[group_first(gg) + row + (GATED ? 0 : which * stream)] = GATED ? gelu_tanh(sum(row)) * sum(row + 4) : sum(row + 4 * which);
+                g.out[group_first(gg) + row + (GATED ? 0 : which * stream)] = GATED ? gelu_tanh(sum(row)) * sum(row + 4)
+                                                                                  : epilogue_value<EPI>(sum(row + 4 * which));
             }
         }
     }

@@ -1,0 +1,627 @@
+// twm_dense_gla.cuh — gated linear attention: per head a matrix state S [dim][vdim] in FP32 with one decay per key
+// channel, S_t = diag(alpha_t) S_{t-1} + k_t v_t^T, o_t = S_t^T q_t; each head's o is RMS-normed, weighted and
+// multiplied by silu(gate).
+//
+// Prompt steps, bfloat16: chunks of 64 tokens.  With b_t the running sum of log alpha inside a chunk,
+//   o_t = (q_t e^{b_t})^T S_chunk + sum_{s <= t} (sum_d q_td k_sd e^{b_td - b_sd}) v_s.
+//   gla_decay_kernel        b, from the low-rank projection
+//   gla_chunk_state_kernel  what each chunk adds to the state, all chunks at once
+//   gla_scan_kernel         the state ahead of every chunk, chunk by chunk, element by element
+//   gla_chunk_out_kernel    o, norm and gate, all chunks at once
+// Every factor with a decay is computed in FP32 and enters a warp-level MMA as a bf16 pair hi + lo.  The exponents are
+// taken against the first token of a 16-token block, so no factor exceeds 1; inside a block against its middle, which
+// is safe while eight steps stay within e^80, and token pair by token pair otherwise.
+// Everything else (FP32, wide heads): gla_rows_kernel walks the tokens one by one, gla_gate_kernel norms and gates.
+// Decoding: gla_decode_kernel.
+#pragma once
+
+#include "twm_dense_attn.cuh"
+#include "twm_dense_rows.cuh"
+
+namespace twm {
+namespace dense {
+
+constexpr int GLA_CHUNK = 64;
+constexpr float GLA_STEP_FLOOR = -10.0f;        // log decay of a step below which a block is done pair by pair
+
+template <typename T>
+struct GlaArgs {
+    const T* proj;              // [rows][ld]: q | k | v | gate | low-rank
+    float* decay;               // [rows][heads * dim_pad]: running sums of log alpha inside chunks of `chunk` rows
+    float* chunk_state;         // [chunks][heads][dim_pad][vdim_pad]
+    float* mix;                 // [rows][heads * vdim_pad], token by token only
+    T* out;                     // [rows][heads * vdim_pad]
+    float* state;               // [slots][heads][dim_pad][vdim_pad]
+    const T* w_decay;           // [heads * dim_pad][rank_pad]
+    const float* decay_bias;    // [heads * dim_pad]
+    const float* head_norm;     // [vdim_pad]
+    const int* meta;
+    int ld, heads, dim_pad, vdim, vdim_pad, rank_pad, rows, chunk;
+    float inv_tau, q_scale, eps;
+    __device__ __forceinline__ int k_off() const { return heads * dim_pad; }
+    __device__ __forceinline__ int v_off() const { return 2 * heads * dim_pad; }
+    __device__ __forceinline__ int gate_off() const { return 2 * heads * dim_pad + heads * vdim_pad; }
+    __device__ __forceinline__ int low_off() const { return 2 * heads * (dim_pad + vdim_pad); }
+    __device__ __forceinline__ float* slot_state(int h) const { return state + ((size_t)meta[1] * heads + h) * dim_pad * vdim_pad; }
+};
+
+// A thread per key channel and run of up to 64 rows: log alpha = log(sigmoid(z)) / tau, summed up within chunks.
+constexpr int GD_THREADS = 128, GD_ROWS = 64, GD_RANK = 32;
+template <typename T>
+__global__ void __launch_bounds__(GD_THREADS)
+gla_decay_kernel(const GlaArgs<T> g)
+{
+    using V = Vec<T>;
+    pdl_launch_dependents();
+    __shared__ __align__(16) float low[GD_ROWS][GD_RANK];
+    const int col = blockIdx.x * GD_THREADS + threadIdx.x, r0 = blockIdx.y * GD_ROWS, n = min(GD_ROWS, g.rows - r0);
+    const int cols = g.heads * g.dim_pad;
+    const float bias = col < cols ? __ldg(g.decay_bias + col) : 0.0f;
+    pdl_wait_prior_grids();
+    float z[GD_ROWS];
+#pragma unroll
+    for (int r = 0; r < GD_ROWS; ++r) z[r] = bias;
+    for (int k0 = 0; k0 < g.rank_pad; k0 += GD_RANK) {
+        const int kn = min(GD_RANK, g.rank_pad - k0);
+        __syncthreads();
+        for (int i = threadIdx.x; i < n * kn; i += GD_THREADS) {
+            const int r = i / kn, k = i - r * kn;
+            low[r][k] = to_f32(g.proj[(size_t)(r0 + r) * g.ld + g.low_off() + k0 + k]);
+        }
+        __syncthreads();
+        if (col < cols) {
+            for (int k = 0; k < kn; k += V::N) {
+                float w[V::N];
+                V::unpack(__ldg(reinterpret_cast<const uint4*>(g.w_decay + (size_t)col * g.rank_pad + k0 + k)), w);
+#pragma unroll
+                for (int r = 0; r < GD_ROWS; ++r)
+#pragma unroll
+                    for (int e = 0; e < V::N; e += 4) {
+                        const float4 a = *reinterpret_cast<const float4*>(&low[r][k + e]);
+                        z[r] = fmaf(w[e], a.x, fmaf(w[e + 1], a.y, fmaf(w[e + 2], a.z, fmaf(w[e + 3], a.w, z[r]))));
+                    }
+            }
+        }
+    }
+    if (col >= cols) return;
+    float sum = 0.0f;
+#pragma unroll
+    for (int r = 0; r < GD_ROWS; ++r) {
+        if (r >= n) break;
+        const float la = log_sigmoid_f32(z[r]) * g.inv_tau;
+        sum = (r0 + r) % g.chunk == 0 ? la : sum + la;
+        g.decay[(size_t)(r0 + r) * cols + col] = sum;
+    }
+}
+
+// Token by token: CTA = 32 value columns of a head, thread = a column and every eighth key channel.
+constexpr int GR_THREADS = 256, GR_COLS = 32, GR_TOKENS = 8;
+__host__ inline size_t gla_rows_smem_bytes(int dim_pad) { return sizeof(float) * (size_t)(dim_pad * GR_COLS + 3 * GR_TOKENS * dim_pad); }
+template <typename T>
+__global__ void __launch_bounds__(GR_THREADS)
+gla_rows_kernel(const GlaArgs<T> g)
+{
+    pdl_launch_dependents();
+    extern __shared__ __align__(16) float gr_smem[];
+    __shared__ float part[GR_TOKENS][8][GR_COLS];
+    float* s = gr_smem;                                    // [dim_pad][32]
+    float* qs = s + g.dim_pad * GR_COLS;                   // [tokens][dim_pad]
+    float* ks = qs + GR_TOKENS * g.dim_pad;
+    float* as = ks + GR_TOKENS * g.dim_pad;
+    pdl_wait_prior_grids();
+    const int h = blockIdx.y, c = threadIdx.x & 31, grp = threadIdx.x >> 5, col = blockIdx.x * GR_COLS + c;
+    const bool in = col < g.vdim_pad;
+    float* st = g.slot_state(h);
+    const bool fresh = g.meta[0] == 0;                     // the state ahead of a sequence's first token is zero
+    for (int d = grp; d < g.dim_pad; d += 8) s[d * GR_COLS + c] = in && !fresh ? st[(size_t)d * g.vdim_pad + col] : 0.0f;
+    for (int t0 = 0; t0 < g.rows; t0 += GR_TOKENS) {
+        const int n = min(GR_TOKENS, g.rows - t0);
+        __syncthreads();
+        for (int i = threadIdx.x; i < n * g.dim_pad; i += GR_THREADS) {
+            const int t = i / g.dim_pad, d = i - t * g.dim_pad;
+            const T* row = g.proj + (size_t)(t0 + t) * g.ld + h * g.dim_pad + d;
+            qs[i] = to_f32(row[0]) * g.q_scale;
+            ks[i] = to_f32(row[g.k_off()]);
+            as[i] = expf(g.decay[(size_t)(t0 + t) * g.heads * g.dim_pad + h * g.dim_pad + d]);
+        }
+        __syncthreads();
+        for (int t = 0; t < n; ++t) {
+            const float v = in ? to_f32(g.proj[(size_t)(t0 + t) * g.ld + g.v_off() + h * g.vdim_pad + col]) : 0.0f;
+            float o = 0.0f;
+            for (int d = grp; d < g.dim_pad; d += 8) {
+                const float x = fmaf(s[d * GR_COLS + c], as[t * g.dim_pad + d], ks[t * g.dim_pad + d] * v);
+                s[d * GR_COLS + c] = x;
+                o = fmaf(x, qs[t * g.dim_pad + d], o);
+            }
+            part[t][grp][c] = o;
+        }
+        __syncthreads();
+        for (int i = threadIdx.x; i < n * GR_COLS; i += GR_THREADS) {
+            const int t = i / GR_COLS, k = i - t * GR_COLS;
+            float o = 0.0f;
+            for (int w = 0; w < 8; ++w) o += part[t][w][k];
+            if (blockIdx.x * GR_COLS + k < g.vdim_pad)
+                g.mix[(size_t)(t0 + t) * g.heads * g.vdim_pad + h * g.vdim_pad + blockIdx.x * GR_COLS + k] = o;
+        }
+    }
+    if (in)
+        for (int d = grp; d < g.dim_pad; d += 8) st[(size_t)d * g.vdim_pad + col] = s[d * GR_COLS + c];
+}
+
+// One warp per (row, head): norm over the head's value columns, weight, silu(gate).
+template <typename T>
+__global__ void __launch_bounds__(ROW_THREADS)
+gla_gate_kernel(const GlaArgs<T> g)
+{
+    pdl_launch_dependents();
+    pdl_wait_prior_grids();
+    const int lane = threadIdx.x & 31, r = blockIdx.x;
+    for (int h = threadIdx.x >> 5; h < g.heads; h += ROW_THREADS / 32) {
+        const float* o = g.mix + ((size_t)r * g.heads + h) * g.vdim_pad;
+        float ss = 0.0f;
+        for (int i = lane; i < g.vdim_pad; i += 32) ss = fmaf(o[i], o[i], ss);
+        const float ir = inv_rms(ops::warp_sum(ss), g.vdim, g.eps);
+        const T* gate = g.proj + (size_t)r * g.ld + g.gate_off() + h * g.vdim_pad;
+        for (int i = lane; i < g.vdim_pad; i += 32)
+            g.out[((size_t)r * g.heads + h) * g.vdim_pad + i] = from_f32<T>(o[i] * ir * __ldg(g.head_norm + i) * silu_f32(to_f32(gate[i])));
+    }
+}
+
+// ------------------------------------------------------------------ chunks --
+constexpr int GC_THREADS = 128;
+constexpr float GLA_LOG2E = 1.4426950408889634f;
+
+// dS[d][v] = sum_t k_td e^{b_last,d - b_td} v_tv of one chunk and head.
+__host__ inline size_t gla_chunk_state_smem_bytes(int dim_pad, int vdim_pad) {
+    return (size_t)GLA_CHUNK * (2 * (dim_pad * 2 + 16) + (vdim_pad * 2 + 16));
+}
+__global__ void __launch_bounds__(GC_THREADS)
+gla_chunk_state_kernel(const GlaArgs<bf16> g)
+{
+    pdl_launch_dependents();
+    extern __shared__ __align__(16) uint8_t gc_smem[];
+    const int krow = g.dim_pad * 2 + 16, vrow = g.vdim_pad * 2 + 16;      // padded: eight rows of a fragment hit distinct banks
+    uint8_t* khi = gc_smem;                                // [64][dim_pad]
+    uint8_t* klo = khi + GLA_CHUNK * krow;
+    uint8_t* vs = klo + GLA_CHUNK * krow;                  // [64][vdim_pad]
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int h = blockIdx.y, r0 = blockIdx.x * GLA_CHUNK, n = min(GLA_CHUNK, g.rows - r0);
+    const int cols = g.heads * g.dim_pad;
+    pdl_wait_prior_grids();
+    const bf16* row0 = g.proj + (size_t)r0 * g.ld;
+    const float* b0 = g.decay + (size_t)r0 * cols + h * g.dim_pad;
+    for (int i = tid; i < GLA_CHUNK * (g.vdim_pad / 8); i += GC_THREADS) {
+        const int t = i / (g.vdim_pad / 8), c = i - t * (g.vdim_pad / 8);
+        ops::att_cp_async16(smem_u32(vs + t * vrow + c * 16), row0 + (size_t)(t < n ? t : 0) * g.ld + g.v_off() + h * g.vdim_pad + c * 8, t < n ? 16 : 0);
+    }
+    ops::att_cp_async_commit();
+    for (int i = tid; i < GLA_CHUNK * (g.dim_pad / 4); i += GC_THREADS) {
+        const int t = i / (g.dim_pad / 4), d = (i - t * (g.dim_pad / 4)) * 4;
+        uint2 hi = make_uint2(0, 0), lo = make_uint2(0, 0);
+        if (t < n) {
+            const float4 k = load4(row0 + (size_t)t * g.ld + g.k_off() + h * g.dim_pad + d);
+            const float4 b = load4(b0 + (size_t)t * cols + d), last = load4(b0 + (size_t)(n - 1) * cols + d);
+            split_bf16(k.x * ex2_approx((last.x - b.x) * GLA_LOG2E), k.y * ex2_approx((last.y - b.y) * GLA_LOG2E), hi.x, lo.x);
+            split_bf16(k.z * ex2_approx((last.z - b.z) * GLA_LOG2E), k.w * ex2_approx((last.w - b.w) * GLA_LOG2E), hi.y, lo.y);
+        }
+        *reinterpret_cast<uint2*>(khi + t * krow + d * 2) = hi;
+        *reinterpret_cast<uint2*>(klo + t * krow + d * 2) = lo;
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    float* out = g.chunk_state + ((size_t)blockIdx.x * g.heads + h) * g.dim_pad * g.vdim_pad;
+    // a warp's unit: 16 key channels x 64 value columns
+    const int mt = g.dim_pad / 16, nb = (g.vdim_pad + 63) / 64;
+    for (int u = warp; u < mt * nb; u += GC_THREADS / 32) {
+        const int m0 = (u % mt) * 16, v0 = (u / mt) * 64;
+        float acc[8][4];
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[j][e] = 0.0f;
+#pragma unroll
+        for (int kk = 0; kk < GLA_CHUNK / 16; ++kk) {
+            // A = K'^T (channels x tokens) out of rows of tokens: transposing loads
+            const uint32_t at = (uint32_t)((kk * 16 + (lane & 7) + (lane >> 4) * 8) * krow + (m0 + ((lane >> 3) & 1) * 8) * 2);
+            uint32_t ahi[4], alo[4];
+            ops::att_ldmatrix_x4_trans(ahi, smem_u32(khi) + at);
+            ops::att_ldmatrix_x4_trans(alo, smem_u32(klo) + at);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                if (v0 + j * 16 >= g.vdim_pad) continue;
+                uint32_t b[4];
+                ops::att_ldmatrix_x4_trans(b, smem_u32(vs) + (kk * 16 + (lane & 15)) * vrow + (v0 + j * 16 + (lane >> 4) * 8) * 2);
+                mma_bf16(acc[2 * j], ahi, b[0], b[1]);
+                mma_bf16(acc[2 * j + 1], ahi, b[2], b[3]);
+                mma_bf16(acc[2 * j], alo, b[0], b[1]);
+                mma_bf16(acc[2 * j + 1], alo, b[2], b[3]);
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const int v = v0 + j * 8 + (lane & 3) * 2, d = m0 + (lane >> 2);
+            if (v0 + j * 8 >= g.vdim_pad) continue;
+            *reinterpret_cast<float2*>(out + (size_t)d * g.vdim_pad + v) = make_float2(acc[j][0], acc[j][1]);
+            *reinterpret_cast<float2*>(out + (size_t)(d + 8) * g.vdim_pad + v) = make_float2(acc[j][2], acc[j][3]);
+        }
+    }
+}
+
+// chunk_state[n] becomes the state ahead of chunk n; the slot's state moves on to the end.  A thread per four columns.
+constexpr int GS_THREADS = 128, GS_AHEAD = 8;
+template <typename T>
+__global__ void __launch_bounds__(GS_THREADS)
+gla_scan_kernel(const GlaArgs<T> g)
+{
+    pdl_launch_dependents();
+    pdl_wait_prior_grids();
+    const int per_head = g.dim_pad * g.vdim_pad / 4, i = blockIdx.x * GS_THREADS + threadIdx.x;
+    if (i >= g.heads * per_head) return;
+    const int h = i / per_head, e = i - h * per_head, d = e * 4 / g.vdim_pad;
+    const int chunks = (g.rows + GLA_CHUNK - 1) / GLA_CHUNK, cols = g.heads * g.dim_pad;
+    float4* st = reinterpret_cast<float4*>(g.slot_state(h)) + e;
+    float4 s = g.meta[0] == 0 ? make_float4(0.f, 0.f, 0.f, 0.f) : *st;
+    float4* cs = reinterpret_cast<float4*>(g.chunk_state) + (size_t)h * per_head + e;
+    const size_t step = (size_t)g.heads * per_head;
+    const float* b = g.decay + h * g.dim_pad + d;
+    for (int n0 = 0; n0 < chunks; n0 += GS_AHEAD) {
+        float4 add[GS_AHEAD];
+        float a[GS_AHEAD];
+#pragma unroll
+        for (int j = 0; j < GS_AHEAD; ++j) {
+            const int n = n0 + j;
+            if (n < chunks) {
+                add[j] = cs[n * step];
+                a[j] = b[(size_t)(min(g.rows, (n + 1) * GLA_CHUNK) - 1) * cols];
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < GS_AHEAD; ++j) {
+            const int n = n0 + j;
+            if (n < chunks) {
+                cs[n * step] = s;
+                const float f = expf(a[j]);
+                s = make_float4(fmaf(s.x, f, add[j].x), fmaf(s.y, f, add[j].y), fmaf(s.z, f, add[j].z), fmaf(s.w, f, add[j].w));
+            }
+        }
+    }
+    *st = s;
+}
+
+// CTA = chunk and head; warp = 16 of its tokens.  DV: value columns the accumulators hold (>= vdim_pad).
+constexpr int GO_SROWS = 32;                               // state rows in shared memory at a time
+__host__ inline size_t gla_chunk_out_smem_bytes(int dim_pad, int vdim_pad) {
+    return (size_t)GLA_CHUNK * (dim_pad * 2 + 16 + vdim_pad * 2 + 16) + (size_t)GLA_CHUNK * (dim_pad * 4 + 32) +
+           (size_t)2 * GO_SROWS * (vdim_pad * 2 + 16) + 4 * 256 * sizeof(float);
+}
+template <int DV>
+__global__ void __launch_bounds__(GC_THREADS, 2)
+gla_chunk_out_kernel(const GlaArgs<bf16> g)
+{
+    pdl_launch_dependents();
+    extern __shared__ __align__(16) uint8_t gc_smem[];
+    const int krow = g.dim_pad * 2 + 16, vrow = g.vdim_pad * 2 + 16, brow = g.dim_pad + 8;
+    uint8_t* ks = gc_smem;                                 // [64][dim_pad]
+    uint8_t* vs = ks + GLA_CHUNK * krow;                   // [64][vdim_pad]
+    float* bs = reinterpret_cast<float*>(vs + GLA_CHUNK * vrow);      // [64][dim_pad] running sums, in powers of two
+    uint8_t* shi = reinterpret_cast<uint8_t*>(bs + GLA_CHUNK * brow); // [GO_SROWS][vdim_pad]
+    uint8_t* slo = shi + GO_SROWS * vrow;
+    float* pairs = reinterpret_cast<float*>(slo + GO_SROWS * vrow);   // [4 warps][16][16]
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int h = blockIdx.y, r0 = blockIdx.x * GLA_CHUNK, n = min(GLA_CHUNK, g.rows - r0);
+    const int cols = g.heads * g.dim_pad;
+    pdl_wait_prior_grids();
+    const bf16* row0 = g.proj + (size_t)r0 * g.ld;
+    const int kp = g.dim_pad / 8, vp = g.vdim_pad / 8;
+    for (int i = tid; i < GLA_CHUNK * kp; i += GC_THREADS) {
+        const int t = i / kp, c = i - t * kp;
+        ops::att_cp_async16(smem_u32(ks + t * krow + c * 16), row0 + (size_t)(t < n ? t : 0) * g.ld + g.k_off() + h * g.dim_pad + c * 8, t < n ? 16 : 0);
+    }
+    for (int i = tid; i < GLA_CHUNK * vp; i += GC_THREADS) {
+        const int t = i / vp, c = i - t * vp;
+        ops::att_cp_async16(smem_u32(vs + t * vrow + c * 16), row0 + (size_t)(t < n ? t : 0) * g.ld + g.v_off() + h * g.vdim_pad + c * 8, t < n ? 16 : 0);
+    }
+    ops::att_cp_async_commit();
+    // rows past the end repeat the last one: their weights are never used
+    bool steep = false;
+    for (int i = tid; i < GLA_CHUNK * (g.dim_pad / 4); i += GC_THREADS) {
+        const int t = i / (g.dim_pad / 4), d = (i - t * (g.dim_pad / 4)) * 4;
+        const float* at = g.decay + (size_t)(r0 + min(t, n - 1)) * cols + h * g.dim_pad + d;
+        const float4 b = load4(at);
+        if (t > 0 && t < n) {
+            const float4 p = load4(at - cols);
+            steep = steep || fminf(fminf(b.x - p.x, b.y - p.y), fminf(b.z - p.z, b.w - p.w)) < GLA_STEP_FLOOR;
+        }
+        *reinterpret_cast<float4*>(bs + t * brow + d) = make_float4(b.x * GLA_LOG2E, b.y * GLA_LOG2E, b.z * GLA_LOG2E, b.w * GLA_LOG2E);
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    steep = __syncthreads_or(steep);
+
+    const int t_lo = warp * 16 + (lane >> 2), t_hi = t_lo + 8, d_in = (lane & 3) * 2;
+    const bf16* q_lo = row0 + (size_t)min(t_lo, n - 1) * g.ld + h * g.dim_pad;
+    const bf16* q_hi = row0 + (size_t)min(t_hi, n - 1) * g.ld + h * g.dim_pad;
+    auto pair_f32 = [](uint32_t w) { return make_float2(__uint_as_float(w << 16), __uint_as_float(w & 0xffff0000u)); };
+    // the warp's queries at channels d, d + 1 of rows t_lo or t_hi, times 2^(b_t - ref)
+    auto q_pair = [&](const bf16* q, int t, int d, float2 ref, uint32_t& hi, uint32_t& lo) {
+        const float2 x = pair_f32(*reinterpret_cast<const uint32_t*>(q + d));
+        const float2 b = *reinterpret_cast<const float2*>(bs + t * brow + d);
+        split_bf16(x.x * g.q_scale * ex2_approx(b.x - ref.x), x.y * g.q_scale * ex2_approx(b.y - ref.y), hi, lo);
+    };
+    auto q_frag = [&](int d0, float2 ref0, float2 ref8, uint32_t (&hi)[4], uint32_t (&lo)[4]) {
+        q_pair(q_lo, t_lo, d0 + d_in, ref0, hi[0], lo[0]);
+        q_pair(q_hi, t_hi, d0 + d_in, ref0, hi[1], lo[1]);
+        q_pair(q_lo, t_lo, d0 + d_in + 8, ref8, hi[2], lo[2]);
+        q_pair(q_hi, t_hi, d0 + d_in + 8, ref8, hi[3], lo[3]);
+    };
+    auto k_pair = [&](int s, int d, float2 ref, uint32_t& hi, uint32_t& lo) {
+        const float2 x = pair_f32(*reinterpret_cast<const uint32_t*>(ks + s * krow + d * 2));
+        const float2 b = *reinterpret_cast<const float2*>(bs + s * brow + d);
+        split_bf16(x.x * ex2_approx(ref.x - b.x), x.y * ex2_approx(ref.y - b.y), hi, lo);
+    };
+    // scores of the warp's 16 tokens against 16 tokens from s0, exponents against row `ref`
+    float a[4][2][4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) a[j][i][e] = 0.0f;
+    auto against = [&](int d0, const uint32_t (&qh)[4], const uint32_t (&ql)[4], int s0, float2 ref0, float2 ref8, float (&acc)[2][4]) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int s = s0 + i * 8 + (lane >> 2);
+            uint32_t h0, l0, h1, l1;
+            k_pair(s, d0 + d_in, ref0, h0, l0);
+            k_pair(s, d0 + d_in + 8, ref8, h1, l1);
+            mma_bf16(acc[i], qh, h0, h1);
+            mma_bf16(acc[i], ql, h0, h1);
+            mma_bf16(acc[i], qh, l0, l1);
+        }
+    };
+    auto ref_at = [&](int t, int d) { return *reinterpret_cast<const float2*>(bs + t * brow + d); };
+    for (int d0 = 0; d0 < g.dim_pad; d0 += 16) {
+        uint32_t qh[4], ql[4];
+        if (warp > 0) {
+            const int t = warp * 16 - 1;
+            const float2 r0_ = ref_at(t, d0 + d_in), r8_ = ref_at(t, d0 + d_in + 8);
+            q_frag(d0, r0_, r8_, qh, ql);
+#pragma unroll
+            for (int j = 0; j < 3; ++j)
+                if (j < warp) against(d0, qh, ql, j * 16, r0_, r8_, a[j]);
+        }
+        if (!steep) {
+            const int t = warp * 16 + 7;
+            const float2 r0_ = ref_at(t, d0 + d_in), r8_ = ref_at(t, d0 + d_in + 8);
+            q_frag(d0, r0_, r8_, qh, ql);
+            against(d0, qh, ql, warp * 16, r0_, r8_, a[3]);
+        }
+    }
+    if (steep) {                                           // the block's own pairs one by one
+        float* mine = pairs + warp * 256;
+        for (int i = 0; i < 16; ++i)
+            for (int j = 0; j <= i; ++j) {
+                const int t = warp * 16 + i, s = warp * 16 + j;
+                float sum = 0.0f;
+                for (int d = lane; d < g.dim_pad; d += 32)
+                    sum = fmaf(to_f32(row0[(size_t)min(t, n - 1) * g.ld + h * g.dim_pad + d]) * g.q_scale *
+                                   to_f32(reinterpret_cast<const bf16*>(ks + s * krow)[d]),
+                               ex2_approx(bs[t * brow + d] - bs[s * brow + d]), sum);
+                sum = ops::warp_sum(sum);
+                if (lane == 0) mine[i * 16 + j] = sum;
+            }
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int t = (lane >> 2) + (e >> 1) * 8, s = i * 8 + d_in + (e & 1);
+                a[3][i][e] = s <= t ? mine[t * 16 + s] : 0.0f;
+            }
+    }
+    // ---- o = scores V + (q 2^b) S ----
+    float o[DV / 8][4];
+#pragma unroll
+    for (int j = 0; j < DV / 8; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[j][e] = 0.0f;
+    auto times_v = [&](float (&x)[2][4], int s0) {
+        uint32_t hi[4], lo[4];
+        split_bf16(x[0][0], x[0][1], hi[0], lo[0]);
+        split_bf16(x[0][2], x[0][3], hi[1], lo[1]);
+        split_bf16(x[1][0], x[1][1], hi[2], lo[2]);
+        split_bf16(x[1][2], x[1][3], hi[3], lo[3]);
+#pragma unroll
+        for (int j = 0; j < DV / 16; ++j) {
+            if (j * 16 >= g.vdim_pad) continue;
+            uint32_t b[4];
+            ops::att_ldmatrix_x4_trans(b, smem_u32(vs) + (s0 + (lane & 15)) * vrow + (j * 16 + (lane >> 4) * 8) * 2);
+            mma_bf16(o[2 * j], hi, b[0], b[1]);
+            mma_bf16(o[2 * j + 1], hi, b[2], b[3]);
+            mma_bf16(o[2 * j], lo, b[0], b[1]);
+            mma_bf16(o[2 * j + 1], lo, b[2], b[3]);
+        }
+    };
+#pragma unroll
+    for (int j = 0; j < 3; ++j)
+        if (j < warp) times_v(a[j], j * 16);
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int t = (lane >> 2) + (e >> 1) * 8, s = i * 8 + d_in + (e & 1);
+            if (s > t) a[3][i][e] = 0.0f;
+        }
+    times_v(a[3], warp * 16);
+    const float* st = g.chunk_state + ((size_t)blockIdx.x * g.heads + h) * g.dim_pad * g.vdim_pad;
+    const float2 zero2 = make_float2(0.0f, 0.0f);
+    for (int d0 = 0; d0 < g.dim_pad; d0 += GO_SROWS) {
+        const int dn = min(GO_SROWS, g.dim_pad - d0);
+        __syncthreads();                                   // the rows before have been used
+        for (int i = tid; i < dn * (g.vdim_pad / 4); i += GC_THREADS) {
+            const int d = i / (g.vdim_pad / 4), v = (i - d * (g.vdim_pad / 4)) * 4;
+            const float4 x = load4(st + (size_t)(d0 + d) * g.vdim_pad + v);
+            uint2 hi, lo;
+            split_bf16(x.x, x.y, hi.x, lo.x);
+            split_bf16(x.z, x.w, hi.y, lo.y);
+            *reinterpret_cast<uint2*>(shi + d * vrow + v * 2) = hi;
+            *reinterpret_cast<uint2*>(slo + d * vrow + v * 2) = lo;
+        }
+        __syncthreads();
+        for (int dk = 0; dk < dn; dk += 16) {
+            uint32_t qh[4], ql[4];
+            q_frag(d0 + dk, zero2, zero2, qh, ql);
+#pragma unroll
+            for (int j = 0; j < DV / 16; ++j) {
+                if (j * 16 >= g.vdim_pad) continue;
+                const uint32_t at = (uint32_t)((dk + (lane & 15)) * vrow + (j * 16 + (lane >> 4) * 8) * 2);
+                uint32_t bh[4], bl[4];
+                ops::att_ldmatrix_x4_trans(bh, smem_u32(shi) + at);
+                ops::att_ldmatrix_x4_trans(bl, smem_u32(slo) + at);
+                mma_bf16(o[2 * j], qh, bh[0], bh[1]);
+                mma_bf16(o[2 * j + 1], qh, bh[2], bh[3]);
+                mma_bf16(o[2 * j], ql, bh[0], bh[1]);
+                mma_bf16(o[2 * j + 1], ql, bh[2], bh[3]);
+                mma_bf16(o[2 * j], qh, bl[0], bl[1]);
+                mma_bf16(o[2 * j + 1], qh, bl[2], bl[3]);
+            }
+        }
+    }
+    // ---- norm over the head's columns, gate, store ----
+    float ss[2] = {0.0f, 0.0f};
+#pragma unroll
+    for (int j = 0; j < DV / 8; ++j) {
+        ss[0] = fmaf(o[j][0], o[j][0], fmaf(o[j][1], o[j][1], ss[0]));
+        ss[1] = fmaf(o[j][2], o[j][2], fmaf(o[j][3], o[j][3], ss[1]));
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], 1);
+        ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], 2);
+        const int t = i == 0 ? t_lo : t_hi;
+        if (t >= n) continue;
+        const float ir = inv_rms(ss[i], g.vdim, g.eps);
+        const bf16* gate = row0 + (size_t)t * g.ld + g.gate_off() + h * g.vdim_pad;
+        bf16* out = g.out + ((size_t)(r0 + t) * g.heads + h) * g.vdim_pad;
+#pragma unroll
+        for (int j = 0; j < DV / 8; ++j) {
+            const int v = j * 8 + d_in;
+            if (j * 8 >= g.vdim_pad) continue;
+            const float2 w = *reinterpret_cast<const float2*>(g.head_norm + v);
+            const float2 z = pair_f32(*reinterpret_cast<const uint32_t*>(gate + v));
+            *reinterpret_cast<__nv_bfloat162*>(out + v) =
+                __floats2bfloat162_rn(o[j][2 * i] * ir * w.x * silu_f32(z.x), o[j][2 * i + 1] * ir * w.y * silu_f32(z.y));
+        }
+    }
+}
+
+// ------------------------------------------------------------------ decode --
+// One token.  A cluster of CTAs per head, each with a share of the value columns: decays, the state's share moved on in
+// place, the share of o; the sums of squares of the cluster make the norm.
+constexpr int GX_THREADS = 256, GX_MAX_SPLITS = 8;
+template <typename T>
+struct GlaDecodeArgs {
+    const float* proj;          // f32: q | k | v | gate | low-rank
+    float* out;                 // f32 [heads * vdim_pad]
+    float* state;
+    const T* w_decay;
+    const float* decay_bias;
+    const float* head_norm;
+    const int* meta;
+    int heads, dim_pad, vdim, vdim_pad, rank_pad;
+    float inv_tau, q_scale, eps;
+};
+__host__ __device__ inline int gla_decode_share(int vdim_pad, int splits) { return ((vdim_pad / 4 + splits - 1) / splits) * 4; }
+__host__ inline size_t gla_decode_smem_bytes(int dim_pad, int vdim_pad, int splits) {
+    const int quads = gla_decode_share(vdim_pad, splits) / 4;
+    const int groups = GX_THREADS / quads < 1 ? 1 : GX_THREADS / quads;
+    return sizeof(float) * ((size_t)3 * dim_pad + (size_t)groups * quads * 4);
+}
+template <typename T>
+__global__ void __launch_bounds__(GX_THREADS)
+gla_decode_kernel(const GlaDecodeArgs<T> g)
+{
+    using V = Vec<T>;
+    pdl_launch_dependents();
+    extern __shared__ __align__(16) float gx_smem[];
+    __shared__ float red[32];
+    __shared__ float recv[GX_MAX_SPLITS];
+    const int splits = gridDim.x, rank = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+    const int share = gla_decode_share(g.vdim_pad, splits), quads = share / 4;
+    const int groups = GX_THREADS / quads < 1 ? 1 : GX_THREADS / quads;
+    float* qs = gx_smem;                                   // [dim_pad]
+    float* ks = qs + g.dim_pad;
+    float* as = ks + g.dim_pad;
+    float* part = as + g.dim_pad;                          // [groups][share]
+    const int kd = g.heads * g.dim_pad, vd = g.heads * g.vdim_pad;
+    asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");
+    // weights do not depend on the kernel before
+    constexpr int WV = 2;                                  // vectors of the decay's weights held ahead
+    uint4 wv[WV];
+    const float bias = tid < g.dim_pad ? __ldg(g.decay_bias + h * g.dim_pad + tid) : 0.0f;
+#pragma unroll
+    for (int i = 0; i < WV; ++i)
+        wv[i] = tid < g.dim_pad && i * V::N < g.rank_pad ? __ldg(reinterpret_cast<const uint4*>(g.w_decay + (size_t)(h * g.dim_pad + tid) * g.rank_pad) + i)
+                                                         : make_uint4(0, 0, 0, 0);
+    pdl_wait_prior_grids();
+    const float* low = g.proj + 2 * kd + 2 * vd;
+    for (int d = tid; d < g.dim_pad; d += GX_THREADS) {
+        qs[d] = g.proj[h * g.dim_pad + d] * g.q_scale;
+        ks[d] = g.proj[kd + h * g.dim_pad + d];
+        float z = d == tid ? bias : __ldg(g.decay_bias + h * g.dim_pad + d);
+        for (int i = 0; i * V::N < g.rank_pad; ++i) {
+            float w[V::N];
+            V::unpack(d == tid && i == 0 ? wv[0] : d == tid && i == 1 ? wv[1]
+                          : __ldg(reinterpret_cast<const uint4*>(g.w_decay + (size_t)(h * g.dim_pad + d) * g.rank_pad) + i), w);
+#pragma unroll
+            for (int e = 0; e < V::N; e += 4) {
+                const float4 a = *reinterpret_cast<const float4*>(low + i * V::N + e);
+                z = fmaf(w[e], a.x, fmaf(w[e + 1], a.y, fmaf(w[e + 2], a.z, fmaf(w[e + 3], a.w, z))));
+            }
+        }
+        as[d] = expf(log_sigmoid_f32(z) * g.inv_tau);
+    }
+    const bool fresh = g.meta[0] == 0;
+    float* st = g.state + ((size_t)g.meta[1] * g.heads + h) * g.dim_pad * g.vdim_pad;
+    __syncthreads();
+    const int c0 = rank * share, grp = tid / quads;
+    for (int qi = tid % quads; qi < quads; qi += GX_THREADS) {            // one round unless a share has more quads than threads
+        const int c = c0 + qi * 4;
+        float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c < g.vdim_pad && grp < groups) {
+            const float4 v = *reinterpret_cast<const float4*>(g.proj + 2 * kd + h * g.vdim_pad + c);
+#pragma unroll 4
+            for (int d = grp; d < g.dim_pad; d += groups) {
+                float4* at = reinterpret_cast<float4*>(st + (size_t)d * g.vdim_pad + c);
+                const float4 s = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *at;
+                const float a = as[d], k = ks[d], q = qs[d];
+                const float4 x = make_float4(fmaf(s.x, a, k * v.x), fmaf(s.y, a, k * v.y), fmaf(s.z, a, k * v.z), fmaf(s.w, a, k * v.w));
+                *at = x;
+                o.x = fmaf(x.x, q, o.x); o.y = fmaf(x.y, q, o.y); o.z = fmaf(x.z, q, o.z); o.w = fmaf(x.w, q, o.w);
+            }
+        }
+        if (grp < groups) *reinterpret_cast<float4*>(part + (size_t)grp * share + qi * 4) = o;
+    }
+    __syncthreads();
+    float ss = 0.0f;
+    for (int i = tid; i < share; i += GX_THREADS) {
+        float o = 0.0f;
+        for (int k = 0; k < groups; ++k) o += part[(size_t)k * share + i];
+        part[i] = o;                                       // column i is this thread's alone
+        if (c0 + i < g.vdim_pad) ss = fmaf(o, o, ss);
+    }
+    ss = group_sum(ss, red, GX_THREADS, 1);
+    asm volatile("barrier.cluster.wait.aligned;" ::: "memory");
+    if (tid < splits) st_cluster_f32(mapa_shared(smem_u32(recv + rank), tid), ss);
+    cluster_sync_all();
+    float all = 0.0f;
+    for (int s = 0; s < splits; ++s) all += recv[s];
+    const float ir = inv_rms(all, g.vdim, g.eps);
+    for (int i = tid; i < share; i += GX_THREADS) {
+        const int c = c0 + i;
+        if (c >= g.vdim_pad) continue;
+        g.out[h * g.vdim_pad + c] = part[i] * ir * __ldg(g.head_norm + c) * silu_f32(g.proj[2 * kd + vd + h * g.vdim_pad + c]);
+    }
+}
+
+}  // namespace dense
+}  // namespace twm

@@ -10,6 +10,23 @@ namespace dense {
 
 constexpr int ROW_THREADS = 256;
 
+// Outputs of the chosen experts: a token's sublayer output is the sum over its `top` slots of weight * row.
+template <typename T>
+struct RoutedOutput {
+    const T* rows;              // [tokens * top][wp], grouped by expert; null = the sublayer was not routed
+    const int* row;             // [tokens][top]: a slot's row
+    const float* weight;        // [tokens][top]
+    int top;
+};
+
+// four consecutive elements as floats
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const bf16* p) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16),
+                       __uint_as_float(v.y & 0xffff0000u));
+}
+
 // One row's residual value, x_in + y * inv_rms(y) * y_norm (or the embedding), element by element.
 template <typename T>
 struct ResidualSource {
@@ -19,15 +36,33 @@ struct ResidualSource {
     const float* x_in;          // [rows][wp]
     const float* y;             // [rows][wp] or null
     const float* y_norm;        // [wp] or null (y joins as it is)
-    float eps;
+    const float* step;          // [wp]: added to every row, or null
+    RoutedOutput<T> routed;     // instead of y
+    float eps, embed_scale;
     int width, wp;
+
+    __device__ __forceinline__ bool has_y() const { return y != nullptr || routed.rows != nullptr; }
+    // four consecutive elements of what joins row r
+    __device__ __forceinline__ float4 y_at(int r, int i4) const {
+        if (y != nullptr) return reinterpret_cast<const float4*>(y + (size_t)r * wp)[i4];
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        const int* at = routed.row + (size_t)r * routed.top;
+        const float* w = routed.weight + (size_t)r * routed.top;
+#pragma unroll 4
+        for (int s = 0; s < routed.top; ++s) {
+            const float4 t = load4(routed.rows + (size_t)at[s] * wp + i4 * 4);
+            const float ws = w[s];
+            v.x = fmaf(t.x, ws, v.x); v.y = fmaf(t.y, ws, v.y); v.z = fmaf(t.z, ws, v.z); v.w = fmaf(t.w, ws, v.w);
+        }
+        return v;
+    }
 
     // four consecutive elements of row r; ir = inverse RMS of y's row
     __device__ __forceinline__ float4 at(int r, int p, int token, int i4, float ir) const {
         float4 v;
         if (tokens != nullptr) {
             const T* e = embed + (size_t)token * wp + i4 * 4;
-            v = make_float4(to_f32(e[0]), to_f32(e[1]), to_f32(e[2]), to_f32(e[3]));
+            v = make_float4(to_f32(e[0]) * embed_scale, to_f32(e[1]) * embed_scale, to_f32(e[2]) * embed_scale, to_f32(e[3]) * embed_scale);
             if (pos_embed != nullptr) {
                 const T* pe = pos_embed + (size_t)p * wp + i4 * 4;
                 v.x += to_f32(pe[0]); v.y += to_f32(pe[1]); v.z += to_f32(pe[2]); v.w += to_f32(pe[3]);
@@ -35,20 +70,23 @@ struct ResidualSource {
         } else {
             v = reinterpret_cast<const float4*>(x_in + (size_t)r * wp)[i4];
         }
-        if (y != nullptr) {
-            const float4 t = reinterpret_cast<const float4*>(y + (size_t)r * wp)[i4];
+        if (has_y()) {
+            const float4 t = y_at(r, i4);
             float4 g = make_float4(1.f, 1.f, 1.f, 1.f);
             if (y_norm != nullptr) g = __ldg(reinterpret_cast<const float4*>(y_norm) + i4);
             v.x += t.x * ir * g.x; v.y += t.y * ir * g.y; v.z += t.z * ir * g.z; v.w += t.w * ir * g.w;
+        }
+        if (step != nullptr) {
+            const float4 t = __ldg(reinterpret_cast<const float4*>(step) + i4);
+            v.x += t.x; v.y += t.y; v.z += t.z; v.w += t.w;
         }
         return v;
     }
     // inverse RMS of y's row (1 without a norm); all `threads` threads of the barrier take part
     __device__ __forceinline__ float row_inv_rms(int r, float* red, int threads, int bar) const {
-        if (y == nullptr || y_norm == nullptr) return 1.0f;
+        if (!has_y() || y_norm == nullptr) return 1.0f;
         float ss = 0.0f;
-        const float4* yr = reinterpret_cast<const float4*>(y + (size_t)r * wp);
-        for (int i = threadIdx.x; i < (wp >> 2); i += threads) ss += ops::sumsq4(yr[i]);
+        for (int i = threadIdx.x; i < (wp >> 2); i += threads) ss += ops::sumsq4(y_at(r, i));
         return inv_rms(group_sum(ss, red, threads, bar), width, eps);
     }
 };
@@ -66,28 +104,26 @@ __device__ __forceinline__ void store4<bf16>(bf16* dst, const float4 v) {
     *reinterpret_cast<uint2*>(dst) = o;
 }
 
-// four consecutive elements as floats
-__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 load4(const bf16* p) {
-    const uint2 v = *reinterpret_cast<const uint2*>(p);
-    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16),
-                       __uint_as_float(v.y & 0xffff0000u));
-}
-
 // x + (before - x) * mix
 __device__ __forceinline__ float4 shift4(const float4 x, const float4 before, const float4 mix) {
     return make_float4(fmaf(before.x - x.x, mix.x, x.x), fmaf(before.y - x.y, mix.y, x.y), fmaf(before.z - x.z, mix.z, x.z),
                        fmaf(before.w - x.w, mix.w, x.w));
 }
 
-// x_out = residual row; a = T(x_out), or T(token shift of x_out).  A CTA walks `rows_per_cta` consecutive rows and
+__device__ __forceinline__ float4 scale4(const float4 x, float s, const float4 g) {
+    return make_float4(x.x * s * g.x, x.y * s * g.y, x.z * s * g.z, x.w * s * g.w);
+}
+
+// x_out = residual row; a = T(x_out), or T(token shift of x_out), or T(rms_norm(x_out) * pre_norm).  clear: words set to
+// zero on the way (the expert counts of the routing that follows).  A CTA walks `rows_per_cta` consecutive rows and
 // keeps the row before; its first row's predecessor is computed again (or comes from the state).  PER > 0: a
 // thread's share of a row is PER vectors, held in registers, every load issued before the first use; PER = 0: rows
 // of any length, in shared memory.
 template <typename T, int PER>
 __global__ void __launch_bounds__(ROW_THREADS)
 residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __restrict__ a, const float* __restrict__ shift,
-                     const float* __restrict__ shift_state, const int* __restrict__ meta, int rows, int rows_per_cta)
+                     const float* __restrict__ shift_state, const float* __restrict__ pre_norm, const int* __restrict__ meta, int rows,
+                     int rows_per_cta, int* __restrict__ clear, int n_clear)
 {
     pdl_launch_dependents();
     extern __shared__ __align__(16) float row_smem[];       // PER = 0: [wp], the residual row before
@@ -96,6 +132,8 @@ residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __rest
     const int wp = src.wp, nvec = wp >> 2;
     const int r0 = blockIdx.x * rows_per_cta, r1 = min(rows, r0 + rows_per_cta);
     const int pos0 = meta[0];
+    if (blockIdx.x == 0)
+        for (int i = threadIdx.x; i < n_clear; i += ROW_THREADS) clear[i] = 0;
     const float* st = shift != nullptr && r0 == 0 && pos0 > 0
                           ? shift_state + ((size_t)meta[1] * 2 + ((pos0 - 1) & 1)) * wp : nullptr;
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -111,19 +149,21 @@ residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __rest
             const int tok = src.tokens != nullptr ? src.tokens[r] : 0;
             ResidualSource<T> plain = src;                  // the row without what joins it
             plain.y = nullptr;
+            plain.routed.rows = nullptr;
 #pragma unroll
             for (int j = 0; j < PER; ++j) {
                 const int i = threadIdx.x + j * ROW_THREADS;
-                y[j] = src.y != nullptr && i < nvec ? reinterpret_cast<const float4*>(src.y + (size_t)r * wp)[i] : zero;
+                y[j] = src.has_y() && i < nvec ? src.y_at(r, i) : zero;
                 x[j] = i < nvec ? plain.at(r, pos0 + r, tok, i, 1.0f) : zero;
             }
             float ir = 1.0f;
-            if (src.y != nullptr && src.y_norm != nullptr) {
+            if (src.has_y() && src.y_norm != nullptr) {
                 float ss = 0.0f;
 #pragma unroll
                 for (int j = 0; j < PER; ++j) ss += ops::sumsq4(y[j]);
                 ir = inv_rms(group_sum(ss, red, ROW_THREADS, 1), src.width, src.eps);
             }
+            float xs = 0.0f, pr = 1.0f;
 #pragma unroll
             for (int j = 0; j < PER; ++j) {
                 const int i = threadIdx.x + j * ROW_THREADS;
@@ -131,10 +171,18 @@ residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __rest
                 float4 n = make_float4(1.f, 1.f, 1.f, 1.f);
                 if (src.y_norm != nullptr) n = __ldg(reinterpret_cast<const float4*>(src.y_norm) + i);
                 x[j].x += y[j].x * ir * n.x; x[j].y += y[j].y * ir * n.y; x[j].z += y[j].z * ir * n.z; x[j].w += y[j].w * ir * n.w;
+                xs += ops::sumsq4(x[j]);
+            }
+            if (pre_norm != nullptr) pr = inv_rms(group_sum(xs, red, ROW_THREADS, 1), src.width, src.eps);
+#pragma unroll
+            for (int j = 0; j < PER; ++j) {
+                const int i = threadIdx.x + j * ROW_THREADS;
+                if (i >= nvec) continue;
                 if (r >= r0) {
                     reinterpret_cast<float4*>(x_out + (size_t)r * wp)[i] = x[j];
                     float4 h = x[j];
                     if (shift != nullptr) h = shift4(x[j], before[j], __ldg(reinterpret_cast<const float4*>(shift) + i));
+                    if (pre_norm != nullptr) h = scale4(x[j], pr, __ldg(reinterpret_cast<const float4*>(pre_norm) + i));
                     if (a != nullptr) store4<T>(a + (size_t)r * wp + i * 4, h);
                 }
                 before[j] = x[j];
@@ -156,6 +204,12 @@ residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __rest
         for (int r = r0; r < r1; ++r) {
             const int tok = src.tokens != nullptr ? src.tokens[r] : 0;
             const float ir = src.row_inv_rms(r, red, ROW_THREADS, 1);
+            float pr = 1.0f;
+            if (pre_norm != nullptr) {
+                float xs = 0.0f;
+                for (int i = threadIdx.x; i < nvec; i += ROW_THREADS) xs += ops::sumsq4(src.at(r, pos0 + r, tok, i, ir));
+                pr = inv_rms(group_sum(xs, red, ROW_THREADS, 1), src.width, src.eps);
+            }
             // every thread reads and replaces its own elements of row_smem: no barrier needed between rows
             for (int i = threadIdx.x; i < nvec; i += ROW_THREADS) {
                 const float4 x = src.at(r, pos0 + r, tok, i, ir);
@@ -166,6 +220,7 @@ residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __rest
                     h = shift4(x, *before, __ldg(reinterpret_cast<const float4*>(shift) + i));
                     *before = x;
                 }
+                if (pre_norm != nullptr) h = scale4(x, pr, __ldg(reinterpret_cast<const float4*>(pre_norm) + i));
                 if (a != nullptr) store4<T>(a + (size_t)r * wp + i * 4, h);
             }
         }

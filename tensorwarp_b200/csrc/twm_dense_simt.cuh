@@ -18,8 +18,8 @@ gemm_simt_kernel(const T* __restrict__ a, int lda, const T* __restrict__ w, int 
 {
     constexpr int NB = EPI == TWM_EPI_GELU_GLU ? 2 : 1;
     pdl_launch_dependents();
-    __shared__ float as[SK][ST + 4];
-    __shared__ float bs[NB][SK][ST + 4];
+    __shared__ __align__(16) float as[SK][ST + 4];
+    __shared__ __align__(16) float bs[NB][SK][ST + 4];
     pdl_wait_prior_grids();
     const int m0 = blockIdx.y * ST, n0 = blockIdx.x * ST;
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;

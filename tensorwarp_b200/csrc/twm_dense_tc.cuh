@@ -7,9 +7,12 @@
 // warp 5 issues tcgen05.mma (128 x BN x 16), warps 0-3 read a finished accumulator back and store it
 // while the next tile accumulates into the other one.  Weights are constants: the first ring-full of
 // them is on its way before the preceding kernel has finished; the activations follow after it.
+//
+// GROUPED: the rows are grouped by expert (offsets[e] .. offsets[e + 1], known on the device only) and each group has a
+// weight matrix of its own.  A tile belongs to one expert; it may load rows of the next one, which are not stored.
 #pragma once
 
-#include "twm_dense_common.cuh"
+#include "twm_dense_moe.cuh"
 #include "twm_gemm_tc.cuh"
 #include "twm_gemm_tcw.cuh"
 
@@ -33,6 +36,8 @@ struct TcArgs {
     void* c;
     int ldc, M, N, K;               // gated: N output columns, 2 N weight rows
     int m_tiles, n_tiles;
+    const int* offsets;             // grouped: [experts + 1]
+    int experts;
     alignas(64) CUtensorMap a_map;  // bf16 [M][K], box 64 x 128
     alignas(64) CUtensorMap w_map;  // bf16 [rows][K], box 64 x BN (gated: 64 x BN/2)
 };
@@ -78,7 +83,7 @@ __device__ __forceinline__ void tc_store16(void* c, size_t row_off, int n, int N
     }
 }
 
-template <int BN, int EPI>
+template <int BN, int EPI, bool GROUPED>
 __global__ void __launch_bounds__(TC_THREADS, 1)
 gemm_tc_kernel(const __grid_constant__ TcArgs g)
 {
@@ -93,8 +98,9 @@ gemm_tc_kernel(const __grid_constant__ TcArgs g)
     __shared__ int abort_s;
     volatile int* abort_flag = &abort_s;
 
+    __shared__ int pre[GROUPED ? MOE_MAX_EXPERTS + 1 : 1];       // grouped: the tiles ahead of each expert's
+
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int tiles = g.m_tiles * g.n_tiles;
     const int k_steps = (g.K + TC_BK - 1) / TC_BK;
 
     if (tid == 0) {
@@ -109,42 +115,66 @@ gemm_tc_kernel(const __grid_constant__ TcArgs g)
         tc::tmem_alloc(&tmem_s, C::TMEM_COLS);
         tc::tc_fence_before();
     }
+    if (GROUPED && warp == 0) {
+        pdl_wait_prior_grids();
+        warp_prefix([&](int e) { return (g.offsets[e + 1] - g.offsets[e] + TC_BM - 1) / TC_BM * g.n_tiles; }, g.experts, pre, lane);
+    }
     __syncthreads();
     tc::tc_fence_after();
     pdl_launch_dependents();
     const uint32_t tmem = tmem_s;
+    const int tiles = GROUPED ? pre[g.experts] : g.m_tiles * g.n_tiles;
+    // tile t: its first row, the end of its rows, its column tile and the first row of its weight matrix
+    struct Tile { int row, end, n, w0; };
+    auto tile_at = [&](int t) {
+        Tile x;
+        if (GROUPED) {
+            const int e = prefix_find(pre, g.experts, t), mt = (pre[e + 1] - pre[e]) / g.n_tiles, i = t - pre[e];
+            x.n = i / mt;
+            x.row = g.offsets[e] + (i - x.n * mt) * TC_BM;
+            x.end = g.offsets[e + 1];
+            x.w0 = e * g.N;
+        } else {
+            int m;
+            tc_tile(t, g.m_tiles, g.n_tiles, m, x.n);
+            x.row = m * TC_BM;
+            x.end = g.M;
+            x.w0 = 0;
+        }
+        return x;
+    };
 
     if (warp == TC_WARP_TMA) {
         if (elect_one()) {
-            auto load_w = [&](int slot, int n, int kk) {
+            auto load_w = [&](int slot, const Tile& x, int kk) {
                 uint8_t* dst = ring + (size_t)slot * C::STAGE_BYTES + TC_A_BYTES;
                 mbar_arrive_expect_tx(&full[slot], (uint32_t)C::STAGE_BYTES);
-                tma_load_2d(dst, &g.w_map, kk * TC_BK, n * OUT, &full[slot]);
-                if (GATED) tma_load_2d(dst + C::B_BYTES / 2, &g.w_map, kk * TC_BK, g.N + n * OUT, &full[slot]);
+                tma_load_2d(dst, &g.w_map, kk * TC_BK, x.w0 + x.n * OUT, &full[slot]);
+                if (GATED) tma_load_2d(dst + C::B_BYTES / 2, &g.w_map, kk * TC_BK, g.N + x.n * OUT, &full[slot]);
             };
-            auto load_a = [&](int slot, int m, int kk) {
-                tma_load_2d(ring + (size_t)slot * C::STAGE_BYTES, &g.a_map, kk * TC_BK, m * TC_BM, &full[slot]);
+            auto load_a = [&](int slot, const Tile& x, int kk) {
+                tma_load_2d(ring + (size_t)slot * C::STAGE_BYTES, &g.a_map, kk * TC_BK, x.row, &full[slot]);
             };
-            int m, n, it = 0;
+            int it = 0;
             bool ok = true;
             // the first tile's first stages: weights before the wait for the preceding kernel, activations after it
             const int early = min(STAGES, k_steps);
             if ((int)blockIdx.x < tiles) {
-                tc_tile(blockIdx.x, g.m_tiles, g.n_tiles, m, n);
-                for (int kk = 0; kk < early; ++kk) load_w(kk, n, kk);
+                const Tile x = tile_at(blockIdx.x);
+                for (int kk = 0; kk < early; ++kk) load_w(kk, x, kk);
                 pdl_wait_prior_grids();
-                for (int kk = 0; kk < early; ++kk) load_a(kk, m, kk);
+                for (int kk = 0; kk < early; ++kk) load_a(kk, x, kk);
             } else {
                 pdl_wait_prior_grids();
             }
             for (int t = blockIdx.x; t < tiles && ok; t += gridDim.x) {
-                tc_tile(t, g.m_tiles, g.n_tiles, m, n);
+                const Tile x = tile_at(t);
                 for (int kk = 0; kk < k_steps; ++kk, ++it) {
                     if (it < early) continue;
                     const int slot = it % STAGES;
                     if (it >= STAGES && !mbar_wait_bounded(&empty[slot], ((it / STAGES) - 1) & 1, abort_flag)) { ok = false; break; }
-                    load_w(slot, n, kk);
-                    load_a(slot, m, kk);
+                    load_w(slot, x, kk);
+                    load_a(slot, x, kk);
                 }
             }
         }
@@ -181,12 +211,11 @@ gemm_tc_kernel(const __grid_constant__ TcArgs g)
         // read-back: thread = row (its TMEM lane), 16 columns at a time
         int nt = 0;
         for (int t = blockIdx.x; t < tiles; t += gridDim.x, ++nt) {
-            int m, n;
-            tc_tile(t, g.m_tiles, g.n_tiles, m, n);
+            const Tile x = tile_at(t);
             const int acc = nt & 1;
             if (!tc::wait_uniform(&acc_full[acc], (nt >> 1) & 1, abort_flag)) break;
             tc::tc_fence_after();
-            const int row = m * TC_BM + warp * 32 + lane;
+            const int row = x.row + warp * 32 + lane;
             const size_t row_off = (size_t)row * g.ldc;
             const uint32_t at = tmem + ((uint32_t)(warp * 32) << 16) + acc * BN;
 #pragma unroll 1
@@ -203,9 +232,9 @@ gemm_tc_kernel(const __grid_constant__ TcArgs g)
                 } else {
                     tc::tmem_wait_ld();
 #pragma unroll
-                    for (int j = 0; j < 16; ++j) v[j] = __uint_as_float(d[j]);
+                    for (int j = 0; j < 16; ++j) v[j] = epilogue_value<EPI>(__uint_as_float(d[j]));
                 }
-                if (row < g.M && n * OUT + c0 < g.N) tc_store16<EPI>(g.c, row_off, n * OUT + c0, g.N, v);
+                if (row < x.end && x.n * OUT + c0 < g.N) tc_store16<EPI>(g.c, row_off, x.n * OUT + c0, g.N, v);
             }
             tc::tc_fence_before();
             __syncwarp();

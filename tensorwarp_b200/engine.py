@@ -36,13 +36,16 @@ class StepEngine(Protocol):
 
 class DenseEngine:
     LOGITS_BYTES = 256 << 20
+    DEFAULT_CAPACITY = 16384            # tokens per sequence of a model without a position limit
 
     def __init__(self, model, max_tokens: Optional[int] = None, max_live: int = 4, portion: int = 4096, use_pdl: bool = True,
                  use_graphs: bool = True):
-        """max_tokens: longest sequence served; portion: most tokens of a prompt per native call."""
+        """max_tokens: longest sequence served (a model without a position limit takes any); portion: most tokens of a prompt
+        per native call."""
         self.model, self.spec, self.device = model, model.spec, model.device
         self.vocab = self.spec.vocab
-        capacity = min(self.spec.max_positions, max_tokens or self.spec.max_positions)
+        limit = self.spec.max_positions
+        capacity = min(limit, max_tokens or limit) if limit is not None else max_tokens or self.DEFAULT_CAPACITY
         self.state = SequenceState(model, max_live, capacity)
         self.capacity, self.max_live = capacity, max_live
         self.flags = _dense.TWM_FLAG_PDL if use_pdl else 0
@@ -61,6 +64,9 @@ class DenseEngine:
         w_in = max([w["w_in"].shape[0] for w in self.model.layers], default=16)
         w_att = max([x.heads * x.vdim_pad for x in lays], default=16)
         w_ff = max([x.ff_pad for x in lays] + [16])
+        slots_per_row = max([x.top if x.experts else 1 for x in lays] + [1])
+        w_act = max([x.ff_pad * (x.top if x.experts else 1) for x in lays] + [16])
+        experts = max([x.experts for x in lays] + [0])
         self.max_rows = rows
         self.max_want = max(1, min(rows, self.LOGITS_BYTES // (4 * self.vocab)))
 
@@ -71,9 +77,24 @@ class DenseEngine:
         self._buf = dict(meta=zeros(8, dtype=i32), tokens=zeros(rows, dtype=i32), want=zeros(self.max_want, dtype=i32),
                          x0=zeros(rows, wp, dtype=f32), x1=zeros(rows, wp, dtype=f32), y=zeros(rows, wp, dtype=f32),
                          a=zeros(rows, wp, dtype=dt), proj=zeros(rows, w_in, dtype=dt), att=zeros(rows, w_att, dtype=dt),
-                         act=zeros(rows, w_ff, dtype=dt), vec=zeros(w_in + w_att + w_ff, dtype=f32),
+                         act=zeros(rows * slots_per_row, w_ff, dtype=dt), vec=zeros(w_in + w_att + w_act + experts, dtype=f32),
                          logits=zeros(self.max_want, self.vocab, dtype=f32))
         b = _dense.Buffers(max_rows=rows, max_want=self.max_want)
+        latent = [x for x in lays if x.mixer == _dense.MIX_LATENT]
+        if latent:
+            b.max_keys = min(self.capacity, rows + max(x.window for x in latent) - 1)
+            self._buf.update(lat=zeros(b.max_keys, max(x.rank_pad + x.rot_pad for x in latent), dtype=dt),
+                             kv=zeros(b.max_keys, max(x.heads * (x.dim_pad + x.vdim_pad) for x in latent), dtype=dt))
+        linear = [x for x in lays if x.mixer == _dense.MIX_GLA]
+        if linear:
+            self._buf.update(decay=zeros(rows, max(x.heads * x.dim_pad for x in linear), dtype=f32),
+                             chunk_state=zeros((rows + 63) // 64, max(x.heads * x.dim_pad * x.vdim_pad for x in linear), dtype=f32),
+                             mix=zeros(rows, max(x.heads * x.vdim_pad for x in linear), dtype=f32))
+        if experts:
+            b.max_slots = rows * slots_per_row
+            self._buf.update(router_logits=zeros(rows, experts, dtype=f32), route=zeros(3 * b.max_slots + 2 * experts + 1, dtype=i32),
+                             route_weight=zeros(b.max_slots, dtype=f32), grouped=zeros(b.max_slots, wp, dtype=dt),
+                             expert_out=zeros(b.max_slots, wp, dtype=dt))
         for name, t in self._buf.items():
             setattr(b, name, t.data_ptr())
         self._b = b
@@ -102,8 +123,8 @@ class DenseEngine:
 
     # ------------------------------------------------------------------- steps --
     def step(self, seq: int, tokens: Sequence[int], want: Sequence[int] = (), layer_trace: Optional[List[torch.Tensor]] = None):
-        """See StepEngine.  layer_trace: a list that receives, per native call, the residual stream after every layer,
-        f32 [layers, tokens, width]."""
+        """See StepEngine.  layer_trace: a list that receives, per native call, the residual stream after every layer run,
+        f32 [layer runs, tokens, width]."""
         tokens, want = list(tokens), list(want)
         self._check_tokens(tokens)
         if any(b <= a for a, b in zip(want, want[1:])) or (want and not 0 <= want[0] <= want[-1] < len(tokens)):
@@ -149,7 +170,7 @@ class DenseEngine:
                 self._buf["want"][:len(want)].copy_(torch.tensor(want, dtype=torch.int32))
             self._set_step(first, slot)
             if trace:
-                out = torch.empty((len(self.spec.layers), len(tokens), self.model.width_pad), dtype=torch.float32, device=self.device)
+                out = torch.empty((len(self.model.runs), len(tokens), self.model.width_pad), dtype=torch.float32, device=self.device)
             self.enqueue_prefill(len(tokens), first, len(want), out)
         return out
 

@@ -15,6 +15,7 @@ from . import checkpoint
 _MODULES = {                    # imported on first use: a model pulls in only its own kernels
     "Bidasun": "tensorwarp_b200.models.bidasun",
     "TWMarlinQ4": "tensorwarp_b200.models.tw_marlin",
+    "Zukotar": "tensorwarp_b200.models.zukotar",
 }
 _BUILDERS: Dict[str, Callable] = {}
 

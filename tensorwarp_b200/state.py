@@ -1,12 +1,13 @@
-"""What a sequence leaves behind between steps: per-layer keys and values and the previous token's mixer input.
+"""What a sequence leaves behind between steps, for every run of a layer: keys and values and the previous token's mixer
+input, latents, or a recurrent state.
 
 The state of `slots` sequences is allocated once; a sequence holds one slot from ``open`` to ``close``.
 Nothing has to be cleared when a slot changes hands: a query sees only positions its own sequence has
-written, and the kernels take the state before position 0 as zero.
+written, and the kernels take the state (recurrent or shifted) before position 0 as zero.
 """
 from __future__ import annotations
 
-from typing import List, Optional
+from typing import Dict, List
 
 import torch
 
@@ -18,21 +19,31 @@ class StateError(RuntimeError):
 class SequenceState:
     def __init__(self, model, slots: int, capacity: int):
         """model: dense.DenseModel; capacity: tokens per slot."""
-        from .dense import pad16
+        from .dense import AttentionSpec, LatentAttentionSpec, pad16
         if slots < 1 or capacity < 1:
             raise ValueError("slots and capacity must be positive")
         self.slots, self.capacity = slots, capacity
         dt, dev = model.dtype, model.device
-        self.k: List[torch.Tensor] = []
-        self.v: List[torch.Tensor] = []
-        self.shift: List[Optional[torch.Tensor]] = []
-        for spec, w in zip(model.spec.layers, model.layers):
-            m = spec.mixer
-            self.k.append(torch.zeros((slots, capacity, m.kv_heads * pad16(m.dim)), dtype=dt, device=dev))
-            self.v.append(torch.zeros((slots, capacity, m.kv_heads * pad16(m.vdim)), dtype=dt, device=dev))
-            # two rows, used in turn by the parity of the position: a step reads one while it writes the other
-            self.shift.append(torch.zeros((slots, 2, model.width_pad), dtype=torch.float32, device=dev)
-                              if w.get("shift") is not None else None)
+        f32 = torch.float32
+        self.runs: List[Dict[str, torch.Tensor]] = []       # by the name of the native layer's field
+
+        def zeros(*shape, dtype=dt):
+            return torch.zeros((slots,) + shape, dtype=dtype, device=dev)
+
+        for i, _ in model.runs:
+            m, run = model.spec.layers[i].mixer, {}
+            if isinstance(m, AttentionSpec):
+                run["k_cache"] = zeros(capacity, m.kv_heads * pad16(m.dim))
+                run["v_cache"] = zeros(capacity, m.kv_heads * pad16(m.vdim))
+                if model.layers[i].get("shift") is not None:
+                    # two rows, used in turn by the parity of the position: a step reads one while it writes the other
+                    run["shift_state"] = zeros(2, model.width_pad, dtype=f32)
+            elif isinstance(m, LatentAttentionSpec):
+                run["latent_cache"] = zeros(capacity, pad16(m.rank) + pad16(m.rot_dim))
+            else:
+                run["gla_state"] = zeros(m.heads, pad16(m.dim), pad16(m.vdim), dtype=f32)
+            self.runs.append(run)
+        self.k, self.v, self.shift = ([run.get(name) for run in self.runs] for name in ("k_cache", "v_cache", "shift_state"))
         self._free = list(range(slots - 1, -1, -1))
         self._length = {}
 
@@ -65,4 +76,4 @@ class SequenceState:
         self._length[slot] = n
 
     def bytes(self) -> int:
-        return sum(t.numel() * t.element_size() for t in self.k + self.v + [s for s in self.shift if s is not None])
+        return sum(t.numel() * t.element_size() for run in self.runs for t in run.values())
