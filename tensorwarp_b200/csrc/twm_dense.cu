@@ -15,6 +15,7 @@
 #include "twm_dense_moe.cuh"
 #include "twm_dense_rows.cuh"
 #include "twm_dense_simt.cuh"
+#include "twm_dense_softmax_tc.cuh"
 #include "twm_dense_tc.cuh"
 #include "twm_dense_tc2.cuh"
 
@@ -517,10 +518,34 @@ twm_status attention(const twm_dense_model* m, const twm_dense_layer& l, const t
 }
 
 // ------------------------------------------------------------------ latent --
+bool softmax_tc_fits(const SoftmaxArgs<float>&) { return false; }
+bool softmax_tc_fits(const SoftmaxArgs<bf16>& g)
+{
+    return g.vdim_pad <= 128 && softmax_tc_kboxes(g.dim_pad, g.rot_pad) <= SX_MAX_KBOXES && g.scale > 0.0f && ((uintptr_t)g.proj & 15) == 0 &&
+           ((uintptr_t)g.kv & 15) == 0 && ((uintptr_t)g.shared & 15) == 0;
+}
+twm_status softmax_tc(const SoftmaxArgs<float>&, int, void*) { return invalid("the tcgen05 attention takes bfloat16"); }
+twm_status softmax_tc(const SoftmaxArgs<bf16>& g, int flags, void* stream)
+{
+    SoftmaxTcArgs t;
+    t.a = g;
+    const long qw = g.dim_pad + g.rot_pad, kv_ld = (long)g.heads * (g.dim_pad + g.vdim_pad), keys = g.first_pos - g.first_key + g.rows;
+    auto heads_map = [&](CUtensorMap* map, const bf16* base, int cols, long per_head, long rows, long ld, int box_rows) {
+        return tensor_map(map, MapKey{MAP_BF16_SWIZZLED, base, 3, {cols, g.heads, rows, 0}, {1, per_head, ld, 0}, {64, 1, box_rows, 0}});
+    };
+    if (!heads_map(&t.q_map, g.proj, g.dim_pad, qw, g.rows, g.ld, SX_Q) || !heads_map(&t.qr_map, g.proj + g.dim_pad, g.rot_pad, qw, g.rows, g.ld, SX_Q) ||
+        !heads_map(&t.k_map, g.kv, g.dim_pad, g.dim_pad, keys, kv_ld, SX_K) || !rows_map(&t.kr_map, g.shared, keys, g.rot_pad, g.shared_ld, SX_K) ||
+        !heads_map(&t.v_map, g.kv + (long)g.heads * g.dim_pad, g.vdim_pad, g.vdim_pad, keys, kv_ld, SX_K))
+        return invalid("cuTensorMapEncodeTiled refused a map of the tcgen05 softmax attention");
+    return launch("attn_softmax_tc", attn_softmax_tc_kernel, dim3((g.rows + SX_Q - 1) / SX_Q, g.heads), SX_THREADS,
+                  softmax_tc_smem_bytes(g.dim_pad, g.rot_pad, g.vdim_pad), flags, stream, 0, t);
+}
 template <typename T>
 twm_status softmax_attention(const SoftmaxArgs<T>& g, int kernel, int flags, void* stream)
 {
-    if (kernel != 0 && kernel != 1) return invalid("kernel");
+    if (kernel != 0 && kernel != 1 && kernel != 3) return invalid("kernel");
+    if (kernel == 3 && !softmax_tc_fits(g)) return invalid("the tcgen05 softmax attention takes bfloat16 heads of up to 128 columns");
+    if (kernel == 3 || (kernel == 0 && softmax_tc_fits(g))) return softmax_tc(g, flags, stream);
     const int vblock = AS_VPT * AS_THREADS;
     return launch("attn_softmax_simt", attn_softmax_simt_kernel<T>, dim3(g.rows, g.heads, (g.vdim_pad + vblock - 1) / vblock), AS_THREADS,
                   sizeof(float) * (size_t)(g.dim_pad + g.rot_pad + AS_THREADS), flags, stream, 0, g);
