@@ -742,6 +742,25 @@ def random_bidasun(torch, config: dict, device, **engine_options):
     return DenseEngine(model, **engine_options)
 
 
+def engine_timer(torch, eng):
+    """Milliseconds per call of something that enqueues on the engine's stream."""
+    def timed(enqueue, steps, warm=3):
+        torch.cuda.synchronize()
+        time.sleep(0.5)          # directly after long prompts everything reads slower for a while
+        with torch.cuda.stream(eng.stream):
+            for _ in range(warm):
+                enqueue()
+            torch.cuda.synchronize()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record(eng.stream)
+            for _ in range(steps):
+                enqueue()
+            e1.record(eng.stream)
+            torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / steps
+    return timed
+
+
 def bidasun_figures(torch, device, name: str, gbs: float, tflops: float) -> dict:
     """Prefill and decode throughput of one size, and its products and attention one by one."""
     import ctypes as C
@@ -760,20 +779,7 @@ def bidasun_figures(torch, device, name: str, gbs: float, tflops: float) -> dict
         t.normal_(generator=gen)
     torch.cuda.synchronize()
 
-    def timed(enqueue, steps, warm=3):
-        torch.cuda.synchronize()
-        time.sleep(0.5)          # directly after long prompts everything reads slower for a while
-        with torch.cuda.stream(eng.stream):
-            for _ in range(warm):
-                enqueue()
-            torch.cuda.synchronize()
-            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            e0.record(eng.stream)
-            for _ in range(steps):
-                enqueue()
-            e1.record(eng.stream)
-            torch.cuda.synchronize()
-        return e0.elapsed_time(e1) / steps
+    timed = engine_timer(torch, eng)
 
     def visible(n):                                  # query-key pairs of an n-token prompt
         full = sum(min(i + 1, size["window"]) for i in range(n))
@@ -860,7 +866,143 @@ def q4_decode_same_size(torch, device, name: str, gbs: float) -> dict:
             "hbm_gbs": round(nbytes / ms / 1e6, 1), "frac_hbm": round(nbytes / ms / 1e6 / gbs, 3), "launches": eng.launches_per_step}
 
 
-def run_bidasun(args):
+# width, layers (linear and latent in turn), heads of both, head size, rotated part, latent, window, experts, chosen, kept groups,
+# expert width, vocabulary; the same widths, heads, depths, windows and vocabularies as the sizes above
+ZUKOTAR_SIZES = {
+    "1b": dict(width=2048, layers=16, heads=16, dim=128, rot=64, rank=512, low=16, window=512, experts=64, top=8, groups=8, keep=4, ff=1024,
+               vocab=32768),
+    "7b": dict(width=3584, layers=28, heads=28, dim=128, rot=64, rank=512, low=16, window=1024, experts=32, top=4, groups=4, keep=2, ff=2560,
+               vocab=152064),
+    "13b-wide": dict(width=5120, layers=12, heads=40, dim=128, rot=64, rank=512, low=32, window=2048, experts=16, top=2, groups=4, keep=2, ff=6144,
+                     vocab=32768),
+}
+
+
+def zukotar_config(size: dict) -> dict:
+    linear = {"type": "gla", "mixer": {"heads": size["heads"], "dim": size["dim"], "vdim": size["dim"], "tau": 16.0}}
+    latent = {"type": "latent_attention",
+              "mixer": {"heads": size["heads"], "dim": size["dim"], "rot_dim": size["rot"], "vdim": size["dim"], "kv_rank": size["rank"],
+                        "scale": (size["dim"] + size["rot"]) ** -0.5, "rot": {"base": 10000.0, "dims": size["rot"]}, "mask": {"size": size["window"]}}}
+    mlp = {"kind": "moe", "expert": {"ff": size["ff"]},
+           "router": {"experts": size["experts"], "top": size["top"], "groups": {"count": size["groups"], "keep": size["keep"]}}}
+    return {"architecture": "Zukotar", "width": size["width"], "vocab": size["vocab"], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "layers": [dict(latent if i % 2 else linear, mlp=mlp) for i in range(size["layers"])]}
+
+
+def random_zukotar(torch, config: dict, low: int, device, **engine_options):
+    """An engine on random bfloat16 weights of the configuration."""
+    from tensorwarp_b200 import dense
+    from tensorwarp_b200.engine import DenseEngine
+    from tensorwarp_b200.models import zukotar
+    gen = torch.Generator(device=device).manual_seed(1)
+
+    def get(name, shape):
+        if "norm" in name.split(".")[-1]:
+            return torch.ones(shape, device=device)
+        if name.endswith("a2.b"):
+            return torch.rand(shape, generator=gen, device=device) * 6
+        return torch.randn(shape, generator=gen, device=device, dtype=torch.bfloat16) * (1.0 if name == "embed" else 0.02)
+
+    spec = zukotar.parse_config(config, lambda name: (low, config["width"]))
+    return DenseEngine(dense.DenseModel(spec, zukotar.model_tensors(spec, get), torch.bfloat16, device), **engine_options)
+
+
+def zukotar_figures(torch, device, name: str, gbs: float, tflops: float) -> dict:
+    """Prefill and decode throughput of one size, and its products and mixers one by one."""
+    import ctypes as C
+
+    from tensorwarp_b200 import _dense
+    size = ZUKOTAR_SIZES[name]
+    eng = random_zukotar(torch, zukotar_config(size), size["low"], device, max_live=1, portion=8192, max_tokens=8192 + 64)
+    lib, model = _dense.lib(), eng.model
+    w, h, d, r, k, v, nl = (size[x] for x in ("width", "heads", "dim", "rot", "rank", "vocab", "layers"))
+    e, top, ff, low = (size[x] for x in ("experts", "top", "ff", "low"))
+    linear_in, latent_in, expand = 4 * h * d + low, h * (d + r) + k + r + (h + 15) // 16 * 16, 2 * h * d
+    mixers = nl // 2 * (w * linear_in + h * d * low + w * latent_in + k * expand) + nl * h * d * w
+    active, routers = nl * top * 2 * ff * w, nl * e * w                    # weights one token meets
+    gen = torch.Generator(device=device).manual_seed(3)
+    b = eng._buf
+    b["tokens"].copy_(torch.randint(0, v, b["tokens"].shape, generator=gen, device=device, dtype=torch.int32))
+    b["want"].zero_()
+    # real operands: products of zeros draw little power and run at clocks that no workload sees
+    for t in [b[x] for x in ("a", "proj", "att", "act", "grouped", "lat", "kv")] + [t for run in eng.state.runs for t in run.values()]:
+        t.normal_(generator=gen)
+    torch.cuda.synchronize()
+    timed = engine_timer(torch, eng)
+    out = {"config": dict(size), "active_weights": mixers + active + routers, "prefill": [], "decode": []}
+    for ctx in (BIDASUN_CONTEXT, 8000):
+        eng._set_step(ctx, 0, 1)
+        graph = eng.capture_decode("greedy")
+        ms = timed(graph.replay, 128, 20)
+        nbytes = 2 * (mixers + active + routers + v * w) + nl // 2 * (min(ctx, size["window"]) * (k + r) * 2 + 2 * h * d * d * 4)
+        out["decode"].append({"context": ctx, "ms": round(ms, 4), "tok_s": round(1e3 / ms, 1), "bytes": nbytes,
+                              "hbm_gbs": round(nbytes / ms / 1e6, 1), "frac_hbm": round(nbytes / ms / 1e6 / gbs, 3),
+                              "launches": eng.launches_per_step})
+
+    def pairs(n):
+        return sum(min(i + 1, size["window"]) for i in range(n))
+
+    def roofline(ms, flops, nbytes):
+        return {"us": round(ms * 1e3, 1), "tflops": round(flops / ms / 1e9, 1), "gbs": round(nbytes / ms / 1e6, 1),
+                "frac_roofline": round(max(flops / ms / 1e9 / tflops, nbytes / ms / 1e6 / gbs), 3)}
+
+    def check(status, what):
+        _dense.check(status, what)
+
+    kernels = []
+    bf16, s = _dense.TWM_DENSE_BF16, eng.stream.cuda_stream
+    offsets = torch.zeros(e + 1, dtype=torch.int32, device=device)
+    for n in BIDASUN_PROMPTS:
+        row = {"tokens": n}
+        for label, wt, src, dst, cols, kk, epi, layers in (
+                ("linear_in", "w_in", "a", "proj", linear_in, w, _dense.EPI_STORE, model.layers[0::2]),
+                ("latent_in", "w_in", "a", "proj", latent_in, w, _dense.EPI_STORE, model.layers[1::2]),
+                ("out", "w_out", "att", "y", w, h * d, _dense.EPI_STORE_F32, model.layers),
+                ("router", "w_router", "a", "router_logits", e, w, _dense.EPI_STORE_F32, model.layers)):
+            def enqueue():
+                for lw in layers:
+                    check(lib.twm_dense_gemm(bf16, b[src].data_ptr(), kk, lw[wt].data_ptr(), kk, b[dst].data_ptr(), cols, n, cols, kk, epi, 0,
+                                             0, s), "gemm")
+            row[label] = roofline(timed(enqueue, 4, 2) / len(layers), 2.0 * n * kk * cols, 2 * kk * cols + 2 * n * (kk + cols))
+        # rows of the experts as an even router would deal them
+        slots = n * top
+        offsets.copy_((torch.arange(e + 1, device=device) * slots) // e)
+        used = min(e, slots)
+        for label, wt, src, dst, cols, kk, epi in (("experts_up", "w_gate_up", "grouped", "act", ff, w, _dense.EPI_RELU2),
+                                                  ("experts_down", "w_down", "act", "expert_out", w, ff, _dense.EPI_STORE)):
+            def enqueue():
+                for lw in model.layers:
+                    check(lib.twm_dense_grouped_gemm(bf16, b[src].data_ptr(), kk, lw[wt].data_ptr(), kk, b[dst].data_ptr(), cols, offsets.data_ptr(),
+                                                     e, slots, cols, kk, epi, 0, 0, s), "grouped_gemm")
+            row[label] = roofline(timed(enqueue, 4, 2) / nl, 2.0 * slots * kk * cols, 2 * used * kk * cols + 2 * slots * (kk + cols))
+        eng._set_step(0, 0)
+
+        def attend():
+            for i in range(1, nl, 2):
+                check(lib.twm_dense_attention(C.byref(eng._desc), i, C.byref(eng._b), n, 0, 0, 0, s), "attention")
+
+        def recur():
+            for i in range(0, nl, 2):
+                check(lib.twm_dense_gla(C.byref(eng._desc), i, C.byref(eng._b), n, 0, 0, s), "gla")
+        b["proj"].normal_(generator=gen)
+        row["latent_attention"] = roofline(timed(attend, 4, 2) / (nl // 2), 2.0 * h * (2 * d + r) * pairs(n) + 2.0 * n * k * expand,
+                                           2 * n * (latent_in + h * d) + 2 * k * expand)
+        # the least a chunk-wise recurrence does: scores, their product with v, state in and state out, in chunks of 64
+        row["linear_attention"] = roofline(timed(recur, 4, 2) / (nl // 2), 2.0 * n * h * (2 * d * d + 64 * d), 2 * n * (linear_in + h * d))
+        kernels.append(row)
+    out["prefill_kernels"] = kernels
+    for n in BIDASUN_PROMPTS:
+        eng._set_step(0, 0)
+        ms = timed(lambda: eng.enqueue_prefill(n, 0, 1), 5)
+        flops = 2.0 * n * (mixers + active + routers) + nl // 2 * (2.0 * h * (2 * d + r) * pairs(n) + 2.0 * n * h * (2 * d * d + 64 * d)) + 2.0 * w * v
+        out["prefill"].append({"tokens": n, "ms": round(ms, 3), "tok_s": round(n / ms * 1e3), "tflops": round(flops / ms / 1e9, 1),
+                               "frac_bf16_peak": round(flops / ms / 1e9 / tflops, 3), "launches": eng.launches_per_step})
+    out["device_error"] = _dense.device_error()
+    return out
+
+
+def run_dense(args):
+    """One line with the figures of a dense-weight decoder at a few sizes, each beside the framework's closest model."""
     import torch
     torch.cuda.set_device(0)
     device = torch.device("cuda", 0)
@@ -870,14 +1012,20 @@ def run_bidasun(args):
     if os.path.exists(path):
         with open(path) as f:
             tflops = float(json.load(f)["bf16_tflops"])
-    line = {"bench": "bidasun", "data": "random weights and tokens", "dtype": "bf16", "peaks": {"hbm_gbs": gbs, "bf16_tflops": tflops,
+    line = {"bench": args.workload, "data": "random weights and tokens", "dtype": "bf16", "peaks": {"hbm_gbs": gbs, "bf16_tflops": tflops,
             "source": source}, "sizes": {}}
     with ClockSampler(0) as clocks:
         for name in args.sizes.split(","):
-            q4 = q4_decode_same_size(torch, device, name, gbs)
-            torch.cuda.empty_cache()
-            line["sizes"][name] = bidasun_figures(torch, device, name, gbs, tflops)
-            line["sizes"][name]["q4_decode_same_size"] = q4
+            if args.workload == "bidasun":
+                q4 = q4_decode_same_size(torch, device, name, gbs)
+                torch.cuda.empty_cache()
+                line["sizes"][name] = bidasun_figures(torch, device, name, gbs, tflops)
+                line["sizes"][name]["q4_decode_same_size"] = q4
+            else:
+                line["sizes"][name] = zukotar_figures(torch, device, name, gbs, tflops)
+                torch.cuda.empty_cache()
+                if not args.alone:
+                    line["sizes"][name]["bidasun_same_size"] = bidasun_figures(torch, device, name, gbs, tflops)
             torch.cuda.empty_cache()
     line["clocks"] = clocks.summary()
     print(json.dumps(line), flush=True)
@@ -1252,12 +1400,14 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-decode", action="store_true", help="skip the configs[3] decode tok/s measurement")
-    ap.add_argument("--workload", default="w4a16", choices=["w4a16", "bidasun"],
-                    help="bidasun: prefill and decode of the Bidasun decoder at a few sizes, beside the 4-bit decoder's step")
-    ap.add_argument("--sizes", default="1b,7b,13b-wide", help="--workload bidasun: which sizes")
+    ap.add_argument("--workload", default="w4a16", choices=["w4a16", "bidasun", "zukotar"],
+                    help="bidasun: prefill and decode of the Bidasun decoder at a few sizes, beside the 4-bit decoder's step; "
+                         "zukotar: the Zukotar decoder's, beside Bidasun")
+    ap.add_argument("--alone", action="store_true", help="--workload zukotar: without Bidasun beside it")
+    ap.add_argument("--sizes", default="1b,7b,13b-wide", help="--workload bidasun or zukotar: which sizes")
     args = ap.parse_args()
-    if args.workload == "bidasun":
-        run_bidasun(args)
+    if args.workload != "w4a16":
+        run_dense(args)
     elif args.impl == "reference":
         args.steps = args.steps if args.steps is not None else 5
         args.warmup = args.warmup if args.warmup is not None else 1

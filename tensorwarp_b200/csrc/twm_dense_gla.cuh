@@ -52,12 +52,12 @@ __global__ void __launch_bounds__(GD_THREADS)
 gla_decay_kernel(const GlaArgs<T> g)
 {
     using V = Vec<T>;
-    pdl_launch_dependents();
     __shared__ __align__(16) float low[GD_ROWS][GD_RANK];
     const int col = blockIdx.x * GD_THREADS + threadIdx.x, r0 = blockIdx.y * GD_ROWS, n = min(GD_ROWS, g.rows - r0);
     const int cols = g.heads * g.dim_pad;
     const float bias = col < cols ? __ldg(g.decay_bias + col) : 0.0f;
     pdl_wait_prior_grids();
+    pdl_launch_dependents();
     float z[GD_ROWS];
 #pragma unroll
     for (int r = 0; r < GD_ROWS; ++r) z[r] = bias;
@@ -101,7 +101,6 @@ template <typename T>
 __global__ void __launch_bounds__(GR_THREADS)
 gla_rows_kernel(const GlaArgs<T> g)
 {
-    pdl_launch_dependents();
     extern __shared__ __align__(16) float gr_smem[];
     __shared__ float part[GR_TOKENS][8][GR_COLS];
     float* s = gr_smem;                                    // [dim_pad][32]
@@ -109,6 +108,7 @@ gla_rows_kernel(const GlaArgs<T> g)
     float* ks = qs + GR_TOKENS * g.dim_pad;
     float* as = ks + GR_TOKENS * g.dim_pad;
     pdl_wait_prior_grids();
+    pdl_launch_dependents();
     const int h = blockIdx.y, c = threadIdx.x & 31, grp = threadIdx.x >> 5, col = blockIdx.x * GR_COLS + c;
     const bool in = col < g.vdim_pad;
     float* st = g.slot_state(h);
@@ -153,8 +153,8 @@ template <typename T>
 __global__ void __launch_bounds__(ROW_THREADS)
 gla_gate_kernel(const GlaArgs<T> g)
 {
-    pdl_launch_dependents();
     pdl_wait_prior_grids();
+    pdl_launch_dependents();
     const int lane = threadIdx.x & 31, r = blockIdx.x;
     for (int h = threadIdx.x >> 5; h < g.heads; h += ROW_THREADS / 32) {
         const float* o = g.mix + ((size_t)r * g.heads + h) * g.vdim_pad;
@@ -178,7 +178,6 @@ __host__ inline size_t gla_chunk_state_smem_bytes(int dim_pad, int vdim_pad) {
 __global__ void __launch_bounds__(GC_THREADS)
 gla_chunk_state_kernel(const GlaArgs<bf16> g)
 {
-    pdl_launch_dependents();
     extern __shared__ __align__(16) uint8_t gc_smem[];
     const int krow = g.dim_pad * 2 + 16, vrow = g.vdim_pad * 2 + 16;      // padded: eight rows of a fragment hit distinct banks
     uint8_t* khi = gc_smem;                                // [64][dim_pad]
@@ -188,6 +187,7 @@ gla_chunk_state_kernel(const GlaArgs<bf16> g)
     const int h = blockIdx.y, r0 = blockIdx.x * GLA_CHUNK, n = min(GLA_CHUNK, g.rows - r0);
     const int cols = g.heads * g.dim_pad;
     pdl_wait_prior_grids();
+    pdl_launch_dependents();
     const bf16* row0 = g.proj + (size_t)r0 * g.ld;
     const float* b0 = g.decay + (size_t)r0 * cols + h * g.dim_pad;
     for (int i = tid; i < GLA_CHUNK * (g.vdim_pad / 8); i += GC_THREADS) {
@@ -253,8 +253,8 @@ template <typename T>
 __global__ void __launch_bounds__(GS_THREADS)
 gla_scan_kernel(const GlaArgs<T> g)
 {
-    pdl_launch_dependents();
     pdl_wait_prior_grids();
+    pdl_launch_dependents();
     const int per_head = g.dim_pad * g.vdim_pad / 4, i = blockIdx.x * GS_THREADS + threadIdx.x;
     if (i >= g.heads * per_head) return;
     const int h = i / per_head, e = i - h * per_head, d = e * 4 / g.vdim_pad;
@@ -298,7 +298,6 @@ template <int DV>
 __global__ void __launch_bounds__(GC_THREADS, 2)
 gla_chunk_out_kernel(const GlaArgs<bf16> g)
 {
-    pdl_launch_dependents();
     extern __shared__ __align__(16) uint8_t gc_smem[];
     const int krow = g.dim_pad * 2 + 16, vrow = g.vdim_pad * 2 + 16, brow = g.dim_pad + 8;
     uint8_t* ks = gc_smem;                                 // [64][dim_pad]
@@ -311,6 +310,7 @@ gla_chunk_out_kernel(const GlaArgs<bf16> g)
     const int h = blockIdx.y, r0 = blockIdx.x * GLA_CHUNK, n = min(GLA_CHUNK, g.rows - r0);
     const int cols = g.heads * g.dim_pad;
     pdl_wait_prior_grids();
+    pdl_launch_dependents();
     const bf16* row0 = g.proj + (size_t)r0 * g.ld;
     const int kp = g.dim_pad / 8, vp = g.vdim_pad / 8;
     for (int i = tid; i < GLA_CHUNK * kp; i += GC_THREADS) {

@@ -35,9 +35,9 @@ template <typename T>
 __global__ void __launch_bounds__(ROW_THREADS)
 latent_rows_kernel(const LatentRowsArgs<T> g)
 {
-    pdl_launch_dependents();
     __shared__ float red[32];
     pdl_wait_prior_grids();
+    pdl_launch_dependents();
     const int width = g.rank_pad + g.rot_pad, pos0 = g.meta[0];
     T* cache = g.cache + (size_t)g.meta[1] * g.capacity * width;
     if ((int)blockIdx.x >= g.rows) {
@@ -98,13 +98,13 @@ __global__ void __launch_bounds__(AS_THREADS)
 attn_softmax_simt_kernel(const SoftmaxArgs<T> g)
 {
     using V = Vec<T>;
-    pdl_launch_dependents();
     extern __shared__ __align__(16) float attn_smem[];
     __shared__ float red[32];
     const int qw = g.dim_pad + g.rot_pad;
     float* qs = attn_smem;                      // [dim_pad + rot_pad]
     float* ws = qs + qw;                        // [AS_THREADS]
     pdl_wait_prior_grids();
+    pdl_launch_dependents();
     const int r = blockIdx.x, h = blockIdx.y, p = g.first_pos + r;
     const int kv_ld = g.heads * (g.dim_pad + g.vdim_pad);
     const T* k_base = g.kv + h * g.dim_pad;

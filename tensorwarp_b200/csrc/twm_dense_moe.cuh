@@ -76,12 +76,12 @@ __global__ void __launch_bounds__(RT_WARPS * 32)
 route_kernel(const float* __restrict__ logits, int ld, const RouterArgs r, int rows, int* __restrict__ ids, float* __restrict__ weights,
              int* __restrict__ place, int* __restrict__ counts)
 {
-    pdl_launch_dependents();
     extern __shared__ float route_smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     float* s = route_smem + warp * (r.experts + r.groups);
     const int t = blockIdx.x * RT_WARPS + warp;
     pdl_wait_prior_grids();
+    pdl_launch_dependents();
     if (t >= rows) return;
     int id;
     float weight;
@@ -128,9 +128,9 @@ __global__ void __launch_bounds__(MG_THREADS)
 group_rows_kernel(const T* __restrict__ a, int wp, const RouterArgs r, int rows, const int* __restrict__ ids, const int* __restrict__ place,
                   const int* __restrict__ counts, int* __restrict__ row, int* __restrict__ offsets, T* __restrict__ grouped)
 {
-    pdl_launch_dependents();
     __shared__ int off[MOE_MAX_EXPERTS + 1];
     pdl_wait_prior_grids();
+    pdl_launch_dependents();
     if (threadIdx.x < 32) warp_prefix([&](int e) { return counts[e]; }, r.experts, off, threadIdx.x);
     __syncthreads();
     if (blockIdx.x == 0)
@@ -156,11 +156,11 @@ __global__ void __launch_bounds__(256)
 moe_gemm_simt_kernel(const T* __restrict__ a, int lda, const T* __restrict__ w, int ldw, void* __restrict__ c, int ldc,
                      const int* __restrict__ offsets, int experts, int N, int K)
 {
-    pdl_launch_dependents();
     __shared__ int pre[MOE_MAX_EXPERTS + 1];
     __shared__ __align__(16) float as[SK][ST + 4];
     __shared__ __align__(16) float bs[SK][ST + 4];
     pdl_wait_prior_grids();
+    pdl_launch_dependents();
     if (threadIdx.x < 32) warp_prefix([&](int e) { return (offsets[e + 1] - offsets[e] + ST - 1) / ST; }, experts, pre, threadIdx.x);
     __syncthreads();
     if ((int)blockIdx.y >= pre[experts]) return;

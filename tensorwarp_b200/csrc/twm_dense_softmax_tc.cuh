@@ -48,7 +48,6 @@ __device__ __forceinline__ uint64_t sx_value_desc(uint32_t addr) {      // colum
 __global__ void __launch_bounds__(SX_THREADS, 2)
 attn_softmax_tc_kernel(const __grid_constant__ SoftmaxTcArgs args)
 {
-    pdl_launch_dependents();
     extern __shared__ uint8_t sx_smem_raw[];
     __shared__ SoftmaxTcSync sm;
     const SoftmaxArgs<bf16>& g = args.a;
@@ -67,15 +66,18 @@ attn_softmax_tc_kernel(const __grid_constant__ SoftmaxTcArgs args)
         sm.abort_flag = 0;
         mbar_fence_init();
     }
+    // Tensor memory is asked for once the kernel before is over (its CTAs and pairs of CTAs have given theirs back), and
+    // the next kernel may come once this CTA has it: an allocation waits without a limit.
+    pdl_wait_prior_grids();
     if (warp == 5) {
         tc::tmem_alloc(&sm.tmem_base, 256);
         tc::tc_fence_before();
     }
     __syncthreads();
     tc::tc_fence_after();
+    pdl_launch_dependents();
     volatile int* abort_flag = &sm.abort_flag;
     const uint32_t tmem = sm.tmem_base, tmem_o = tmem + 2 * SX_K;
-    pdl_wait_prior_grids();
 
     const int h = blockIdx.y, r0 = blockIdx.x * SX_Q;
     const int p0 = g.first_pos + r0, p1 = g.first_pos + min(g.rows, r0 + SX_Q) - 1;      // positions of the CTA's first and last query
