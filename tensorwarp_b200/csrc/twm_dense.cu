@@ -441,8 +441,7 @@ twm_status grouped_gemm(const T* a, int lda, const T* w, int ldw, void* c, int l
 
 twm_status route(const float* logits, const RouterArgs& r, int rows, int* ids, float* weights, int* place, int* counts, int flags, void* stream)
 {
-    return launch("route", route_kernel, dim3((rows + RT_WARPS - 1) / RT_WARPS), RT_WARPS * 32, sizeof(float) * RT_WARPS * (r.experts + r.groups),
-                  flags, stream, 0, logits, r.experts, r, rows, ids, weights, place, counts);
+    return launch("route", route_kernel, dim3((rows + RT_WARPS - 1) / RT_WARPS), RT_WARPS * 32, route_smem_bytes(r), flags, stream, 0, logits, r.experts, r, rows, ids, weights, place, counts);
 }
 
 template <typename T>

@@ -84,6 +84,8 @@ __device__ __forceinline__ bool elect_one() {
     return p != 0;
 }
 
+__device__ __forceinline__ void l2_prefetch(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p) : "memory"); }
+
 // Ask for a tensor map (kernel-parameter space) ahead of the first load that uses it.
 __device__ __forceinline__ void prefetch_map(const CUtensorMap* map) {
     asm volatile("prefetch.tensormap [%0];" ::"l"(reinterpret_cast<uint64_t>(map)) : "memory");

@@ -101,11 +101,11 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
     const int row_bytes = g.ldw * (int)sizeof(T);
     const int pieces = (row_bytes + GV_PIECE - 1) / GV_PIECE;        // of one row as it lies in memory
     const int chunks = ROUTE == ROUTE_COLUMNS ? pieces * g.router.top : pieces;
-    // where row o of the list lies, its chunk's expert given
-    auto physical = [&](int o, int slot) {
-        if (ROUTE == ROUTE_ROWS) return ids_s[o / g.expert_rows] * g.expert_rows + o % g.expert_rows;
-        if (ROUTE == ROUTE_COLUMNS) return ids_s[slot] * g.expert_rows + o;
-        return o;
+    // where row o of the list lies (ROUTE_COLUMNS: in an expert's matrix)
+    auto physical = [&](int o) {
+        if (ROUTE != ROUTE_ROWS) return o;
+        const int slot = o / g.expert_rows;
+        return ids_s[slot] * g.expert_rows + o - slot * g.expert_rows;
     };
     const int iters = groups * chunks;
 
@@ -122,29 +122,32 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
         // ------------------------------------------------------------ producer --
         if (ROUTE != ROUTE_NONE) named_bar_sync(2, 64);              // the choice is in ids_s
         if (elect_one()) {
-            int slot = 0, c = 0, gi = 0;
+            int slot = 0, c = 0, gi = 0, piece = 0, part = 0, first = 0, second_first = 0;
             uint32_t phase = 0;
             for (int it = 0; it < iters; ++it) {
                 if (it >= g.stages && !mbar_wait_bounded(&empty[slot], phase, abort_flag)) break;
                 uint8_t* dst = ring + (size_t)slot * GV_STAGE;
                 const int o0 = group_first(gi);
-                const int part = ROUTE == ROUTE_COLUMNS ? c / pieces : 0, piece = c - part * pieces;
-                // a full group's four rows lie together: an expert's rows are a multiple of 16
-                if (gi < g.rounds && it >= g.stages) {
+                if (c == 0) { first = physical(o0); second_first = physical(stream + o0); }
+                const int matrix = ROUTE == ROUTE_COLUMNS ? ids_s[part] * g.expert_rows : 0;
+                // a full group's four rows lie together: an expert's rows are a multiple of 16.  Routed products have nothing to gain
+                // from row copies: by the time the choice is known the map has been fetched.
+                if (gi < g.rounds && (it >= g.stages || ROUTE != ROUTE_NONE)) {
                     mbar_arrive_expect_tx(&full[slot], GV_STAGE);
-                    tma_load_2d(dst, &g.w_map, piece * (GV_PIECE / 8), physical(o0, part), &full[slot]);
-                    tma_load_2d(dst + OUT_ROWS * GV_PIECE, &g.w_map, piece * (GV_PIECE / 8), physical(stream + o0, part), &full[slot]);
+                    tma_load_2d(dst, &g.w_map, piece * (GV_PIECE / 8), matrix + first, &full[slot]);
+                    tma_load_2d(dst + OUT_ROWS * GV_PIECE, &g.w_map, piece * (GV_PIECE / 8), matrix + second_first, &full[slot]);
                 } else {
                     const int bytes = min(GV_PIECE, row_bytes - piece * GV_PIECE), valid = group_rows(gi), second = second_rows(gi);
                     mbar_arrive_expect_tx(&full[slot], (uint32_t)bytes * (uint32_t)(valid + second));
                     const uint8_t* src = reinterpret_cast<const uint8_t*>(g.w) + (size_t)piece * GV_PIECE;
                     for (int r = 0; r < valid; ++r)
-                        bulk_g2s(dst + r * GV_PIECE, src + (size_t)physical(o0 + r, part) * row_bytes, (uint32_t)bytes, &full[slot]);
+                        bulk_g2s(dst + r * GV_PIECE, src + (size_t)(matrix + physical(o0 + r)) * row_bytes, (uint32_t)bytes, &full[slot]);
                     for (int r = 0; r < second; ++r)
-                        bulk_g2s(dst + (r + OUT_ROWS) * GV_PIECE, src + (size_t)physical(stream + o0 + r, part) * row_bytes, (uint32_t)bytes,
+                        bulk_g2s(dst + (r + OUT_ROWS) * GV_PIECE, src + (size_t)(matrix + physical(stream + o0 + r)) * row_bytes, (uint32_t)bytes,
                                  &full[slot]);
                 }
-                if (++c == chunks) { c = 0; ++gi; }
+                if (++piece == pieces) { piece = 0; ++part; }
+                if (++c == chunks) { c = 0; part = 0; ++gi; }
                 if (++slot == g.stages) { slot = 0; if (it >= g.stages) phase ^= 1u; }
             }
         }

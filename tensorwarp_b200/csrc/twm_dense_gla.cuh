@@ -8,9 +8,9 @@
 //   gla_chunk_state_kernel  what each chunk adds to the state, all chunks at once
 //   gla_scan_kernel         the state ahead of every chunk, chunk by chunk, element by element
 //   gla_chunk_out_kernel    o, norm and gate, all chunks at once
-// Every factor with a decay is computed in FP32 and enters a warp-level MMA as a bf16 pair hi + lo.  The exponents are
-// taken against the first token of a 16-token block, so no factor exceeds 1; inside a block against its middle, which
-// is safe while eight steps stay within e^80, and token pair by token pair otherwise.
+// Every factor with a decay is computed in FP32 and enters a warp-level MMA as a bf16 pair hi + lo.  The scores inside a
+// chunk are one product, with the exponents taken against the chunk's middle token: safe while neither half of the
+// chunk decays by more than e^60; a chunk that does is scored token pair by token pair.
 // Everything else (FP32, wide heads): gla_rows_kernel walks the tokens one by one, gla_gate_kernel norms and gates.
 // Decoding: gla_decode_kernel.
 #pragma once
@@ -21,8 +21,8 @@
 namespace twm {
 namespace dense {
 
-constexpr int GLA_CHUNK = 64;
-constexpr float GLA_STEP_FLOOR = -10.0f;        // log decay of a step below which a block is done pair by pair
+constexpr int GLA_CHUNK = 64, GLA_MIDDLE = 31;
+constexpr float GLA_HALF_LIMIT = 60.0f;         // largest decay (its logarithm) of half a chunk that goes through one product
 
 template <typename T>
 struct GlaArgs {
@@ -46,7 +46,15 @@ struct GlaArgs {
 };
 
 // A thread per key channel and run of up to 64 rows: log alpha = log(sigmoid(z)) / tau, summed up within chunks.
-constexpr int GD_THREADS = 128, GD_ROWS = 64, GD_RANK = 32;
+constexpr int GD_THREADS = 64, GD_ROWS = 64, GD_RANK = 32;
+// log(sigmoid(z)) to about 2^-22 of itself or 2e-7, whichever is larger
+__device__ __forceinline__ float log_sigmoid_fast(float z) {
+    const float e = ex2_approx(-1.4426950408889634f * fabsf(z));
+    const float near_one = e * fmaf(-e, fmaf(-e, fmaf(-e, 0.25f, 1.0f / 3.0f), 0.5f), 1.0f);      // log(1 + e) for small e
+    return fminf(z, 0.0f) - (e < 0.0078125f ? near_one : __logf(1.0f + e));
+}
+__device__ __forceinline__ float log_sigmoid_of(float z, float) { return log_sigmoid_f32(z); }
+__device__ __forceinline__ float log_sigmoid_of(float z, bf16) { return log_sigmoid_fast(z); }
 template <typename T>
 __global__ void __launch_bounds__(GD_THREADS)
 gla_decay_kernel(const GlaArgs<T> g)
@@ -88,7 +96,7 @@ gla_decay_kernel(const GlaArgs<T> g)
 #pragma unroll
     for (int r = 0; r < GD_ROWS; ++r) {
         if (r >= n) break;
-        const float la = log_sigmoid_f32(z[r]) * g.inv_tau;
+        const float la = log_sigmoid_of(z[r], T()) * g.inv_tau;
         sum = (r0 + r) % g.chunk == 0 ? la : sum + la;
         g.decay[(size_t)(r0 + r) * cols + col] = sum;
     }
@@ -168,8 +176,23 @@ gla_gate_kernel(const GlaArgs<T> g)
 }
 
 // ------------------------------------------------------------------ chunks --
-constexpr int GC_THREADS = 128;
+constexpr int GC_THREADS = 256;
 constexpr float GLA_LOG2E = 1.4426950408889634f;
+
+// eight values times 2^(e - f), as bf16 pairs hi + lo
+__device__ __forceinline__ void decayed8(const uint4& x, const float4& e0, const float4& e1, const float4& f0, const float4& f1, float factor,
+                                         uint4& hi, uint4& lo)
+{
+    float v[8];
+    Vec<bf16>::unpack(x, v);
+    const float e[8] = {e0.x, e0.y, e0.z, e0.w, e1.x, e1.y, e1.z, e1.w}, f[8] = {f0.x, f0.y, f0.z, f0.w, f1.x, f1.y, f1.z, f1.w};
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] *= factor * ex2_approx((e[i] - f[i]) * GLA_LOG2E);
+    split_bf16(v[0], v[1], hi.x, lo.x);
+    split_bf16(v[2], v[3], hi.y, lo.y);
+    split_bf16(v[4], v[5], hi.z, lo.z);
+    split_bf16(v[6], v[7], hi.w, lo.w);
+}
 
 // dS[d][v] = sum_t k_td e^{b_last,d - b_td} v_tv of one chunk and head.
 __host__ inline size_t gla_chunk_state_smem_bytes(int dim_pad, int vdim_pad) {
@@ -190,22 +213,23 @@ gla_chunk_state_kernel(const GlaArgs<bf16> g)
     pdl_launch_dependents();
     const bf16* row0 = g.proj + (size_t)r0 * g.ld;
     const float* b0 = g.decay + (size_t)r0 * cols + h * g.dim_pad;
-    for (int i = tid; i < GLA_CHUNK * (g.vdim_pad / 8); i += GC_THREADS) {
-        const int t = i / (g.vdim_pad / 8), c = i - t * (g.vdim_pad / 8);
+    const int kp = g.dim_pad / 8, vp = g.vdim_pad / 8;
+    for (int i = tid; i < GLA_CHUNK * vp; i += GC_THREADS) {
+        const int t = i / vp, c = i - t * vp;
         ops::att_cp_async16(smem_u32(vs + t * vrow + c * 16), row0 + (size_t)(t < n ? t : 0) * g.ld + g.v_off() + h * g.vdim_pad + c * 8, t < n ? 16 : 0);
     }
     ops::att_cp_async_commit();
-    for (int i = tid; i < GLA_CHUNK * (g.dim_pad / 4); i += GC_THREADS) {
-        const int t = i / (g.dim_pad / 4), d = (i - t * (g.dim_pad / 4)) * 4;
-        uint2 hi = make_uint2(0, 0), lo = make_uint2(0, 0);
+#pragma unroll 2
+    for (int i = tid; i < GLA_CHUNK * kp; i += GC_THREADS) {
+        const int t = i / kp, d = (i - t * kp) * 8;
+        uint4 hi = make_uint4(0, 0, 0, 0), lo = hi;
         if (t < n) {
-            const float4 k = load4(row0 + (size_t)t * g.ld + g.k_off() + h * g.dim_pad + d);
-            const float4 b = load4(b0 + (size_t)t * cols + d), last = load4(b0 + (size_t)(n - 1) * cols + d);
-            split_bf16(k.x * ex2_approx((last.x - b.x) * GLA_LOG2E), k.y * ex2_approx((last.y - b.y) * GLA_LOG2E), hi.x, lo.x);
-            split_bf16(k.z * ex2_approx((last.z - b.z) * GLA_LOG2E), k.w * ex2_approx((last.w - b.w) * GLA_LOG2E), hi.y, lo.y);
+            const float *b = b0 + (size_t)t * cols + d, *last = b0 + (size_t)(n - 1) * cols + d;
+            decayed8(*reinterpret_cast<const uint4*>(row0 + (size_t)t * g.ld + g.k_off() + h * g.dim_pad + d), load4(last), load4(last + 4), load4(b),
+                     load4(b + 4), 1.0f, hi, lo);
         }
-        *reinterpret_cast<uint2*>(khi + t * krow + d * 2) = hi;
-        *reinterpret_cast<uint2*>(klo + t * krow + d * 2) = lo;
+        *reinterpret_cast<uint4*>(khi + t * krow + d * 2) = hi;
+        *reinterpret_cast<uint4*>(klo + t * krow + d * 2) = lo;
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
@@ -288,228 +312,235 @@ gla_scan_kernel(const GlaArgs<T> g)
     *st = s;
 }
 
-// CTA = chunk and head; warp = 16 of its tokens.  DV: value columns the accumulators hold (>= vdim_pad).
-constexpr int GO_SROWS = 32;                               // state rows in shared memory at a time
+// CTA = chunk and head; a pair of warps = 16 of its tokens.  DV: value columns the accumulators hold (>= vdim_pad).
+constexpr int GO_AROW = GLA_CHUNK * 2 + 16;                // bytes of a row of scores
+__host__ __device__ inline int gla_out_row(int dim_pad, int vdim_pad) { return (dim_pad > vdim_pad ? dim_pad : vdim_pad) * 2 + 16; }
 __host__ inline size_t gla_chunk_out_smem_bytes(int dim_pad, int vdim_pad) {
-    return (size_t)GLA_CHUNK * (dim_pad * 2 + 16 + vdim_pad * 2 + 16) + (size_t)GLA_CHUNK * (dim_pad * 4 + 32) +
-           (size_t)2 * GO_SROWS * (vdim_pad * 2 + 16) + 4 * 256 * sizeof(float);
+    return (size_t)GLA_CHUNK * (2 * (dim_pad * 2 + 16) + 2 * gla_out_row(dim_pad, vdim_pad) + vdim_pad * 2 + 16 + 2 * GO_AROW) +
+           sizeof(float) * (size_t)(dim_pad + 2 * GLA_CHUNK);
 }
 template <int DV>
 __global__ void __launch_bounds__(GC_THREADS, 2)
 gla_chunk_out_kernel(const GlaArgs<bf16> g)
 {
     extern __shared__ __align__(16) uint8_t gc_smem[];
-    const int krow = g.dim_pad * 2 + 16, vrow = g.vdim_pad * 2 + 16, brow = g.dim_pad + 8;
-    uint8_t* ks = gc_smem;                                 // [64][dim_pad]
-    uint8_t* vs = ks + GLA_CHUNK * krow;                   // [64][vdim_pad]
-    float* bs = reinterpret_cast<float*>(vs + GLA_CHUNK * vrow);      // [64][dim_pad] running sums, in powers of two
-    uint8_t* shi = reinterpret_cast<uint8_t*>(bs + GLA_CHUNK * brow); // [GO_SROWS][vdim_pad]
-    uint8_t* slo = shi + GO_SROWS * vrow;
-    float* pairs = reinterpret_cast<float*>(slo + GO_SROWS * vrow);   // [4 warps][16][16]
+    const int krow = g.dim_pad * 2 + 16, vrow = g.vdim_pad * 2 + 16, wide = gla_out_row(g.dim_pad, g.vdim_pad);
+    uint8_t* qhi = gc_smem;                                // [64][dim_pad] q 2^(b_t - ref)
+    uint8_t* qlo = qhi + GLA_CHUNK * krow;
+    uint8_t* khi = qlo + GLA_CHUNK * krow;                 // [64][dim_pad] k 2^(ref - b_t); later 64 rows of the state
+    uint8_t* klo = khi + GLA_CHUNK * wide;
+    uint8_t* vs = klo + GLA_CHUNK * wide;                  // [64][vdim_pad]
+    uint8_t* ahi = vs + GLA_CHUNK * vrow;                  // [64][64] scores
+    uint8_t* alo = ahi + GLA_CHUNK * GO_AROW;
+    float* refs = reinterpret_cast<float*>(alo + GLA_CHUNK * GO_AROW);      // [dim_pad]: e^ref
+    float* sums = refs + g.dim_pad;                        // [2][64]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int h = blockIdx.y, r0 = blockIdx.x * GLA_CHUNK, n = min(GLA_CHUNK, g.rows - r0);
     const int cols = g.heads * g.dim_pad;
     pdl_wait_prior_grids();
     pdl_launch_dependents();
     const bf16* row0 = g.proj + (size_t)r0 * g.ld;
-    const int kp = g.dim_pad / 8, vp = g.vdim_pad / 8;
-    for (int i = tid; i < GLA_CHUNK * kp; i += GC_THREADS) {
-        const int t = i / kp, c = i - t * kp;
-        ops::att_cp_async16(smem_u32(ks + t * krow + c * 16), row0 + (size_t)(t < n ? t : 0) * g.ld + g.k_off() + h * g.dim_pad + c * 8, t < n ? 16 : 0);
-    }
+    const float* b0 = g.decay + (size_t)r0 * cols + h * g.dim_pad;
+    const int kp = g.dim_pad / 8, vp = g.vdim_pad / 8, middle = min(GLA_MIDDLE, n - 1);
     for (int i = tid; i < GLA_CHUNK * vp; i += GC_THREADS) {
         const int t = i / vp, c = i - t * vp;
         ops::att_cp_async16(smem_u32(vs + t * vrow + c * 16), row0 + (size_t)(t < n ? t : 0) * g.ld + g.v_off() + h * g.vdim_pad + c * 8, t < n ? 16 : 0);
     }
     ops::att_cp_async_commit();
-    // rows past the end repeat the last one: their weights are never used
     bool steep = false;
-    for (int i = tid; i < GLA_CHUNK * (g.dim_pad / 4); i += GC_THREADS) {
-        const int t = i / (g.dim_pad / 4), d = (i - t * (g.dim_pad / 4)) * 4;
-        const float* at = g.decay + (size_t)(r0 + min(t, n - 1)) * cols + h * g.dim_pad + d;
-        const float4 b = load4(at);
-        if (t > 0 && t < n) {
-            const float4 p = load4(at - cols);
-            steep = steep || fminf(fminf(b.x - p.x, b.y - p.y), fminf(b.z - p.z, b.w - p.w)) < GLA_STEP_FLOOR;
+    for (int d = tid; d < g.dim_pad; d += GC_THREADS) {
+        const float first = b0[d], mid = b0[(size_t)middle * cols + d], last = b0[(size_t)(n - 1) * cols + d];
+        steep = steep || first - mid > GLA_HALF_LIMIT || mid - last > GLA_HALF_LIMIT;
+        refs[d] = mid;
+    }
+    steep = __syncthreads_or(steep);
+    const float4 zero4 = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 2
+    for (int i = tid; i < GLA_CHUNK * kp; i += GC_THREADS) {
+        const int t = i / kp, d = (i - t * kp) * 8;
+        uint4 qh = make_uint4(0, 0, 0, 0), ql = qh, kh = qh, kl = qh;
+        if (t < n) {
+            const bf16* row = row0 + (size_t)t * g.ld + h * g.dim_pad + d;
+            const uint4 q = *reinterpret_cast<const uint4*>(row), k = *reinterpret_cast<const uint4*>(row + g.k_off());
+            const float4 e0 = load4(b0 + (size_t)t * cols + d), e1 = load4(b0 + (size_t)t * cols + d + 4);
+            const float4 f0 = steep ? zero4 : load4(refs + d), f1 = steep ? zero4 : load4(refs + d + 4);
+            decayed8(q, e0, e1, f0, f1, g.q_scale, qh, ql);
+            if (!steep) decayed8(k, f0, f1, e0, e1, 1.0f, kh, kl);
         }
-        *reinterpret_cast<float4*>(bs + t * brow + d) = make_float4(b.x * GLA_LOG2E, b.y * GLA_LOG2E, b.z * GLA_LOG2E, b.w * GLA_LOG2E);
+        *reinterpret_cast<uint4*>(qhi + t * krow + d * 2) = qh;
+        *reinterpret_cast<uint4*>(qlo + t * krow + d * 2) = ql;
+        *reinterpret_cast<uint4*>(khi + t * wide + d * 2) = kh;
+        *reinterpret_cast<uint4*>(klo + t * wide + d * 2) = kl;
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
-    steep = __syncthreads_or(steep);
+    __syncthreads();
+    // state rows on their way: 64 x vdim_pad, four columns at a time
+    const float* st = g.chunk_state + ((size_t)blockIdx.x * g.heads + h) * g.dim_pad * g.vdim_pad;
+    constexpr int SV = DV / 16;
+    float4 sv[SV];
+    auto load_state = [&](int d0) {
+        const int count = min(GLA_CHUNK, g.dim_pad - d0) * (g.vdim_pad / 4);
+#pragma unroll
+        for (int j = 0; j < SV; ++j) {
+            const int i = tid + j * GC_THREADS;
+            if (i < count) sv[j] = load4(st + (size_t)d0 * g.vdim_pad + i * 4);
+        }
+    };
+    load_state(0);
 
-    const int t_lo = warp * 16 + (lane >> 2), t_hi = t_lo + 8, d_in = (lane & 3) * 2;
-    const bf16* q_lo = row0 + (size_t)min(t_lo, n - 1) * g.ld + h * g.dim_pad;
-    const bf16* q_hi = row0 + (size_t)min(t_hi, n - 1) * g.ld + h * g.dim_pad;
-    auto pair_f32 = [](uint32_t w) { return make_float2(__uint_as_float(w << 16), __uint_as_float(w & 0xffff0000u)); };
-    // the warp's queries at channels d, d + 1 of rows t_lo or t_hi, times 2^(b_t - ref)
-    auto q_pair = [&](const bf16* q, int t, int d, float2 ref, uint32_t& hi, uint32_t& lo) {
-        const float2 x = pair_f32(*reinterpret_cast<const uint32_t*>(q + d));
-        const float2 b = *reinterpret_cast<const float2*>(bs + t * brow + d);
-        split_bf16(x.x * g.q_scale * ex2_approx(b.x - ref.x), x.y * g.q_scale * ex2_approx(b.y - ref.y), hi, lo);
-    };
-    auto q_frag = [&](int d0, float2 ref0, float2 ref8, uint32_t (&hi)[4], uint32_t (&lo)[4]) {
-        q_pair(q_lo, t_lo, d0 + d_in, ref0, hi[0], lo[0]);
-        q_pair(q_hi, t_hi, d0 + d_in, ref0, hi[1], lo[1]);
-        q_pair(q_lo, t_lo, d0 + d_in + 8, ref8, hi[2], lo[2]);
-        q_pair(q_hi, t_hi, d0 + d_in + 8, ref8, hi[3], lo[3]);
-    };
-    auto k_pair = [&](int s, int d, float2 ref, uint32_t& hi, uint32_t& lo) {
-        const float2 x = pair_f32(*reinterpret_cast<const uint32_t*>(ks + s * krow + d * 2));
-        const float2 b = *reinterpret_cast<const float2*>(bs + s * brow + d);
-        split_bf16(x.x * ex2_approx(ref.x - b.x), x.y * ex2_approx(ref.y - b.y), hi, lo);
-    };
-    // scores of the warp's 16 tokens against 16 tokens from s0, exponents against row `ref`
-    float a[4][2][4];
+    const int block = warp >> 1, half = warp & 1;          // this warp's 16 tokens; which 32 tokens they are scored against, which columns
+    const uint32_t q_at = (uint32_t)((block * 16 + (lane & 15)) * krow + (lane >> 4) * 16);
+    if (!steep) {
+        if (half * 32 <= block * 16 + 15) {
+            float a[4][4];
 #pragma unroll
-    for (int j = 0; j < 4; ++j)
+            for (int j = 0; j < 4; ++j)
 #pragma unroll
-        for (int i = 0; i < 2; ++i)
+                for (int e = 0; e < 4; ++e) a[j][e] = 0.0f;
+            const uint32_t k_at = (uint32_t)((half * 32 + (lane & 7) + (lane >> 4) * 8) * wide + ((lane >> 3) & 1) * 16);
+            for (int c = 0; c < g.dim_pad / 16; ++c) {
+                uint32_t qh[4], ql[4];
+                ldmatrix_x4(qh, smem_u32(qhi) + q_at + c * 32);
+                ldmatrix_x4(ql, smem_u32(qlo) + q_at + c * 32);
 #pragma unroll
-            for (int e = 0; e < 4; ++e) a[j][i][e] = 0.0f;
-    auto against = [&](int d0, const uint32_t (&qh)[4], const uint32_t (&ql)[4], int s0, float2 ref0, float2 ref8, float (&acc)[2][4]) {
+                for (int j = 0; j < 2; ++j) {
+                    if (half * 32 + j * 16 > block * 16) continue;
+                    uint32_t kh[4], kl[4];
+                    ldmatrix_x4(kh, smem_u32(khi) + k_at + j * 16 * wide + c * 32);
+                    ldmatrix_x4(kl, smem_u32(klo) + k_at + j * 16 * wide + c * 32);
 #pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            const int s = s0 + i * 8 + (lane >> 2);
-            uint32_t h0, l0, h1, l1;
-            k_pair(s, d0 + d_in, ref0, h0, l0);
-            k_pair(s, d0 + d_in + 8, ref8, h1, l1);
-            mma_bf16(acc[i], qh, h0, h1);
-            mma_bf16(acc[i], ql, h0, h1);
-            mma_bf16(acc[i], qh, l0, l1);
+                    for (int i = 0; i < 2; ++i) {
+                        mma_bf16(a[2 * j + i], qh, kh[2 * i], kh[2 * i + 1]);
+                        mma_bf16(a[2 * j + i], ql, kh[2 * i], kh[2 * i + 1]);
+                        mma_bf16(a[2 * j + i], qh, kl[2 * i], kl[2 * i + 1]);
+                    }
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    const int t = block * 16 + (lane >> 2) + i * 8, s = half * 32 + j * 8 + (lane & 3) * 2;
+                    uint32_t hi, lo;
+                    split_bf16(s <= t ? a[j][2 * i] : 0.0f, s + 1 <= t ? a[j][2 * i + 1] : 0.0f, hi, lo);
+                    *reinterpret_cast<uint32_t*>(ahi + t * GO_AROW + s * 2) = hi;
+                    *reinterpret_cast<uint32_t*>(alo + t * GO_AROW + s * 2) = lo;
+                }
         }
-    };
-    auto ref_at = [&](int t, int d) { return *reinterpret_cast<const float2*>(bs + t * brow + d); };
-    for (int d0 = 0; d0 < g.dim_pad; d0 += 16) {
-        uint32_t qh[4], ql[4];
-        if (warp > 0) {
-            const int t = warp * 16 - 1;
-            const float2 r0_ = ref_at(t, d0 + d_in), r8_ = ref_at(t, d0 + d_in + 8);
-            q_frag(d0, r0_, r8_, qh, ql);
-#pragma unroll
-            for (int j = 0; j < 3; ++j)
-                if (j < warp) against(d0, qh, ql, j * 16, r0_, r8_, a[j]);
-        }
-        if (!steep) {
-            const int t = warp * 16 + 7;
-            const float2 r0_ = ref_at(t, d0 + d_in), r8_ = ref_at(t, d0 + d_in + 8);
-            q_frag(d0, r0_, r8_, qh, ql);
-            against(d0, qh, ql, warp * 16, r0_, r8_, a[3]);
-        }
-    }
-    if (steep) {                                           // the block's own pairs one by one
-        float* mine = pairs + warp * 256;
-        for (int i = 0; i < 16; ++i)
-            for (int j = 0; j <= i; ++j) {
-                const int t = warp * 16 + i, s = warp * 16 + j;
-                float sum = 0.0f;
+    } else {                                               // a warp per token pair
+        for (int u = warp; u < GLA_CHUNK * GLA_CHUNK; u += GC_THREADS / 32) {
+            const int t = u / GLA_CHUNK, s = u - t * GLA_CHUNK;
+            float sum = 0.0f;
+            if (s <= t && t < n)
                 for (int d = lane; d < g.dim_pad; d += 32)
-                    sum = fmaf(to_f32(row0[(size_t)min(t, n - 1) * g.ld + h * g.dim_pad + d]) * g.q_scale *
-                                   to_f32(reinterpret_cast<const bf16*>(ks + s * krow)[d]),
-                               ex2_approx(bs[t * brow + d] - bs[s * brow + d]), sum);
-                sum = ops::warp_sum(sum);
-                if (lane == 0) mine[i * 16 + j] = sum;
+                    sum = fmaf(to_f32(row0[(size_t)t * g.ld + h * g.dim_pad + d]) * g.q_scale * to_f32(row0[(size_t)s * g.ld + g.k_off() + h * g.dim_pad + d]),
+                               ex2_approx((b0[(size_t)t * cols + d] - b0[(size_t)s * cols + d]) * GLA_LOG2E), sum);
+            sum = ops::warp_sum(sum);
+            const bf16 hi = __float2bfloat16_rn(sum);
+            if (lane == 0) {
+                reinterpret_cast<bf16*>(ahi + t * GO_AROW)[s] = hi;
+                reinterpret_cast<bf16*>(alo + t * GO_AROW)[s] = __float2bfloat16_rn(sum - to_f32(hi));
             }
-        __syncwarp();
-#pragma unroll
-        for (int i = 0; i < 2; ++i)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int t = (lane >> 2) + (e >> 1) * 8, s = i * 8 + d_in + (e & 1);
-                a[3][i][e] = s <= t ? mine[t * 16 + s] : 0.0f;
-            }
+        }
     }
-    // ---- o = scores V + (q 2^b) S ----
-    float o[DV / 8][4];
+    __syncthreads();                                       // the scores are there, the keys have been used
+
+    // ---- o = scores V + (q 2^(b - ref)) (2^ref S): the warp takes every other 16 value columns ----
+    float o[DV / 16][4];
 #pragma unroll
-    for (int j = 0; j < DV / 8; ++j)
+    for (int j = 0; j < DV / 16; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) o[j][e] = 0.0f;
-    auto times_v = [&](float (&x)[2][4], int s0) {
-        uint32_t hi[4], lo[4];
-        split_bf16(x[0][0], x[0][1], hi[0], lo[0]);
-        split_bf16(x[0][2], x[0][3], hi[1], lo[1]);
-        split_bf16(x[1][0], x[1][1], hi[2], lo[2]);
-        split_bf16(x[1][2], x[1][3], hi[3], lo[3]);
+    auto store_state = [&](int d0) {
+        const int vq = g.vdim_pad / 4, count = min(GLA_CHUNK, g.dim_pad - d0) * vq;
 #pragma unroll
-        for (int j = 0; j < DV / 16; ++j) {
-            if (j * 16 >= g.vdim_pad) continue;
-            uint32_t b[4];
-            ops::att_ldmatrix_x4_trans(b, smem_u32(vs) + (s0 + (lane & 15)) * vrow + (j * 16 + (lane >> 4) * 8) * 2);
-            mma_bf16(o[2 * j], hi, b[0], b[1]);
-            mma_bf16(o[2 * j + 1], hi, b[2], b[3]);
-            mma_bf16(o[2 * j], lo, b[0], b[1]);
-            mma_bf16(o[2 * j + 1], lo, b[2], b[3]);
+        for (int j = 0; j < SV; ++j) {
+            const int i = tid + j * GC_THREADS;
+            if (i >= count) continue;
+            const int d = i / vq, v = (i - d * vq) * 4;
+            const float f = steep ? 1.0f : ex2_approx(refs[d0 + d] * GLA_LOG2E);
+            uint2 hi, lo;
+            split_bf16(sv[j].x * f, sv[j].y * f, hi.x, lo.x);
+            split_bf16(sv[j].z * f, sv[j].w * f, hi.y, lo.y);
+            *reinterpret_cast<uint2*>(khi + d * wide + v * 2) = hi;
+            *reinterpret_cast<uint2*>(klo + d * wide + v * 2) = lo;
         }
     };
+    store_state(0);
+    const uint32_t a_at = (uint32_t)((block * 16 + (lane & 15)) * GO_AROW + (lane >> 4) * 16);
+    for (int kk = 0; kk <= block; ++kk) {
+        uint32_t xh[4], xl[4];
+        ldmatrix_x4(xh, smem_u32(ahi) + a_at + kk * 32);
+        ldmatrix_x4(xl, smem_u32(alo) + a_at + kk * 32);
 #pragma unroll
-    for (int j = 0; j < 3; ++j)
-        if (j < warp) times_v(a[j], j * 16);
-#pragma unroll
-    for (int i = 0; i < 2; ++i)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int t = (lane >> 2) + (e >> 1) * 8, s = i * 8 + d_in + (e & 1);
-            if (s > t) a[3][i][e] = 0.0f;
+        for (int j = 0; j < DV / 32; ++j) {
+            const int v0 = (2 * j + half) * 16;
+            if (v0 >= g.vdim_pad) continue;
+            uint32_t b[4];
+            ops::att_ldmatrix_x4_trans(b, smem_u32(vs) + (kk * 16 + (lane & 15)) * vrow + (v0 + (lane >> 4) * 8) * 2);
+            mma_bf16(o[2 * j], xh, b[0], b[1]);
+            mma_bf16(o[2 * j + 1], xh, b[2], b[3]);
+            mma_bf16(o[2 * j], xl, b[0], b[1]);
+            mma_bf16(o[2 * j + 1], xl, b[2], b[3]);
         }
-    times_v(a[3], warp * 16);
-    const float* st = g.chunk_state + ((size_t)blockIdx.x * g.heads + h) * g.dim_pad * g.vdim_pad;
-    const float2 zero2 = make_float2(0.0f, 0.0f);
-    for (int d0 = 0; d0 < g.dim_pad; d0 += GO_SROWS) {
-        const int dn = min(GO_SROWS, g.dim_pad - d0);
-        __syncthreads();                                   // the rows before have been used
-        for (int i = tid; i < dn * (g.vdim_pad / 4); i += GC_THREADS) {
-            const int d = i / (g.vdim_pad / 4), v = (i - d * (g.vdim_pad / 4)) * 4;
-            const float4 x = load4(st + (size_t)(d0 + d) * g.vdim_pad + v);
-            uint2 hi, lo;
-            split_bf16(x.x, x.y, hi.x, lo.x);
-            split_bf16(x.z, x.w, hi.y, lo.y);
-            *reinterpret_cast<uint2*>(shi + d * vrow + v * 2) = hi;
-            *reinterpret_cast<uint2*>(slo + d * vrow + v * 2) = lo;
-        }
-        __syncthreads();
-        for (int dk = 0; dk < dn; dk += 16) {
+    }
+    for (int d0 = 0; d0 < g.dim_pad; d0 += GLA_CHUNK) {
+        __syncthreads();                                   // this part of the state is in shared memory
+        if (d0 + GLA_CHUNK < g.dim_pad) load_state(d0 + GLA_CHUNK);
+        const int steps = min(GLA_CHUNK, g.dim_pad - d0) / 16;
+        for (int c = 0; c < steps; ++c) {
             uint32_t qh[4], ql[4];
-            q_frag(d0 + dk, zero2, zero2, qh, ql);
+            ldmatrix_x4(qh, smem_u32(qhi) + q_at + (d0 + c * 16) * 2);
+            ldmatrix_x4(ql, smem_u32(qlo) + q_at + (d0 + c * 16) * 2);
 #pragma unroll
-            for (int j = 0; j < DV / 16; ++j) {
-                if (j * 16 >= g.vdim_pad) continue;
-                const uint32_t at = (uint32_t)((dk + (lane & 15)) * vrow + (j * 16 + (lane >> 4) * 8) * 2);
+            for (int j = 0; j < DV / 32; ++j) {
+                const int v0 = (2 * j + half) * 16;
+                if (v0 >= g.vdim_pad) continue;
+                const uint32_t at = (uint32_t)((c * 16 + (lane & 15)) * wide + (v0 + (lane >> 4) * 8) * 2);
                 uint32_t bh[4], bl[4];
-                ops::att_ldmatrix_x4_trans(bh, smem_u32(shi) + at);
-                ops::att_ldmatrix_x4_trans(bl, smem_u32(slo) + at);
-                mma_bf16(o[2 * j], qh, bh[0], bh[1]);
-                mma_bf16(o[2 * j + 1], qh, bh[2], bh[3]);
-                mma_bf16(o[2 * j], ql, bh[0], bh[1]);
-                mma_bf16(o[2 * j + 1], ql, bh[2], bh[3]);
-                mma_bf16(o[2 * j], qh, bl[0], bl[1]);
-                mma_bf16(o[2 * j + 1], qh, bl[2], bl[3]);
+                ops::att_ldmatrix_x4_trans(bh, smem_u32(khi) + at);
+                ops::att_ldmatrix_x4_trans(bl, smem_u32(klo) + at);
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    mma_bf16(o[2 * j + i], qh, bh[2 * i], bh[2 * i + 1]);
+                    mma_bf16(o[2 * j + i], ql, bh[2 * i], bh[2 * i + 1]);
+                    mma_bf16(o[2 * j + i], qh, bl[2 * i], bl[2 * i + 1]);
+                }
             }
+        }
+        if (d0 + GLA_CHUNK < g.dim_pad) {
+            __syncthreads();                               // the part before has been used
+            store_state(d0 + GLA_CHUNK);
         }
     }
     // ---- norm over the head's columns, gate, store ----
-    float ss[2] = {0.0f, 0.0f};
-#pragma unroll
-    for (int j = 0; j < DV / 8; ++j) {
-        ss[0] = fmaf(o[j][0], o[j][0], fmaf(o[j][1], o[j][1], ss[0]));
-        ss[1] = fmaf(o[j][2], o[j][2], fmaf(o[j][3], o[j][3], ss[1]));
-    }
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
-        ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], 1);
-        ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], 2);
-        const int t = i == 0 ? t_lo : t_hi;
+        float ss = 0.0f;
+#pragma unroll
+        for (int j = 0; j < DV / 16; ++j) ss = fmaf(o[j][2 * i], o[j][2 * i], fmaf(o[j][2 * i + 1], o[j][2 * i + 1], ss));
+        ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+        ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+        if ((lane & 3) == 0) sums[half * GLA_CHUNK + block * 16 + (lane >> 2) + i * 8] = ss;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        const int t = block * 16 + (lane >> 2) + i * 8;
         if (t >= n) continue;
-        const float ir = inv_rms(ss[i], g.vdim, g.eps);
+        const float ir = inv_rms(sums[t] + sums[GLA_CHUNK + t], g.vdim, g.eps);
         const bf16* gate = row0 + (size_t)t * g.ld + g.gate_off() + h * g.vdim_pad;
         bf16* out = g.out + ((size_t)(r0 + t) * g.heads + h) * g.vdim_pad;
 #pragma unroll
-        for (int j = 0; j < DV / 8; ++j) {
-            const int v = j * 8 + d_in;
-            if (j * 8 >= g.vdim_pad) continue;
+        for (int j = 0; j < DV / 16; ++j) {
+            const int v = (2 * (j >> 1) + half) * 16 + (j & 1) * 8 + (lane & 3) * 2;
+            if (v >= g.vdim_pad) continue;
             const float2 w = *reinterpret_cast<const float2*>(g.head_norm + v);
-            const float2 z = pair_f32(*reinterpret_cast<const uint32_t*>(gate + v));
+            const uint32_t z = *reinterpret_cast<const uint32_t*>(gate + v);
+            const float z0 = __uint_as_float(z << 16), z1 = __uint_as_float(z & 0xffff0000u);
             *reinterpret_cast<__nv_bfloat162*>(out + v) =
-                __floats2bfloat162_rn(o[j][2 * i] * ir * w.x * silu_f32(z.x), o[j][2 * i + 1] * ir * w.y * silu_f32(z.y));
+                __floats2bfloat162_rn(o[j][2 * i] * ir * w.x * z0 * rcp_approx(1.0f + ex2_approx(-GLA_LOG2E * z0)),
+                                      o[j][2 * i + 1] * ir * w.y * z1 * rcp_approx(1.0f + ex2_approx(-GLA_LOG2E * z1)));
         }
     }
 }
@@ -562,6 +593,12 @@ gla_decode_kernel(const GlaDecodeArgs<T> g)
     for (int i = 0; i < WV; ++i)
         wv[i] = tid < g.dim_pad && i * V::N < g.rank_pad ? __ldg(reinterpret_cast<const uint4*>(g.w_decay + (size_t)(h * g.dim_pad + tid) * g.rank_pad) + i)
                                                          : make_uint4(0, 0, 0, 0);
+    {   // the state's share into L2; the slot as it is now (a stale one prefetches another sequence's)
+        const float* st_now = g.state + ((size_t)*(volatile const int*)(g.meta + 1) * g.heads + h) * g.dim_pad * g.vdim_pad + rank * share;
+        if (rank * share < g.vdim_pad)
+            for (int d = tid; d < g.dim_pad; d += GX_THREADS)
+                for (int c = 0; c < share; c += 32) l2_prefetch(st_now + (size_t)d * g.vdim_pad + c);
+    }
     pdl_wait_prior_grids();
     const float* low = g.proj + 2 * kd + 2 * vd;
     for (int d = tid; d < g.dim_pad; d += GX_THREADS) {

@@ -196,8 +196,8 @@ __host__ inline int latent_decode_parts(int rank_pad) {
 }
 // floats in front of the token rows
 __host__ __device__ inline int latent_decode_floats(int dim_pad, int rot_pad, int rank_pad, int chunk, int parts, int splits) {
-    const int slice = latent_decode_slice(rank_pad, splits), width = rank_pad + rot_pad;
-    const int absorb = LD_THREADS * 8 + 0 * slice;          // partial sums of the query's map: at most 8 columns a thread
+    const int width = rank_pad + rot_pad;
+    const int absorb = LD_THREADS * 8;                      // partial sums of the query's map: at most 8 columns a thread
     const int share = parts * rank_pad > absorb ? parts * rank_pad : absorb;
     return dim_pad + width + chunk + share + splits * rank_pad + 2 * LD_MAX_SPLITS;
 }
@@ -233,6 +233,25 @@ latent_decode_kernel(const LatentDecodeArgs<T> g)
     uint8_t* rows = reinterpret_cast<uint8_t*>(recv_ml + 2 * LD_MAX_SPLITS);
     const int row_bytes = width * (int)sizeof(T), stride = row_bytes + 16;     // a padded row: keys start in distinct banks
     const int pieces = row_bytes / 16;
+    // What this CTA will read, into L2 while the kernel before runs.  Position and slot are read as they are now: a stale one
+    // prefetches other rows of the cache.
+    const int first = rank * slice, own = min(slice, g.rank_pad - first);          // this CTA's latent columns; own may be <= 0
+    const int per_cta = (g.vdim_pad + splits - 1) / splits;
+    const T* w_uk = g.w_expand + (size_t)h * g.dim_pad * g.rank_pad + first;
+    const T* w_uv = g.w_expand + (size_t)g.heads * g.dim_pad * g.rank_pad + (size_t)h * g.vdim_pad * g.rank_pad;
+    if (own > 0)
+        for (int i = tid; i < g.dim_pad; i += LD_THREADS)
+            for (int c = 0; c < own * (int)sizeof(T); c += 128) l2_prefetch(reinterpret_cast<const uint8_t*>(w_uk + (size_t)i * g.rank_pad) + c);
+    for (int e = rank * per_cta + tid; e < min(g.vdim_pad, (rank + 1) * per_cta); e += LD_THREADS)
+        l2_prefetch_bulk(w_uv + (size_t)e * g.rank_pad, (uint32_t)(g.rank_pad * sizeof(T)));
+    if (h == 0) {
+        const int now = min(max(*(volatile const int*)g.meta, 0), g.capacity - 1), from = max(0, now - g.window + 1), share_now = (now - from) / splits + 1;
+        const T* rows_now = g.cache + (size_t)*(volatile const int*)(g.meta + 1) * g.capacity * width;
+        for (int i = tid; i < share_now; i += LD_THREADS) {
+            const int j = from + rank * share_now + i;
+            if (j < now) l2_prefetch_bulk(rows_now + (size_t)j * width, (uint32_t)row_bytes);
+        }
+    }
     pdl_wait_prior_grids();
     const int p = g.meta[0];
     T* cache = g.cache + (size_t)g.meta[1] * g.capacity * width;
@@ -260,7 +279,6 @@ latent_decode_kernel(const LatentDecodeArgs<T> g)
     __syncthreads();
     asm volatile("barrier.cluster.wait.aligned;" ::: "memory");    // every CTA of the cluster has started
     {
-        const int first = rank * slice, own = min(slice, g.rank_pad - first);          // columns; own may be <= 0
         const int vecs = own > 0 ? (own + V::N - 1) / V::N : 1;
         const int vpp = min(vecs, LD_THREADS);                     // column vectors at a time
         const int groups = max(1, LD_THREADS / vpp);
@@ -268,7 +286,7 @@ latent_decode_kernel(const LatentDecodeArgs<T> g)
             const int vi = v0 + tid % vpp, dg = tid / vpp;
             float acc[V::N] = {};
             if (dg < groups && vi < vecs) {
-                const T* w = g.w_expand + (size_t)h * g.dim_pad * g.rank_pad + first + vi * V::N;
+                const T* w = w_uk + vi * V::N;
 #pragma unroll 4
                 for (int d = dg; d < g.dim_pad; d += groups) {
                     float f[V::N];
@@ -401,8 +419,6 @@ latent_decode_kernel(const LatentDecodeArgs<T> g)
     }
     __syncthreads();
     const float gate = sigmoid_f32(g.proj[g.heads * qw + width + h]);
-    const int per_cta = (g.vdim_pad + splits - 1) / splits;
-    const T* w_uv = g.w_expand + (size_t)g.heads * g.dim_pad * g.rank_pad + (size_t)h * g.vdim_pad * g.rank_pad;
     for (int e = rank * per_cta + warp; e < min(g.vdim_pad, (rank + 1) * per_cta); e += LD_THREADS / 32) {
         float s = 0.0f;
         for (int c = lane; c < g.rank_pad / V::N; c += 32) {

@@ -12,13 +12,78 @@ constexpr int MOE_MAX_EXPERTS = 1024, MOE_MAX_TOP = 32;
 
 struct RouterArgs { int experts, top, groups, keep; };
 
-// (value, index) of the largest value over the warp; the smaller index wins a tie
-__device__ __forceinline__ void warp_argmax(float& v, int& i) {
+// The largest of the lanes' N values each (value j of a lane stands for index lane + 32 j; negative = not there): its index,
+// the smallest on a tie, and in `best` its value; its owner's copy becomes negative.
+template <int N>
+__device__ __forceinline__ int warp_take_largest(float (&v)[N], int lane, float& best) {
+    unsigned top = 0;
+    int at = 0;
 #pragma unroll
-    for (int d = 16; d > 0; d >>= 1) {
-        const float ov = __shfl_xor_sync(0xffffffffu, v, d);
-        const int oi = __shfl_xor_sync(0xffffffffu, i, d);
-        if (ov > v || (ov == v && oi < i)) { v = ov; i = oi; }
+    for (int j = 0; j < N; ++j) {
+        const unsigned key = v[j] < 0.0f ? 0u : __float_as_uint(v[j]) + 1u;      // scores are not negative: their bits sort as they do
+        if (key > top) { top = key; at = lane + 32 * j; }
+    }
+    const unsigned all = __reduce_max_sync(0xffffffffu, top);
+    const int index = (int)__reduce_min_sync(0xffffffffu, top == all ? (unsigned)at : 0x7fffffffu);
+#pragma unroll
+    for (int j = 0; j < N; ++j)
+        if (index == lane + 32 * j) v[j] = -1.0f;
+    best = __uint_as_float(all - 1u);
+    return index;
+}
+
+template <int N>
+__device__ __forceinline__ void route_values(const float* logits, const RouterArgs& r, float* s, float* gs, int lane, int& id, float& weight)
+{
+    float v[N], m = -INFINITY, sum = 0.0f;
+#pragma unroll
+    for (int j = 0; j < N; ++j) {
+        const int e = lane + 32 * j;
+        v[j] = e < r.experts ? logits[e] : -INFINITY;
+        m = fmaxf(m, v[j]);
+    }
+    m = ops::warp_max(m);
+#pragma unroll
+    for (int j = 0; j < N; ++j) {
+        v[j] = expf(v[j] - m);
+        sum += v[j];
+    }
+    sum = ops::warp_sum(sum);
+#pragma unroll
+    for (int j = 0; j < N; ++j) v[j] = lane + 32 * j < r.experts ? v[j] / sum : -1.0f;
+    if (r.keep < r.groups) {
+        const int per = r.experts / r.groups;
+#pragma unroll
+        for (int j = 0; j < N; ++j)
+            if (lane + 32 * j < r.experts) s[lane + 32 * j] = v[j];
+        __syncwarp();
+        float best[N];
+#pragma unroll
+        for (int j = 0; j < N; ++j) {
+            const int g = lane + 32 * j;
+            best[j] = -1.0f;
+            if (g < r.groups) {
+                for (int e = 0; e < per; ++e) best[j] = fmaxf(best[j], s[g * per + e]);
+                gs[g] = 0.0f;
+            }
+        }
+        __syncwarp();
+        for (int k = 0; k < r.keep; ++k) {
+            float unused;
+            const int g = warp_take_largest<N>(best, lane, unused);
+            if (lane == 0) gs[g] = 1.0f;
+        }
+        __syncwarp();
+#pragma unroll
+        for (int j = 0; j < N; ++j)
+            if (lane + 32 * j < r.experts && gs[(lane + 32 * j) / per] == 0.0f) v[j] = -1.0f;
+    }
+    id = 0;
+    weight = 0.0f;
+    for (int k = 0; k < r.top; ++k) {
+        float best;
+        const int e = warp_take_largest<N>(v, lane, best);
+        if (lane == k) { id = e < r.experts ? e : 0; weight = best; }           // an index past the end: scores that are not numbers
     }
 }
 
@@ -27,51 +92,16 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
 // of shared memory.  Lane k < top returns choice k.
 __device__ __forceinline__ void route_warp(const float* logits, const RouterArgs& r, float* s, float* gs, int lane, int& id, float& weight)
 {
-    float m = -INFINITY;
-    for (int e = lane; e < r.experts; e += 32) { const float v = logits[e]; s[e] = v; m = fmaxf(m, v); }
-    m = ops::warp_max(m);
-    float sum = 0.0f;
-    for (int e = lane; e < r.experts; e += 32) { const float v = expf(s[e] - m); s[e] = v; sum += v; }
-    sum = ops::warp_sum(sum);
-    for (int e = lane; e < r.experts; e += 32) s[e] /= sum;
-    __syncwarp();
-    const int per = r.experts / r.groups;
-    const bool limited = r.keep < r.groups;
-    if (limited) {
-        for (int g = lane; g < r.groups; g += 32) {
-            float best = -1.0f;
-            for (int e = 0; e < per; ++e) best = fmaxf(best, s[g * per + e]);
-            gs[g] = best;
-        }
-        __syncwarp();
-        for (int k = 0; k < r.keep; ++k) {                  // a kept group's score becomes -1
-            float v = -2.0f;
-            int g = 0;
-            for (int i = lane; i < r.groups; i += 32)
-                if (gs[i] > v) { v = gs[i]; g = i; }
-            warp_argmax(v, g);
-            if (lane == 0) gs[g] = -1.0f;
-            __syncwarp();
-        }
-    }
-    id = 0;
-    weight = 0.0f;
-    for (int k = 0; k < r.top; ++k) {                       // a chosen expert's score becomes -1
-        float v = -2.0f;
-        int e = 0;
-        for (int i = lane; i < r.experts; i += 32)
-            if (s[i] > v && (!limited || gs[i / per] == -1.0f)) { v = s[i]; e = i; }
-        warp_argmax(v, e);
-        if (lane == k) { id = e; weight = v; }
-        __syncwarp();
-        if (lane == 0) s[e] = -1.0f;
-        __syncwarp();
-    }
+    if (r.experts <= 64) route_values<2>(logits, r, s, gs, lane, id, weight);
+    else if (r.experts <= 256) route_values<8>(logits, r, s, gs, lane, id, weight);
+    else route_values<MOE_MAX_EXPERTS / 32>(logits, r, s, gs, lane, id, weight);
 }
 
 // A warp per token: choices and weights [rows][top], and each choice's place among its expert's rows (in no
-// particular order: the rows of a product do not depend on one another).
-constexpr int RT_WARPS = 4;
+// particular order: the rows of a product do not depend on one another).  A CTA counts its tokens' choices itself and
+// asks for its places once per expert.
+constexpr int RT_WARPS = 16;
+__host__ __device__ inline size_t route_smem_bytes(const RouterArgs& r) { return sizeof(float) * (RT_WARPS * (size_t)(r.experts + r.groups) + 2 * (size_t)r.experts); }
 __global__ void __launch_bounds__(RT_WARPS * 32)
 route_kernel(const float* __restrict__ logits, int ld, const RouterArgs r, int rows, int* __restrict__ ids, float* __restrict__ weights,
              int* __restrict__ place, int* __restrict__ counts)
@@ -79,18 +109,29 @@ route_kernel(const float* __restrict__ logits, int ld, const RouterArgs r, int r
     extern __shared__ float route_smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     float* s = route_smem + warp * (r.experts + r.groups);
-    const int t = blockIdx.x * RT_WARPS + warp;
+    int* own = reinterpret_cast<int*>(route_smem + RT_WARPS * (r.experts + r.groups));      // [experts] this CTA's choices
+    int* base = own + r.experts;
+    for (int e = threadIdx.x; e < r.experts; e += RT_WARPS * 32) own[e] = 0;
     pdl_wait_prior_grids();
     pdl_launch_dependents();
-    if (t >= rows) return;
-    int id;
-    float weight;
-    route_warp(logits + (size_t)t * ld, r, s, s + r.experts, lane, id, weight);
-    if (lane < r.top) {
-        ids[t * r.top + lane] = id;
-        weights[t * r.top + lane] = weight;
-        if (counts != nullptr) place[t * r.top + lane] = atomicAdd(counts + id, 1);
+    __syncthreads();
+    const int t = blockIdx.x * RT_WARPS + warp;
+    int id = 0, rank = 0;
+    const bool valid = t < rows && lane < r.top;
+    if (t < rows) {
+        float weight;
+        route_warp(logits + (size_t)t * ld, r, s, s + r.experts, lane, id, weight);
+        if (valid) {
+            ids[t * r.top + lane] = id;
+            weights[t * r.top + lane] = weight;
+            rank = atomicAdd(own + id, 1);
+        }
     }
+    if (counts == nullptr) return;
+    __syncthreads();
+    for (int e = threadIdx.x; e < r.experts; e += RT_WARPS * 32) base[e] = own[e] > 0 ? atomicAdd(counts + e, own[e]) : 0;
+    __syncthreads();
+    if (valid) place[t * r.top + lane] = base[id] + rank;
 }
 
 // One warp: out[0 .. n] = running sums of f(0) ... f(n - 1)

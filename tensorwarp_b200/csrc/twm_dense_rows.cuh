@@ -48,7 +48,7 @@ struct ResidualSource {
         float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
         const int* at = routed.row + (size_t)r * routed.top;
         const float* w = routed.weight + (size_t)r * routed.top;
-#pragma unroll 4
+#pragma unroll 8
         for (int s = 0; s < routed.top; ++s) {
             const float4 t = load4(routed.rows + (size_t)at[s] * wp + i4 * 4);
             const float ws = w[s];
