@@ -581,15 +581,8 @@ GlaArgs<T> gla_args(const twm_dense_model* m, const twm_dense_layer& l, const tw
     g.proj = (const T*)b->proj; g.decay = b->decay; g.chunk_state = b->chunk_state; g.mix = b->mix; g.out = (T*)b->att; g.state = l.gla_state;
     g.w_decay = (const T*)l.w_decay; g.decay_bias = l.decay_bias; g.head_norm = l.head_norm; g.meta = b->meta;
     g.ld = sizes_of(l).in; g.heads = l.heads; g.dim_pad = l.dim_pad; g.vdim = l.vdim; g.vdim_pad = l.vdim_pad; g.rank_pad = l.rank_pad;
-    g.rows = rows; g.chunk = 1; g.inv_tau = l.inv_tau; g.q_scale = l.scale; g.eps = m->eps;
+    g.rows = rows; g.inv_tau = l.inv_tau; g.q_scale = l.scale; g.eps = m->eps;
     return g;
-}
-template <typename T>
-twm_status gla_decays(const GlaArgs<T>& g, int flags, void* stream)
-{
-    const int cols = g.heads * g.dim_pad;
-    return launch("gla_decay", gla_decay_kernel<T>, dim3((cols + GD_THREADS - 1) / GD_THREADS, (g.rows + GD_ROWS - 1) / GD_ROWS), GD_THREADS, 0,
-                  flags, stream, 0, g);
 }
 bool gla_chunks_fit(const GlaArgs<float>&) { return false; }
 bool gla_chunks_fit(const GlaArgs<bf16>& g)
@@ -598,11 +591,9 @@ bool gla_chunks_fit(const GlaArgs<bf16>& g)
            gla_chunk_state_smem_bytes(g.dim_pad, g.vdim_pad) <= kSmemLimit;
 }
 twm_status gla_chunks(const GlaArgs<float>&, int, void*) { return invalid("the chunked linear attention takes bfloat16"); }
-twm_status gla_chunks(GlaArgs<bf16> g, int flags, void* stream)
+twm_status gla_chunks(const GlaArgs<bf16>& g, int flags, void* stream)
 {
     const dim3 grid((g.rows + GLA_CHUNK - 1) / GLA_CHUNK, g.heads);
-    g.chunk = GLA_CHUNK;
-    TRY(gla_decays(g, flags, stream));
     TRY(launch("gla_chunk_state", gla_chunk_state_kernel, grid, GC_THREADS, gla_chunk_state_smem_bytes(g.dim_pad, g.vdim_pad), flags, stream, 0, g));
     const int quads = g.heads * g.dim_pad * g.vdim_pad / 4;
     TRY(launch("gla_scan", gla_scan_kernel<bf16>, dim3((quads + GS_THREADS - 1) / GS_THREADS), GS_THREADS, 0, flags, stream, 0, g));
@@ -616,7 +607,9 @@ twm_status gla_mixer(const twm_dense_model* m, const twm_dense_layer& l, const t
     if (kernel < 0 || kernel > 2) return invalid("kernel");
     if (kernel == 2 && !gla_chunks_fit(g)) return invalid("the chunked linear attention takes bfloat16 heads that fit shared memory");
     if (kernel == 2 || (kernel == 0 && gla_chunks_fit(g))) return gla_chunks(g, flags, stream);
-    TRY(gla_decays(g, flags, stream));
+    const int cols = g.heads * g.dim_pad;
+    TRY(launch("gla_decay", gla_decay_kernel<T>, dim3((cols + GD_THREADS - 1) / GD_THREADS, (rows + GD_ROWS - 1) / GD_ROWS), GD_THREADS, 0, flags,
+               stream, 0, g));
     TRY(launch("gla_rows", gla_rows_kernel<T>, dim3((g.vdim_pad + GR_COLS - 1) / GR_COLS, g.heads), GR_THREADS, gla_rows_smem_bytes(g.dim_pad), flags,
                stream, 0, g));
     return launch("gla_gate", gla_gate_kernel<T>, dim3(rows), ROW_THREADS, 0, flags, stream, 0, g);

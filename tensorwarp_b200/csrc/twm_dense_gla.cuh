@@ -4,14 +4,14 @@
 //
 // Prompt steps, bfloat16: chunks of 64 tokens.  With b_t the running sum of log alpha inside a chunk,
 //   o_t = (q_t e^{b_t})^T S_chunk + sum_{s <= t} (sum_d q_td k_sd e^{b_td - b_sd}) v_s.
-//   gla_decay_kernel        b, from the low-rank projection
-//   gla_chunk_state_kernel  what each chunk adds to the state, all chunks at once
+//   gla_chunk_state_kernel  b, from the low-rank projection, and what each chunk adds to the state, all chunks at once
 //   gla_scan_kernel         the state ahead of every chunk, chunk by chunk, element by element
 //   gla_chunk_out_kernel    o, norm and gate, all chunks at once
 // Every factor with a decay is computed in FP32 and enters a warp-level MMA as a bf16 pair hi + lo.  The scores inside a
 // chunk are one product, with the exponents taken against the chunk's middle token: safe while neither half of the
 // chunk decays by more than e^60; a chunk that does is scored token pair by token pair.
-// Everything else (FP32, wide heads): gla_rows_kernel walks the tokens one by one, gla_gate_kernel norms and gates.
+// Everything else (FP32, wide heads): gla_decay_kernel makes log alpha, gla_rows_kernel walks the tokens one by one,
+// gla_gate_kernel norms and gates.
 // Decoding: gla_decode_kernel.
 #pragma once
 
@@ -27,7 +27,7 @@ constexpr float GLA_HALF_LIMIT = 60.0f;         // largest decay (its logarithm)
 template <typename T>
 struct GlaArgs {
     const T* proj;              // [rows][ld]: q | k | v | gate | low-rank
-    float* decay;               // [rows][heads * dim_pad]: running sums of log alpha inside chunks of `chunk` rows
+    float* decay;               // [rows][heads * dim_pad]: log alpha, or (chunks) its running sums inside a chunk
     float* chunk_state;         // [chunks][heads][dim_pad][vdim_pad]
     float* mix;                 // [rows][heads * vdim_pad], token by token only
     T* out;                     // [rows][heads * vdim_pad]
@@ -36,7 +36,7 @@ struct GlaArgs {
     const float* decay_bias;    // [heads * dim_pad]
     const float* head_norm;     // [vdim_pad]
     const int* meta;
-    int ld, heads, dim_pad, vdim, vdim_pad, rank_pad, rows, chunk;
+    int ld, heads, dim_pad, vdim, vdim_pad, rank_pad, rows;
     float inv_tau, q_scale, eps;
     __device__ __forceinline__ int k_off() const { return heads * dim_pad; }
     __device__ __forceinline__ int v_off() const { return 2 * heads * dim_pad; }
@@ -45,16 +45,15 @@ struct GlaArgs {
     __device__ __forceinline__ float* slot_state(int h) const { return state + ((size_t)meta[1] * heads + h) * dim_pad * vdim_pad; }
 };
 
-// A thread per key channel and run of up to 64 rows: log alpha = log(sigmoid(z)) / tau, summed up within chunks.
-constexpr int GD_THREADS = 64, GD_ROWS = 64, GD_RANK = 32;
 // log(sigmoid(z)) to about 2^-22 of itself or 2e-7, whichever is larger
 __device__ __forceinline__ float log_sigmoid_fast(float z) {
     const float e = ex2_approx(-1.4426950408889634f * fabsf(z));
     const float near_one = e * fmaf(-e, fmaf(-e, fmaf(-e, 0.25f, 1.0f / 3.0f), 0.5f), 1.0f);      // log(1 + e) for small e
     return fminf(z, 0.0f) - (e < 0.0078125f ? near_one : __logf(1.0f + e));
 }
-__device__ __forceinline__ float log_sigmoid_of(float z, float) { return log_sigmoid_f32(z); }
-__device__ __forceinline__ float log_sigmoid_of(float z, bf16) { return log_sigmoid_fast(z); }
+
+// A thread per key channel and run of rows: log alpha = log(sigmoid(z)) / tau.
+constexpr int GD_THREADS = 128, GD_ROWS = 16, GD_RANK = 32;
 template <typename T>
 __global__ void __launch_bounds__(GD_THREADS)
 gla_decay_kernel(const GlaArgs<T> g)
@@ -72,9 +71,9 @@ gla_decay_kernel(const GlaArgs<T> g)
     for (int k0 = 0; k0 < g.rank_pad; k0 += GD_RANK) {
         const int kn = min(GD_RANK, g.rank_pad - k0);
         __syncthreads();
-        for (int i = threadIdx.x; i < n * kn; i += GD_THREADS) {
+        for (int i = threadIdx.x; i < GD_ROWS * kn; i += GD_THREADS) {
             const int r = i / kn, k = i - r * kn;
-            low[r][k] = to_f32(g.proj[(size_t)(r0 + r) * g.ld + g.low_off() + k0 + k]);
+            low[r][k] = r < n ? to_f32(g.proj[(size_t)(r0 + r) * g.ld + g.low_off() + k0 + k]) : 0.0f;
         }
         __syncthreads();
         if (col < cols) {
@@ -92,14 +91,9 @@ gla_decay_kernel(const GlaArgs<T> g)
         }
     }
     if (col >= cols) return;
-    float sum = 0.0f;
 #pragma unroll
-    for (int r = 0; r < GD_ROWS; ++r) {
-        if (r >= n) break;
-        const float la = log_sigmoid_of(z[r], T()) * g.inv_tau;
-        sum = (r0 + r) % g.chunk == 0 ? la : sum + la;
-        g.decay[(size_t)(r0 + r) * cols + col] = sum;
-    }
+    for (int r = 0; r < GD_ROWS; ++r)
+        if (r < n) g.decay[(size_t)(r0 + r) * cols + col] = log_sigmoid_f32(z[r]) * g.inv_tau;
 }
 
 // Token by token: CTA = 32 value columns of a head, thread = a column and every eighth key channel.
@@ -194,42 +188,90 @@ __device__ __forceinline__ void decayed8(const uint4& x, const float4& e0, const
     split_bf16(v[6], v[7], hi.w, lo.w);
 }
 
-// dS[d][v] = sum_t k_td e^{b_last,d - b_td} v_tv of one chunk and head.
+constexpr int GC_BATCH = 4;                                // vectors whose loads a thread has in flight
+// The running sums b of log alpha of one chunk and head, and dS[d][v] = sum_t k_td e^{b_last,d - b_td} v_tv.
 __host__ inline size_t gla_chunk_state_smem_bytes(int dim_pad, int vdim_pad) {
-    return (size_t)GLA_CHUNK * (2 * (dim_pad * 2 + 16) + (vdim_pad * 2 + 16));
+    return (size_t)GLA_CHUNK * (2 * (dim_pad * 2 + 16) + (vdim_pad * 2 + 16) + (dim_pad + 4) * sizeof(float));
 }
 __global__ void __launch_bounds__(GC_THREADS)
 gla_chunk_state_kernel(const GlaArgs<bf16> g)
 {
     extern __shared__ __align__(16) uint8_t gc_smem[];
     const int krow = g.dim_pad * 2 + 16, vrow = g.vdim_pad * 2 + 16;      // padded: eight rows of a fragment hit distinct banks
+    const int brow = g.dim_pad + 4;
     uint8_t* khi = gc_smem;                                // [64][dim_pad]
     uint8_t* klo = khi + GLA_CHUNK * krow;
     uint8_t* vs = klo + GLA_CHUNK * krow;                  // [64][vdim_pad]
+    float* bs = reinterpret_cast<float*>(vs + GLA_CHUNK * vrow);          // [64][dim_pad]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int h = blockIdx.y, r0 = blockIdx.x * GLA_CHUNK, n = min(GLA_CHUNK, g.rows - r0);
     const int cols = g.heads * g.dim_pad;
     pdl_wait_prior_grids();
     pdl_launch_dependents();
     const bf16* row0 = g.proj + (size_t)r0 * g.ld;
-    const float* b0 = g.decay + (size_t)r0 * cols + h * g.dim_pad;
     const int kp = g.dim_pad / 8, vp = g.vdim_pad / 8;
     for (int i = tid; i < GLA_CHUNK * vp; i += GC_THREADS) {
         const int t = i / vp, c = i - t * vp;
         ops::att_cp_async16(smem_u32(vs + t * vrow + c * 16), row0 + (size_t)(t < n ? t : 0) * g.ld + g.v_off() + h * g.vdim_pad + c * 8, t < n ? 16 : 0);
     }
     ops::att_cp_async_commit();
-#pragma unroll 2
-    for (int i = tid; i < GLA_CHUNK * kp; i += GC_THREADS) {
-        const int t = i / kp, d = (i - t * kp) * 8;
-        uint4 hi = make_uint4(0, 0, 0, 0), lo = hi;
-        if (t < n) {
-            const float *b = b0 + (size_t)t * cols + d, *last = b0 + (size_t)(n - 1) * cols + d;
-            decayed8(*reinterpret_cast<const uint4*>(row0 + (size_t)t * g.ld + g.k_off() + h * g.dim_pad + d), load4(last), load4(last + 4), load4(b),
-                     load4(b + 4), 1.0f, hi, lo);
+    // keys on their way; their decays are made meanwhile
+    uint4 kv[GC_BATCH];
+    auto load_keys = [&](int i0) {
+#pragma unroll
+        for (int j = 0; j < GC_BATCH; ++j) {
+            const int i = i0 + j * GC_THREADS, t = i / kp, d = (i - t * kp) * 8;
+            kv[j] = i < GLA_CHUNK * kp && t < n ? *reinterpret_cast<const uint4*>(row0 + (size_t)t * g.ld + g.k_off() + h * g.dim_pad + d)
+                                                : make_uint4(0, 0, 0, 0);
         }
-        *reinterpret_cast<uint4*>(khi + t * krow + d * 2) = hi;
-        *reinterpret_cast<uint4*>(klo + t * krow + d * 2) = lo;
+    };
+    load_keys(tid);
+    {   // z = low-rank row times the decay's weights: a warp's unit is 16 tokens x 8 channels
+        const int nt = g.dim_pad / 8;
+        for (int u = warp; u < 4 * nt; u += GC_THREADS / 32) {
+            const int t0 = (u & 3) * 16, c0 = (u >> 2) * 8;
+            const int ta = min(t0 + (lane >> 2), n - 1), tb = min(t0 + (lane >> 2) + 8, n - 1), k = (lane & 3) * 2;
+            const bf16 *la = row0 + (size_t)ta * g.ld + g.low_off() + k, *lb = row0 + (size_t)tb * g.ld + g.low_off() + k;
+            const bf16* w = g.w_decay + (size_t)(h * g.dim_pad + c0 + (lane >> 2)) * g.rank_pad + k;
+            float z[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+            for (int k0 = 0; k0 < g.rank_pad; k0 += 16) {
+                const uint32_t a[4] = {*reinterpret_cast<const uint32_t*>(la + k0), *reinterpret_cast<const uint32_t*>(lb + k0),
+                                       *reinterpret_cast<const uint32_t*>(la + k0 + 8), *reinterpret_cast<const uint32_t*>(lb + k0 + 8)};
+                mma_bf16(z, a, __ldg(reinterpret_cast<const uint32_t*>(w + k0)), __ldg(reinterpret_cast<const uint32_t*>(w + k0 + 8)));
+            }
+            const float2 bias = __ldg(reinterpret_cast<const float2*>(g.decay_bias + h * g.dim_pad + c0 + k));
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+                *reinterpret_cast<float2*>(bs + (t0 + (lane >> 2) + i * 8) * brow + c0 + k) =
+                    make_float2(log_sigmoid_fast(z[2 * i] + bias.x) * g.inv_tau, log_sigmoid_fast(z[2 * i + 1] + bias.y) * g.inv_tau);
+        }
+    }
+    __syncthreads();
+    for (int d = tid; d < g.dim_pad; d += GC_THREADS) {    // running sums, kept for the kernels that follow
+        float* to = g.decay + (size_t)r0 * cols + h * g.dim_pad + d;
+        float sum = 0.0f;
+#pragma unroll 8
+        for (int t = 0; t < n; ++t) {
+            sum += bs[t * brow + d];
+            bs[t * brow + d] = sum;
+            to[(size_t)t * cols] = sum;
+        }
+    }
+    __syncthreads();
+    for (int i0 = tid; i0 < GLA_CHUNK * kp; i0 += GC_BATCH * GC_THREADS) {
+        if (i0 > tid) load_keys(i0);
+#pragma unroll
+        for (int j = 0; j < GC_BATCH; ++j) {
+            const int i = i0 + j * GC_THREADS, t = i / kp, d = (i - t * kp) * 8;
+            if (i >= GLA_CHUNK * kp) continue;
+            uint4 hi = make_uint4(0, 0, 0, 0), lo = hi;
+            if (t < n) {
+                const float *b = bs + t * brow + d, *last = bs + (n - 1) * brow + d;
+                decayed8(kv[j], load4(last), load4(last + 4), load4(b), load4(b + 4), 1.0f, hi, lo);
+            }
+            *reinterpret_cast<uint4*>(khi + t * krow + d * 2) = hi;
+            *reinterpret_cast<uint4*>(klo + t * krow + d * 2) = lo;
+        }
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
@@ -288,25 +330,24 @@ gla_scan_kernel(const GlaArgs<T> g)
     float4* cs = reinterpret_cast<float4*>(g.chunk_state) + (size_t)h * per_head + e;
     const size_t step = (size_t)g.heads * per_head;
     const float* b = g.decay + h * g.dim_pad + d;
+    float4 add[GS_AHEAD];
+    float a[GS_AHEAD];
+    auto fetch = [&](int j, int n) {
+        if (n >= chunks) return;
+        add[j] = cs[n * step];
+        a[j] = b[(size_t)(min(g.rows, (n + 1) * GLA_CHUNK) - 1) * cols];
+    };
+#pragma unroll
+    for (int j = 0; j < GS_AHEAD; ++j) fetch(j, j);
     for (int n0 = 0; n0 < chunks; n0 += GS_AHEAD) {
-        float4 add[GS_AHEAD];
-        float a[GS_AHEAD];
 #pragma unroll
         for (int j = 0; j < GS_AHEAD; ++j) {
             const int n = n0 + j;
-            if (n < chunks) {
-                add[j] = cs[n * step];
-                a[j] = b[(size_t)(min(g.rows, (n + 1) * GLA_CHUNK) - 1) * cols];
-            }
-        }
-#pragma unroll
-        for (int j = 0; j < GS_AHEAD; ++j) {
-            const int n = n0 + j;
-            if (n < chunks) {
-                cs[n * step] = s;
-                const float f = expf(a[j]);
-                s = make_float4(fmaf(s.x, f, add[j].x), fmaf(s.y, f, add[j].y), fmaf(s.z, f, add[j].z), fmaf(s.w, f, add[j].w));
-            }
+            if (n >= chunks) break;
+            cs[n * step] = s;
+            const float f = expf(a[j]);
+            s = make_float4(fmaf(s.x, f, add[j].x), fmaf(s.y, f, add[j].y), fmaf(s.z, f, add[j].z), fmaf(s.w, f, add[j].w));
+            fetch(j, n + GS_AHEAD);                        // eight chunks ahead of its use
         }
     }
     *st = s;
@@ -347,6 +388,21 @@ gla_chunk_out_kernel(const GlaArgs<bf16> g)
         ops::att_cp_async16(smem_u32(vs + t * vrow + c * 16), row0 + (size_t)(t < n ? t : 0) * g.ld + g.v_off() + h * g.vdim_pad + c * 8, t < n ? 16 : 0);
     }
     ops::att_cp_async_commit();
+    uint4 qv[GC_BATCH], kv[GC_BATCH];
+    float4 bv[GC_BATCH][2];
+    auto load_rows = [&](int i0) {
+#pragma unroll
+        for (int j = 0; j < GC_BATCH; ++j) {
+            const int i = i0 + j * GC_THREADS, t = i / kp, d = (i - t * kp) * 8;
+            if (i >= GLA_CHUNK * kp || t >= n) continue;
+            const bf16* row = row0 + (size_t)t * g.ld + h * g.dim_pad + d;
+            qv[j] = *reinterpret_cast<const uint4*>(row);
+            kv[j] = *reinterpret_cast<const uint4*>(row + g.k_off());
+            bv[j][0] = load4(b0 + (size_t)t * cols + d);
+            bv[j][1] = load4(b0 + (size_t)t * cols + d + 4);
+        }
+    };
+    load_rows(tid);
     bool steep = false;
     for (int d = tid; d < g.dim_pad; d += GC_THREADS) {
         const float first = b0[d], mid = b0[(size_t)middle * cols + d], last = b0[(size_t)(n - 1) * cols + d];
@@ -355,22 +411,23 @@ gla_chunk_out_kernel(const GlaArgs<bf16> g)
     }
     steep = __syncthreads_or(steep);
     const float4 zero4 = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 2
-    for (int i = tid; i < GLA_CHUNK * kp; i += GC_THREADS) {
-        const int t = i / kp, d = (i - t * kp) * 8;
-        uint4 qh = make_uint4(0, 0, 0, 0), ql = qh, kh = qh, kl = qh;
-        if (t < n) {
-            const bf16* row = row0 + (size_t)t * g.ld + h * g.dim_pad + d;
-            const uint4 q = *reinterpret_cast<const uint4*>(row), k = *reinterpret_cast<const uint4*>(row + g.k_off());
-            const float4 e0 = load4(b0 + (size_t)t * cols + d), e1 = load4(b0 + (size_t)t * cols + d + 4);
-            const float4 f0 = steep ? zero4 : load4(refs + d), f1 = steep ? zero4 : load4(refs + d + 4);
-            decayed8(q, e0, e1, f0, f1, g.q_scale, qh, ql);
-            if (!steep) decayed8(k, f0, f1, e0, e1, 1.0f, kh, kl);
+    for (int i0 = tid; i0 < GLA_CHUNK * kp; i0 += GC_BATCH * GC_THREADS) {
+        if (i0 > tid) load_rows(i0);
+#pragma unroll
+        for (int j = 0; j < GC_BATCH; ++j) {
+            const int i = i0 + j * GC_THREADS, t = i / kp, d = (i - t * kp) * 8;
+            if (i >= GLA_CHUNK * kp) continue;
+            uint4 qh = make_uint4(0, 0, 0, 0), ql = qh, kh = qh, kl = qh;
+            if (t < n) {
+                const float4 f0 = steep ? zero4 : load4(refs + d), f1 = steep ? zero4 : load4(refs + d + 4);
+                decayed8(qv[j], bv[j][0], bv[j][1], f0, f1, g.q_scale, qh, ql);
+                if (!steep) decayed8(kv[j], f0, f1, bv[j][0], bv[j][1], 1.0f, kh, kl);
+            }
+            *reinterpret_cast<uint4*>(qhi + t * krow + d * 2) = qh;
+            *reinterpret_cast<uint4*>(qlo + t * krow + d * 2) = ql;
+            *reinterpret_cast<uint4*>(khi + t * wide + d * 2) = kh;
+            *reinterpret_cast<uint4*>(klo + t * wide + d * 2) = kl;
         }
-        *reinterpret_cast<uint4*>(qhi + t * krow + d * 2) = qh;
-        *reinterpret_cast<uint4*>(qlo + t * krow + d * 2) = ql;
-        *reinterpret_cast<uint4*>(khi + t * wide + d * 2) = kh;
-        *reinterpret_cast<uint4*>(klo + t * wide + d * 2) = kl;
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();

@@ -3,12 +3,13 @@
 // decode one is twm_dense_decode.cuh's, with its rows looked up by expert).
 #pragma once
 
+#include "twm_dense_rows.cuh"
 #include "twm_dense_simt.cuh"
 
 namespace twm {
 namespace dense {
 
-constexpr int MOE_MAX_EXPERTS = 1024, MOE_MAX_TOP = 32;
+constexpr int MOE_MAX_EXPERTS = 1024, MOE_MAX_TOP = MAX_TOP;
 
 struct RouterArgs { int experts, top, groups, keep; };
 

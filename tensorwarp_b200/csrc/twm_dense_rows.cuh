@@ -9,6 +9,7 @@ namespace twm {
 namespace dense {
 
 constexpr int ROW_THREADS = 256;
+constexpr int MAX_TOP = 32;                             // experts a token uses, at most
 
 // Outputs of the chosen experts: a token's sublayer output is the sum over its `top` slots of weight * row.
 template <typename T>
@@ -138,6 +139,8 @@ residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __rest
                           ? shift_state + ((size_t)meta[1] * 2 + ((pos0 - 1) & 1)) * wp : nullptr;
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     if constexpr (PER > 0) {
+        __shared__ int slot_row[MAX_TOP];
+        __shared__ float slot_weight[MAX_TOP];
         float4 before[PER];
 #pragma unroll
         for (int j = 0; j < PER; ++j) {
@@ -146,6 +149,14 @@ residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __rest
         }
         for (int r = (shift != nullptr && r0 > 0) ? r0 - 1 : r0; r < r1; ++r) {
             float4 x[PER], y[PER];
+            if (src.routed.rows != nullptr) {               // the row's slots, known before the first of their loads
+                __syncthreads();
+                if (threadIdx.x < src.routed.top) {
+                    slot_row[threadIdx.x] = src.routed.row[(size_t)r * src.routed.top + threadIdx.x];
+                    slot_weight[threadIdx.x] = src.routed.weight[(size_t)r * src.routed.top + threadIdx.x];
+                }
+                __syncthreads();
+            }
             const int tok = src.tokens != nullptr ? src.tokens[r] : 0;
             ResidualSource<T> plain = src;                  // the row without what joins it
             plain.y = nullptr;
@@ -153,8 +164,22 @@ residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __rest
 #pragma unroll
             for (int j = 0; j < PER; ++j) {
                 const int i = threadIdx.x + j * ROW_THREADS;
-                y[j] = src.has_y() && i < nvec ? src.y_at(r, i) : zero;
+                y[j] = src.y != nullptr && i < nvec ? src.y_at(r, i) : zero;
                 x[j] = i < nvec ? plain.at(r, pos0 + r, tok, i, 1.0f) : zero;
+            }
+            if (src.routed.rows != nullptr) {
+#pragma unroll 4
+                for (int s = 0; s < src.routed.top; ++s) {
+                    const T* row = src.routed.rows + (size_t)slot_row[s] * wp;
+                    const float ws = slot_weight[s];
+#pragma unroll
+                    for (int j = 0; j < PER; ++j) {
+                        const int i = threadIdx.x + j * ROW_THREADS;
+                        if (i >= nvec) continue;
+                        const float4 t = load4(row + i * 4);
+                        y[j].x = fmaf(t.x, ws, y[j].x); y[j].y = fmaf(t.y, ws, y[j].y); y[j].z = fmaf(t.z, ws, y[j].z); y[j].w = fmaf(t.w, ws, y[j].w);
+                    }
+                }
             }
             float ir = 1.0f;
             if (src.has_y() && src.y_norm != nullptr) {
