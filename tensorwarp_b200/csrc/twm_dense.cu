@@ -588,17 +588,20 @@ bool gla_chunks_fit(const GlaArgs<float>&) { return false; }
 bool gla_chunks_fit(const GlaArgs<bf16>& g)
 {
     return g.vdim_pad <= 128 && gla_chunk_out_smem_bytes(g.dim_pad, g.vdim_pad) <= kSmemLimit &&
-           gla_chunk_state_smem_bytes(g.dim_pad, g.vdim_pad) <= kSmemLimit;
+           gla_chunk_state_smem_bytes(g.vdim_pad) <= kSmemLimit;
 }
 twm_status gla_chunks(const GlaArgs<float>&, int, void*) { return invalid("the chunked linear attention takes bfloat16"); }
 twm_status gla_chunks(const GlaArgs<bf16>& g, int flags, void* stream)
 {
-    const dim3 grid((g.rows + GLA_CHUNK - 1) / GLA_CHUNK, g.heads);
-    TRY(launch("gla_chunk_state", gla_chunk_state_kernel, grid, GC_THREADS, gla_chunk_state_smem_bytes(g.dim_pad, g.vdim_pad), flags, stream, 0, g));
-    const int quads = g.heads * g.dim_pad * g.vdim_pad / 4;
+    const int chunks = (g.rows + GLA_CHUNK - 1) / GLA_CHUNK, quads = g.heads * g.dim_pad * g.vdim_pad / 4;
+    const bool d128 = g.dim_pad == 128 && g.vdim_pad == 128, d64 = g.dim_pad == 64 && g.vdim_pad == 64;
+    auto state = d128 ? gla_chunk_state_kernel<128, 128> : d64 ? gla_chunk_state_kernel<64, 64> : gla_chunk_state_kernel<0, 0>;
+    auto out = d128 ? gla_chunk_out_kernel<128, 128> : d64 ? gla_chunk_out_kernel<64, 64> : g.vdim_pad <= 64 ? gla_chunk_out_kernel<0, 64>
+                                                                                                     : gla_chunk_out_kernel<0, 128>;
+    TRY(launch("gla_chunk_state", state, dim3(chunks, g.heads, (g.dim_pad + GC_DIMS - 1) / GC_DIMS), GC_THREADS,
+               gla_chunk_state_smem_bytes(g.vdim_pad), flags, stream, 0, g));
     TRY(launch("gla_scan", gla_scan_kernel<bf16>, dim3((quads + GS_THREADS - 1) / GS_THREADS), GS_THREADS, 0, flags, stream, 0, g));
-    auto out = g.vdim_pad <= 64 ? gla_chunk_out_kernel<64> : gla_chunk_out_kernel<128>;
-    return launch("gla_chunk_out", out, grid, GC_THREADS, gla_chunk_out_smem_bytes(g.dim_pad, g.vdim_pad), flags, stream, 0, g);
+    return launch("gla_chunk_out", out, dim3(chunks, g.heads), GO_THREADS, gla_chunk_out_smem_bytes(g.dim_pad, g.vdim_pad), flags, stream, 0, g);
 }
 template <typename T>
 twm_status gla_mixer(const twm_dense_model* m, const twm_dense_layer& l, const twm_dense_buffers* b, int rows, int kernel, int flags, void* stream)

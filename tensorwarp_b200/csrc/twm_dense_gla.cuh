@@ -188,98 +188,105 @@ __device__ __forceinline__ void decayed8(const uint4& x, const float4& e0, const
     split_bf16(v[6], v[7], hi.w, lo.w);
 }
 
-constexpr int GC_BATCH = 4;                                // vectors whose loads a thread has in flight
-// The running sums b of log alpha of one chunk and head, and dS[d][v] = sum_t k_td e^{b_last,d - b_td} v_tv.
-__host__ inline size_t gla_chunk_state_smem_bytes(int dim_pad, int vdim_pad) {
-    return (size_t)GLA_CHUNK * (2 * (dim_pad * 2 + 16) + (vdim_pad * 2 + 16) + (dim_pad + 4) * sizeof(float));
+// The chunk kernels take 64 key channels at a time: rows of 64 bf16, padded so that eight rows of a fragment hit distinct banks.
+constexpr int GC_DIMS = 64, GC_ROW = GC_DIMS * 2 + 16, GC_BROW = GC_DIMS + 4;
+
+// CTA = chunk, head and 64 key channels: the running sums b of log alpha, and dS[d][v] = sum_t k_td e^{b_last,d - b_td} v_tv.
+// DK, DV: padded head sizes (0: read from the arguments).
+__host__ inline size_t gla_chunk_state_smem_bytes(int vdim_pad) {
+    return (size_t)GLA_CHUNK * (2 * GC_ROW + vdim_pad * 2 + 16 + GC_BROW * sizeof(float)) + 4 * GC_DIMS * sizeof(float);
 }
+template <int DK, int DV>
 __global__ void __launch_bounds__(GC_THREADS)
 gla_chunk_state_kernel(const GlaArgs<bf16> g)
 {
     extern __shared__ __align__(16) uint8_t gc_smem[];
-    const int krow = g.dim_pad * 2 + 16, vrow = g.vdim_pad * 2 + 16;      // padded: eight rows of a fragment hit distinct banks
-    const int brow = g.dim_pad + 4;
-    uint8_t* khi = gc_smem;                                // [64][dim_pad]
-    uint8_t* klo = khi + GLA_CHUNK * krow;
-    uint8_t* vs = klo + GLA_CHUNK * krow;                  // [64][vdim_pad]
-    float* bs = reinterpret_cast<float*>(vs + GLA_CHUNK * vrow);          // [64][dim_pad]
+    const int dim_pad = DK > 0 ? DK : g.dim_pad, vdim_pad = DV > 0 ? DV : g.vdim_pad;
+    const int vrow = vdim_pad * 2 + 16;
+    uint8_t* khi = gc_smem;                                // [64][64]
+    uint8_t* klo = khi + GLA_CHUNK * GC_ROW;
+    uint8_t* vs = klo + GLA_CHUNK * GC_ROW;                // [64][vdim_pad]
+    float* bs = reinterpret_cast<float*>(vs + GLA_CHUNK * vrow);          // [64][64]
+    float* quarter_sum = bs + GLA_CHUNK * GC_BROW;         // [4][64]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int h = blockIdx.y, r0 = blockIdx.x * GLA_CHUNK, n = min(GLA_CHUNK, g.rows - r0);
-    const int cols = g.heads * g.dim_pad;
+    const int d0 = blockIdx.z * GC_DIMS, dims = min(GC_DIMS, dim_pad - d0);
+    const int cols = g.heads * dim_pad;
     pdl_wait_prior_grids();
     pdl_launch_dependents();
     const bf16* row0 = g.proj + (size_t)r0 * g.ld;
-    const int kp = g.dim_pad / 8, vp = g.vdim_pad / 8;
+    const int vp = vdim_pad / 8;
     for (int i = tid; i < GLA_CHUNK * vp; i += GC_THREADS) {
         const int t = i / vp, c = i - t * vp;
-        ops::att_cp_async16(smem_u32(vs + t * vrow + c * 16), row0 + (size_t)(t < n ? t : 0) * g.ld + g.v_off() + h * g.vdim_pad + c * 8, t < n ? 16 : 0);
+        ops::att_cp_async16(smem_u32(vs + t * vrow + c * 16), row0 + (size_t)(t < n ? t : 0) * g.ld + g.v_off() + h * vdim_pad + c * 8, t < n ? 16 : 0);
     }
     ops::att_cp_async_commit();
-    // keys on their way; their decays are made meanwhile
-    uint4 kv[GC_BATCH];
-    auto load_keys = [&](int i0) {
+    // keys on their way; their decays are made meanwhile.  Vector i: token i / 8, channels 8 (i % 8) on
+    constexpr int KV = GLA_CHUNK * GC_DIMS / 8 / GC_THREADS;
+    uint4 kv[KV];
 #pragma unroll
-        for (int j = 0; j < GC_BATCH; ++j) {
-            const int i = i0 + j * GC_THREADS, t = i / kp, d = (i - t * kp) * 8;
-            kv[j] = i < GLA_CHUNK * kp && t < n ? *reinterpret_cast<const uint4*>(row0 + (size_t)t * g.ld + g.k_off() + h * g.dim_pad + d)
-                                                : make_uint4(0, 0, 0, 0);
+    for (int j = 0; j < KV; ++j) {
+        const int i = tid + j * GC_THREADS, t = i >> 3, d = (i & 7) * 8;
+        kv[j] = t < n && d < dims ? *reinterpret_cast<const uint4*>(row0 + (size_t)t * g.ld + g.k_off() + h * dim_pad + d0 + d) : make_uint4(0, 0, 0, 0);
+    }
+    // z = low-rank row times the decay's weights: a warp's unit is 16 tokens x 8 channels
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        const int u = warp + j * (GC_THREADS / 32), t0 = (u & 3) * 16, c0 = (u >> 2) * 8;
+        if (c0 >= dims) break;
+        const int ta = min(t0 + (lane >> 2), n - 1), tb = min(t0 + (lane >> 2) + 8, n - 1), k = (lane & 3) * 2;
+        const bf16 *la = row0 + (size_t)ta * g.ld + g.low_off() + k, *lb = row0 + (size_t)tb * g.ld + g.low_off() + k;
+        const bf16* w = g.w_decay + (size_t)(h * dim_pad + d0 + c0 + (lane >> 2)) * g.rank_pad + k;
+        float z[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+        for (int k0 = 0; k0 < g.rank_pad; k0 += 16) {
+            const uint32_t a[4] = {*reinterpret_cast<const uint32_t*>(la + k0), *reinterpret_cast<const uint32_t*>(lb + k0),
+                                   *reinterpret_cast<const uint32_t*>(la + k0 + 8), *reinterpret_cast<const uint32_t*>(lb + k0 + 8)};
+            mma_bf16(z, a, __ldg(reinterpret_cast<const uint32_t*>(w + k0)), __ldg(reinterpret_cast<const uint32_t*>(w + k0 + 8)));
         }
-    };
-    load_keys(tid);
-    {   // z = low-rank row times the decay's weights: a warp's unit is 16 tokens x 8 channels
-        const int nt = g.dim_pad / 8;
-        for (int u = warp; u < 4 * nt; u += GC_THREADS / 32) {
-            const int t0 = (u & 3) * 16, c0 = (u >> 2) * 8;
-            const int ta = min(t0 + (lane >> 2), n - 1), tb = min(t0 + (lane >> 2) + 8, n - 1), k = (lane & 3) * 2;
-            const bf16 *la = row0 + (size_t)ta * g.ld + g.low_off() + k, *lb = row0 + (size_t)tb * g.ld + g.low_off() + k;
-            const bf16* w = g.w_decay + (size_t)(h * g.dim_pad + c0 + (lane >> 2)) * g.rank_pad + k;
-            float z[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-            for (int k0 = 0; k0 < g.rank_pad; k0 += 16) {
-                const uint32_t a[4] = {*reinterpret_cast<const uint32_t*>(la + k0), *reinterpret_cast<const uint32_t*>(lb + k0),
-                                       *reinterpret_cast<const uint32_t*>(la + k0 + 8), *reinterpret_cast<const uint32_t*>(lb + k0 + 8)};
-                mma_bf16(z, a, __ldg(reinterpret_cast<const uint32_t*>(w + k0)), __ldg(reinterpret_cast<const uint32_t*>(w + k0 + 8)));
-            }
-            const float2 bias = __ldg(reinterpret_cast<const float2*>(g.decay_bias + h * g.dim_pad + c0 + k));
+        const float2 bias = __ldg(reinterpret_cast<const float2*>(g.decay_bias + h * dim_pad + d0 + c0 + k));
 #pragma unroll
-            for (int i = 0; i < 2; ++i)
-                *reinterpret_cast<float2*>(bs + (t0 + (lane >> 2) + i * 8) * brow + c0 + k) =
-                    make_float2(log_sigmoid_fast(z[2 * i] + bias.x) * g.inv_tau, log_sigmoid_fast(z[2 * i + 1] + bias.y) * g.inv_tau);
+        for (int i = 0; i < 2; ++i)
+            *reinterpret_cast<float2*>(bs + (t0 + (lane >> 2) + i * 8) * GC_BROW + c0 + k) =
+                make_float2(log_sigmoid_fast(z[2 * i] + bias.x) * g.inv_tau, log_sigmoid_fast(z[2 * i + 1] + bias.y) * g.inv_tau);
+    }
+    __syncthreads();
+    {   // running sums, kept for the kernels that follow: a thread sums 16 tokens of a channel
+        const int d = tid & 63, q = tid >> 6;
+        float sum[16];
+#pragma unroll
+        for (int t = 0; t < 16; ++t) sum[t] = bs[(q * 16 + t) * GC_BROW + d] + (t > 0 ? sum[t - 1] : 0.0f);
+        quarter_sum[q * GC_DIMS + d] = sum[15];
+        __syncthreads();
+        float before = 0.0f;
+        for (int k = 0; k < q; ++k) before += quarter_sum[k * GC_DIMS + d];
+        float* to = g.decay + (size_t)r0 * cols + h * dim_pad + d0 + d;
+#pragma unroll
+        for (int t = 0; t < 16; ++t) {
+            const float b = before + sum[t];
+            bs[(q * 16 + t) * GC_BROW + d] = b;
+            if (q * 16 + t < n && d < dims) to[(size_t)(q * 16 + t) * cols] = b;
         }
     }
     __syncthreads();
-    for (int d = tid; d < g.dim_pad; d += GC_THREADS) {    // running sums, kept for the kernels that follow
-        float* to = g.decay + (size_t)r0 * cols + h * g.dim_pad + d;
-        float sum = 0.0f;
-#pragma unroll 8
-        for (int t = 0; t < n; ++t) {
-            sum += bs[t * brow + d];
-            bs[t * brow + d] = sum;
-            to[(size_t)t * cols] = sum;
-        }
-    }
-    __syncthreads();
-    for (int i0 = tid; i0 < GLA_CHUNK * kp; i0 += GC_BATCH * GC_THREADS) {
-        if (i0 > tid) load_keys(i0);
 #pragma unroll
-        for (int j = 0; j < GC_BATCH; ++j) {
-            const int i = i0 + j * GC_THREADS, t = i / kp, d = (i - t * kp) * 8;
-            if (i >= GLA_CHUNK * kp) continue;
-            uint4 hi = make_uint4(0, 0, 0, 0), lo = hi;
-            if (t < n) {
-                const float *b = bs + t * brow + d, *last = bs + (n - 1) * brow + d;
-                decayed8(kv[j], load4(last), load4(last + 4), load4(b), load4(b + 4), 1.0f, hi, lo);
-            }
-            *reinterpret_cast<uint4*>(khi + t * krow + d * 2) = hi;
-            *reinterpret_cast<uint4*>(klo + t * krow + d * 2) = lo;
+    for (int j = 0; j < KV; ++j) {
+        const int i = tid + j * GC_THREADS, t = i >> 3, d = (i & 7) * 8;
+        uint4 hi = make_uint4(0, 0, 0, 0), lo = hi;
+        if (t < n && d < dims) {
+            const float *b = bs + t * GC_BROW + d, *last = bs + (n - 1) * GC_BROW + d;
+            decayed8(kv[j], load4(last), load4(last + 4), load4(b), load4(b + 4), 1.0f, hi, lo);
         }
+        *reinterpret_cast<uint4*>(khi + t * GC_ROW + d * 2) = hi;
+        *reinterpret_cast<uint4*>(klo + t * GC_ROW + d * 2) = lo;
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
-    float* out = g.chunk_state + ((size_t)blockIdx.x * g.heads + h) * g.dim_pad * g.vdim_pad;
+    float* out = g.chunk_state + (((size_t)blockIdx.x * g.heads + h) * dim_pad + d0) * vdim_pad;
     // a warp's unit: 16 key channels x 64 value columns
-    const int mt = g.dim_pad / 16, nb = (g.vdim_pad + 63) / 64;
-    for (int u = warp; u < mt * nb; u += GC_THREADS / 32) {
-        const int m0 = (u % mt) * 16, v0 = (u / mt) * 64;
+    const int nb = (vdim_pad + 63) / 64;
+    for (int u = warp; u < 4 * nb; u += GC_THREADS / 32) {
+        const int m0 = (u & 3) * 16, v0 = (u >> 2) * 64;
+        if (m0 >= dims) continue;
         float acc[8][4];
 #pragma unroll
         for (int j = 0; j < 8; ++j)
@@ -288,13 +295,13 @@ gla_chunk_state_kernel(const GlaArgs<bf16> g)
 #pragma unroll
         for (int kk = 0; kk < GLA_CHUNK / 16; ++kk) {
             // A = K'^T (channels x tokens) out of rows of tokens: transposing loads
-            const uint32_t at = (uint32_t)((kk * 16 + (lane & 7) + (lane >> 4) * 8) * krow + (m0 + ((lane >> 3) & 1) * 8) * 2);
+            const uint32_t at = (uint32_t)((kk * 16 + (lane & 7) + (lane >> 4) * 8) * GC_ROW + (m0 + ((lane >> 3) & 1) * 8) * 2);
             uint32_t ahi[4], alo[4];
             ops::att_ldmatrix_x4_trans(ahi, smem_u32(khi) + at);
             ops::att_ldmatrix_x4_trans(alo, smem_u32(klo) + at);
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
-                if (v0 + j * 16 >= g.vdim_pad) continue;
+                if (v0 + j * 16 >= vdim_pad) continue;
                 uint32_t b[4];
                 ops::att_ldmatrix_x4_trans(b, smem_u32(vs) + (kk * 16 + (lane & 15)) * vrow + (v0 + j * 16 + (lane >> 4) * 8) * 2);
                 mma_bf16(acc[2 * j], ahi, b[0], b[1]);
@@ -306,9 +313,9 @@ gla_chunk_state_kernel(const GlaArgs<bf16> g)
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
             const int v = v0 + j * 8 + (lane & 3) * 2, d = m0 + (lane >> 2);
-            if (v0 + j * 8 >= g.vdim_pad) continue;
-            *reinterpret_cast<float2*>(out + (size_t)d * g.vdim_pad + v) = make_float2(acc[j][0], acc[j][1]);
-            *reinterpret_cast<float2*>(out + (size_t)(d + 8) * g.vdim_pad + v) = make_float2(acc[j][2], acc[j][3]);
+            if (v0 + j * 8 >= vdim_pad) continue;
+            *reinterpret_cast<float2*>(out + (size_t)d * vdim_pad + v) = make_float2(acc[j][0], acc[j][1]);
+            *reinterpret_cast<float2*>(out + (size_t)(d + 8) * vdim_pad + v) = make_float2(acc[j][2], acc[j][3]);
         }
     }
 }
@@ -353,210 +360,133 @@ gla_scan_kernel(const GlaArgs<T> g)
     *st = s;
 }
 
-// CTA = chunk and head; a pair of warps = 16 of its tokens.  DV: value columns the accumulators hold (>= vdim_pad).
-constexpr int GO_AROW = GLA_CHUNK * 2 + 16;                // bytes of a row of scores
-__host__ __device__ inline int gla_out_row(int dim_pad, int vdim_pad) { return (dim_pad > vdim_pad ? dim_pad : vdim_pad) * 2 + 16; }
+// CTA = chunk and head; four warps = 16 of its tokens.  For 64 key channels at a time: the scores' share and the state's,
+// (q 2^(b - ref)) (2^ref S); then scores V.  DK, DV: padded head sizes (DK = 0: read from the arguments, vdim_pad <= DV).
 __host__ inline size_t gla_chunk_out_smem_bytes(int dim_pad, int vdim_pad) {
-    return (size_t)GLA_CHUNK * (2 * (dim_pad * 2 + 16) + 2 * gla_out_row(dim_pad, vdim_pad) + vdim_pad * 2 + 16 + 2 * GO_AROW) +
-           sizeof(float) * (size_t)(dim_pad + 2 * GLA_CHUNK);
+    return (size_t)GLA_CHUNK * (4 * GC_ROW + 2 * (vdim_pad * 2 + 16)) + sizeof(float) * (size_t)(dim_pad + 4 * GLA_CHUNK);
 }
-template <int DV>
-__global__ void __launch_bounds__(GC_THREADS, 2)
+constexpr int GO_THREADS = 512;
+template <int DK, int DV>
+__global__ void __launch_bounds__(GO_THREADS, 2)
 gla_chunk_out_kernel(const GlaArgs<bf16> g)
 {
     extern __shared__ __align__(16) uint8_t gc_smem[];
-    const int krow = g.dim_pad * 2 + 16, vrow = g.vdim_pad * 2 + 16, wide = gla_out_row(g.dim_pad, g.vdim_pad);
-    uint8_t* qhi = gc_smem;                                // [64][dim_pad] q 2^(b_t - ref)
-    uint8_t* qlo = qhi + GLA_CHUNK * krow;
-    uint8_t* khi = qlo + GLA_CHUNK * krow;                 // [64][dim_pad] k 2^(ref - b_t); later 64 rows of the state
-    uint8_t* klo = khi + GLA_CHUNK * wide;
-    uint8_t* vs = klo + GLA_CHUNK * wide;                  // [64][vdim_pad]
-    uint8_t* ahi = vs + GLA_CHUNK * vrow;                  // [64][64] scores
-    uint8_t* alo = ahi + GLA_CHUNK * GO_AROW;
-    float* refs = reinterpret_cast<float*>(alo + GLA_CHUNK * GO_AROW);      // [dim_pad]: e^ref
-    float* sums = refs + g.dim_pad;                        // [2][64]
+    const int dim_pad = DK > 0 ? DK : g.dim_pad, vdim_pad = DK > 0 ? DV : g.vdim_pad;
+    const int vrow = vdim_pad * 2 + 16;
+    uint8_t* qhi = gc_smem;                                // [64][64] q 2^(b_t - ref); at the end the scores
+    uint8_t* qlo = qhi + GLA_CHUNK * GC_ROW;
+    uint8_t* khi = qlo + GLA_CHUNK * GC_ROW;               // [64][64] k 2^(ref - b_t)
+    uint8_t* klo = khi + GLA_CHUNK * GC_ROW;
+    uint8_t* shi = klo + GLA_CHUNK * GC_ROW;               // [64][vdim_pad] rows of the state; at the end the values
+    uint8_t* slo = shi + GLA_CHUNK * vrow;
+    float* refs = reinterpret_cast<float*>(slo + GLA_CHUNK * vrow);       // [dim_pad]
+    float* sums = refs + dim_pad;                          // [4][64]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int h = blockIdx.y, r0 = blockIdx.x * GLA_CHUNK, n = min(GLA_CHUNK, g.rows - r0);
-    const int cols = g.heads * g.dim_pad;
+    const int cols = g.heads * dim_pad, middle = min(GLA_MIDDLE, n - 1);
     pdl_wait_prior_grids();
     pdl_launch_dependents();
     const bf16* row0 = g.proj + (size_t)r0 * g.ld;
-    const float* b0 = g.decay + (size_t)r0 * cols + h * g.dim_pad;
-    const int kp = g.dim_pad / 8, vp = g.vdim_pad / 8, middle = min(GLA_MIDDLE, n - 1);
-    for (int i = tid; i < GLA_CHUNK * vp; i += GC_THREADS) {
-        const int t = i / vp, c = i - t * vp;
-        ops::att_cp_async16(smem_u32(vs + t * vrow + c * 16), row0 + (size_t)(t < n ? t : 0) * g.ld + g.v_off() + h * g.vdim_pad + c * 8, t < n ? 16 : 0);
-    }
-    ops::att_cp_async_commit();
-    uint4 qv[GC_BATCH], kv[GC_BATCH];
-    float4 bv[GC_BATCH][2];
-    auto load_rows = [&](int i0) {
+    const float* b0 = g.decay + (size_t)r0 * cols + h * dim_pad;
+    const float* st = g.chunk_state + ((size_t)blockIdx.x * g.heads + h) * dim_pad * vdim_pad;
+    constexpr int QV = GLA_CHUNK * GC_DIMS / 8 / GO_THREADS, SV = DV / 32;
+    uint4 qv[QV], kv[QV];
+    float4 bv[QV][2];
+    auto load_rows = [&](int d0) {                         // vector i: token i / 8, channels 8 (i % 8) on
 #pragma unroll
-        for (int j = 0; j < GC_BATCH; ++j) {
-            const int i = i0 + j * GC_THREADS, t = i / kp, d = (i - t * kp) * 8;
-            if (i >= GLA_CHUNK * kp || t >= n) continue;
-            const bf16* row = row0 + (size_t)t * g.ld + h * g.dim_pad + d;
+        for (int j = 0; j < QV; ++j) {
+            const int i = tid + j * GO_THREADS, t = i >> 3, d = d0 + (i & 7) * 8;
+            if (t >= n || d >= dim_pad) continue;
+            const bf16* row = row0 + (size_t)t * g.ld + h * dim_pad + d;
             qv[j] = *reinterpret_cast<const uint4*>(row);
             kv[j] = *reinterpret_cast<const uint4*>(row + g.k_off());
             bv[j][0] = load4(b0 + (size_t)t * cols + d);
             bv[j][1] = load4(b0 + (size_t)t * cols + d + 4);
         }
     };
-    load_rows(tid);
+    load_rows(0);
     bool steep = false;
-    for (int d = tid; d < g.dim_pad; d += GC_THREADS) {
+    for (int d = tid; d < dim_pad; d += GO_THREADS) {
         const float first = b0[d], mid = b0[(size_t)middle * cols + d], last = b0[(size_t)(n - 1) * cols + d];
         steep = steep || first - mid > GLA_HALF_LIMIT || mid - last > GLA_HALF_LIMIT;
         refs[d] = mid;
     }
     steep = __syncthreads_or(steep);
     const float4 zero4 = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int i0 = tid; i0 < GLA_CHUNK * kp; i0 += GC_BATCH * GC_THREADS) {
-        if (i0 > tid) load_rows(i0);
+    const int block = warp >> 2, quarter = warp & 3;       // this warp's 16 tokens; which 16 tokens they are scored against, which columns
+    const uint32_t q_at = (uint32_t)((block * 16 + (lane & 15)) * GC_ROW + (lane >> 4) * 16);
+    const bool scoring = !steep && quarter <= block;
+    float a[2][4], o[DV / 32][4];
 #pragma unroll
-        for (int j = 0; j < GC_BATCH; ++j) {
-            const int i = i0 + j * GC_THREADS, t = i / kp, d = (i - t * kp) * 8;
-            if (i >= GLA_CHUNK * kp) continue;
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) a[j][e] = 0.0f;
+#pragma unroll
+    for (int j = 0; j < DV / 32; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[j][e] = 0.0f;
+
+    for (int d0 = 0; d0 < dim_pad; d0 += GC_DIMS) {
+        const int dims = min(GC_DIMS, dim_pad - d0);
+        if (d0 > 0) load_rows(d0);
+        float4 sv[SV];
+        const int vq = vdim_pad / 4, count = dims * vq;
+#pragma unroll
+        for (int j = 0; j < SV; ++j) {
+            const int i = tid + j * GO_THREADS;
+            if (i < count) sv[j] = load4(st + (size_t)d0 * vdim_pad + i * 4);
+        }
+#pragma unroll
+        for (int j = 0; j < QV; ++j) {
+            const int i = tid + j * GO_THREADS, t = i >> 3, d = (i & 7) * 8;
             uint4 qh = make_uint4(0, 0, 0, 0), ql = qh, kh = qh, kl = qh;
-            if (t < n) {
-                const float4 f0 = steep ? zero4 : load4(refs + d), f1 = steep ? zero4 : load4(refs + d + 4);
+            if (t < n && d < dims) {
+                const float4 f0 = steep ? zero4 : load4(refs + d0 + d), f1 = steep ? zero4 : load4(refs + d0 + d + 4);
                 decayed8(qv[j], bv[j][0], bv[j][1], f0, f1, g.q_scale, qh, ql);
                 if (!steep) decayed8(kv[j], f0, f1, bv[j][0], bv[j][1], 1.0f, kh, kl);
             }
-            *reinterpret_cast<uint4*>(qhi + t * krow + d * 2) = qh;
-            *reinterpret_cast<uint4*>(qlo + t * krow + d * 2) = ql;
-            *reinterpret_cast<uint4*>(khi + t * wide + d * 2) = kh;
-            *reinterpret_cast<uint4*>(klo + t * wide + d * 2) = kl;
+            *reinterpret_cast<uint4*>(qhi + t * GC_ROW + d * 2) = qh;
+            *reinterpret_cast<uint4*>(qlo + t * GC_ROW + d * 2) = ql;
+            *reinterpret_cast<uint4*>(khi + t * GC_ROW + d * 2) = kh;
+            *reinterpret_cast<uint4*>(klo + t * GC_ROW + d * 2) = kl;
         }
-    }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();
-    // state rows on their way: 64 x vdim_pad, four columns at a time
-    const float* st = g.chunk_state + ((size_t)blockIdx.x * g.heads + h) * g.dim_pad * g.vdim_pad;
-    constexpr int SV = DV / 16;
-    float4 sv[SV];
-    auto load_state = [&](int d0) {
-        const int count = min(GLA_CHUNK, g.dim_pad - d0) * (g.vdim_pad / 4);
 #pragma unroll
         for (int j = 0; j < SV; ++j) {
-            const int i = tid + j * GC_THREADS;
-            if (i < count) sv[j] = load4(st + (size_t)d0 * g.vdim_pad + i * 4);
-        }
-    };
-    load_state(0);
-
-    const int block = warp >> 1, half = warp & 1;          // this warp's 16 tokens; which 32 tokens they are scored against, which columns
-    const uint32_t q_at = (uint32_t)((block * 16 + (lane & 15)) * krow + (lane >> 4) * 16);
-    if (!steep) {
-        if (half * 32 <= block * 16 + 15) {
-            float a[4][4];
-#pragma unroll
-            for (int j = 0; j < 4; ++j)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) a[j][e] = 0.0f;
-            const uint32_t k_at = (uint32_t)((half * 32 + (lane & 7) + (lane >> 4) * 8) * wide + ((lane >> 3) & 1) * 16);
-            for (int c = 0; c < g.dim_pad / 16; ++c) {
-                uint32_t qh[4], ql[4];
-                ldmatrix_x4(qh, smem_u32(qhi) + q_at + c * 32);
-                ldmatrix_x4(ql, smem_u32(qlo) + q_at + c * 32);
-#pragma unroll
-                for (int j = 0; j < 2; ++j) {
-                    if (half * 32 + j * 16 > block * 16) continue;
-                    uint32_t kh[4], kl[4];
-                    ldmatrix_x4(kh, smem_u32(khi) + k_at + j * 16 * wide + c * 32);
-                    ldmatrix_x4(kl, smem_u32(klo) + k_at + j * 16 * wide + c * 32);
-#pragma unroll
-                    for (int i = 0; i < 2; ++i) {
-                        mma_bf16(a[2 * j + i], qh, kh[2 * i], kh[2 * i + 1]);
-                        mma_bf16(a[2 * j + i], ql, kh[2 * i], kh[2 * i + 1]);
-                        mma_bf16(a[2 * j + i], qh, kl[2 * i], kl[2 * i + 1]);
-                    }
-                }
-            }
-#pragma unroll
-            for (int j = 0; j < 4; ++j)
-#pragma unroll
-                for (int i = 0; i < 2; ++i) {
-                    const int t = block * 16 + (lane >> 2) + i * 8, s = half * 32 + j * 8 + (lane & 3) * 2;
-                    uint32_t hi, lo;
-                    split_bf16(s <= t ? a[j][2 * i] : 0.0f, s + 1 <= t ? a[j][2 * i + 1] : 0.0f, hi, lo);
-                    *reinterpret_cast<uint32_t*>(ahi + t * GO_AROW + s * 2) = hi;
-                    *reinterpret_cast<uint32_t*>(alo + t * GO_AROW + s * 2) = lo;
-                }
-        }
-    } else {                                               // a warp per token pair
-        for (int u = warp; u < GLA_CHUNK * GLA_CHUNK; u += GC_THREADS / 32) {
-            const int t = u / GLA_CHUNK, s = u - t * GLA_CHUNK;
-            float sum = 0.0f;
-            if (s <= t && t < n)
-                for (int d = lane; d < g.dim_pad; d += 32)
-                    sum = fmaf(to_f32(row0[(size_t)t * g.ld + h * g.dim_pad + d]) * g.q_scale * to_f32(row0[(size_t)s * g.ld + g.k_off() + h * g.dim_pad + d]),
-                               ex2_approx((b0[(size_t)t * cols + d] - b0[(size_t)s * cols + d]) * GLA_LOG2E), sum);
-            sum = ops::warp_sum(sum);
-            const bf16 hi = __float2bfloat16_rn(sum);
-            if (lane == 0) {
-                reinterpret_cast<bf16*>(ahi + t * GO_AROW)[s] = hi;
-                reinterpret_cast<bf16*>(alo + t * GO_AROW)[s] = __float2bfloat16_rn(sum - to_f32(hi));
-            }
-        }
-    }
-    __syncthreads();                                       // the scores are there, the keys have been used
-
-    // ---- o = scores V + (q 2^(b - ref)) (2^ref S): the warp takes every other 16 value columns ----
-    float o[DV / 16][4];
-#pragma unroll
-    for (int j = 0; j < DV / 16; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) o[j][e] = 0.0f;
-    auto store_state = [&](int d0) {
-        const int vq = g.vdim_pad / 4, count = min(GLA_CHUNK, g.dim_pad - d0) * vq;
-#pragma unroll
-        for (int j = 0; j < SV; ++j) {
-            const int i = tid + j * GC_THREADS;
+            const int i = tid + j * GO_THREADS;
             if (i >= count) continue;
             const int d = i / vq, v = (i - d * vq) * 4;
             const float f = steep ? 1.0f : ex2_approx(refs[d0 + d] * GLA_LOG2E);
             uint2 hi, lo;
             split_bf16(sv[j].x * f, sv[j].y * f, hi.x, lo.x);
             split_bf16(sv[j].z * f, sv[j].w * f, hi.y, lo.y);
-            *reinterpret_cast<uint2*>(khi + d * wide + v * 2) = hi;
-            *reinterpret_cast<uint2*>(klo + d * wide + v * 2) = lo;
+            *reinterpret_cast<uint2*>(shi + d * vrow + v * 2) = hi;
+            *reinterpret_cast<uint2*>(slo + d * vrow + v * 2) = lo;
         }
-    };
-    store_state(0);
-    const uint32_t a_at = (uint32_t)((block * 16 + (lane & 15)) * GO_AROW + (lane >> 4) * 16);
-    for (int kk = 0; kk <= block; ++kk) {
-        uint32_t xh[4], xl[4];
-        ldmatrix_x4(xh, smem_u32(ahi) + a_at + kk * 32);
-        ldmatrix_x4(xl, smem_u32(alo) + a_at + kk * 32);
-#pragma unroll
-        for (int j = 0; j < DV / 32; ++j) {
-            const int v0 = (2 * j + half) * 16;
-            if (v0 >= g.vdim_pad) continue;
-            uint32_t b[4];
-            ops::att_ldmatrix_x4_trans(b, smem_u32(vs) + (kk * 16 + (lane & 15)) * vrow + (v0 + (lane >> 4) * 8) * 2);
-            mma_bf16(o[2 * j], xh, b[0], b[1]);
-            mma_bf16(o[2 * j + 1], xh, b[2], b[3]);
-            mma_bf16(o[2 * j], xl, b[0], b[1]);
-            mma_bf16(o[2 * j + 1], xl, b[2], b[3]);
-        }
-    }
-    for (int d0 = 0; d0 < g.dim_pad; d0 += GLA_CHUNK) {
-        __syncthreads();                                   // this part of the state is in shared memory
-        if (d0 + GLA_CHUNK < g.dim_pad) load_state(d0 + GLA_CHUNK);
-        const int steps = min(GLA_CHUNK, g.dim_pad - d0) / 16;
-        for (int c = 0; c < steps; ++c) {
+        __syncthreads();
+        const uint32_t k_at = (uint32_t)((quarter * 16 + (lane & 7) + (lane >> 4) * 8) * GC_ROW + ((lane >> 3) & 1) * 16);
+        for (int c = 0; c < dims / 16; ++c) {
             uint32_t qh[4], ql[4];
-            ldmatrix_x4(qh, smem_u32(qhi) + q_at + (d0 + c * 16) * 2);
-            ldmatrix_x4(ql, smem_u32(qlo) + q_at + (d0 + c * 16) * 2);
+            ldmatrix_x4(qh, smem_u32(qhi) + q_at + c * 32);
+            ldmatrix_x4(ql, smem_u32(qlo) + q_at + c * 32);
+            if (scoring) {
+                uint32_t kh[4], kl[4];
+                ldmatrix_x4(kh, smem_u32(khi) + k_at + c * 32);
+                ldmatrix_x4(kl, smem_u32(klo) + k_at + c * 32);
 #pragma unroll
-            for (int j = 0; j < DV / 32; ++j) {
-                const int v0 = (2 * j + half) * 16;
-                if (v0 >= g.vdim_pad) continue;
-                const uint32_t at = (uint32_t)((c * 16 + (lane & 15)) * wide + (v0 + (lane >> 4) * 8) * 2);
+                for (int i = 0; i < 2; ++i) {
+                    mma_bf16(a[i], qh, kh[2 * i], kh[2 * i + 1]);
+                    mma_bf16(a[i], ql, kh[2 * i], kh[2 * i + 1]);
+                    mma_bf16(a[i], qh, kl[2 * i], kl[2 * i + 1]);
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < DV / 64; ++j) {            // the warp takes every fourth 16 value columns
+                const int v0 = (4 * j + quarter) * 16;
+                if (v0 >= vdim_pad) continue;
+                const uint32_t at = (uint32_t)((c * 16 + (lane & 15)) * vrow + (v0 + (lane >> 4) * 8) * 2);
                 uint32_t bh[4], bl[4];
-                ops::att_ldmatrix_x4_trans(bh, smem_u32(khi) + at);
-                ops::att_ldmatrix_x4_trans(bl, smem_u32(klo) + at);
+                ops::att_ldmatrix_x4_trans(bh, smem_u32(shi) + at);
+                ops::att_ldmatrix_x4_trans(bl, smem_u32(slo) + at);
 #pragma unroll
                 for (int i = 0; i < 2; ++i) {
                     mma_bf16(o[2 * j + i], qh, bh[2 * i], bh[2 * i + 1]);
@@ -565,9 +495,60 @@ gla_chunk_out_kernel(const GlaArgs<bf16> g)
                 }
             }
         }
-        if (d0 + GLA_CHUNK < g.dim_pad) {
-            __syncthreads();                               // the part before has been used
-            store_state(d0 + GLA_CHUNK);
+        __syncthreads();                                   // this part has been used
+    }
+    // ---- the values over the state's rows, the scores over the queries ----
+    uint8_t *vs = shi, *ahi = qhi, *alo = qlo;
+    const int vp = vdim_pad / 8;
+    for (int i = tid; i < GLA_CHUNK * vp; i += GO_THREADS) {
+        const int t = i / vp, c = i - t * vp;
+        ops::att_cp_async16(smem_u32(vs + t * vrow + c * 16), row0 + (size_t)(t < n ? t : 0) * g.ld + g.v_off() + h * vdim_pad + c * 8, t < n ? 16 : 0);
+    }
+    ops::att_cp_async_commit();
+    if (scoring) {
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                const int t = block * 16 + (lane >> 2) + i * 8, s = quarter * 16 + j * 8 + (lane & 3) * 2;
+                uint32_t hi, lo;
+                split_bf16(s <= t ? a[j][2 * i] : 0.0f, s + 1 <= t ? a[j][2 * i + 1] : 0.0f, hi, lo);
+                *reinterpret_cast<uint32_t*>(ahi + t * GC_ROW + s * 2) = hi;
+                *reinterpret_cast<uint32_t*>(alo + t * GC_ROW + s * 2) = lo;
+            }
+    }
+    if (steep) {                                           // a warp per token pair
+        for (int u = warp; u < GLA_CHUNK * GLA_CHUNK; u += GO_THREADS / 32) {
+            const int t = u / GLA_CHUNK, s = u - t * GLA_CHUNK;
+            float sum = 0.0f;
+            if (s <= t && t < n)
+                for (int d = lane; d < dim_pad; d += 32)
+                    sum = fmaf(to_f32(row0[(size_t)t * g.ld + h * dim_pad + d]) * g.q_scale * to_f32(row0[(size_t)s * g.ld + g.k_off() + h * dim_pad + d]),
+                               ex2_approx((b0[(size_t)t * cols + d] - b0[(size_t)s * cols + d]) * GLA_LOG2E), sum);
+            sum = ops::warp_sum(sum);
+            const bf16 hi = __float2bfloat16_rn(sum);
+            if (lane == 0) {
+                reinterpret_cast<bf16*>(ahi + t * GC_ROW)[s] = hi;
+                reinterpret_cast<bf16*>(alo + t * GC_ROW)[s] = __float2bfloat16_rn(sum - to_f32(hi));
+            }
+        }
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    for (int kk = 0; kk <= block; ++kk) {
+        uint32_t xh[4], xl[4];
+        ldmatrix_x4(xh, smem_u32(ahi) + q_at + kk * 32);
+        ldmatrix_x4(xl, smem_u32(alo) + q_at + kk * 32);
+#pragma unroll
+        for (int j = 0; j < DV / 64; ++j) {
+            const int v0 = (4 * j + quarter) * 16;
+            if (v0 >= vdim_pad) continue;
+            uint32_t b[4];
+            ops::att_ldmatrix_x4_trans(b, smem_u32(vs) + (kk * 16 + (lane & 15)) * vrow + (v0 + (lane >> 4) * 8) * 2);
+            mma_bf16(o[2 * j], xh, b[0], b[1]);
+            mma_bf16(o[2 * j + 1], xh, b[2], b[3]);
+            mma_bf16(o[2 * j], xl, b[0], b[1]);
+            mma_bf16(o[2 * j + 1], xl, b[2], b[3]);
         }
     }
     // ---- norm over the head's columns, gate, store ----
@@ -575,23 +556,23 @@ gla_chunk_out_kernel(const GlaArgs<bf16> g)
     for (int i = 0; i < 2; ++i) {
         float ss = 0.0f;
 #pragma unroll
-        for (int j = 0; j < DV / 16; ++j) ss = fmaf(o[j][2 * i], o[j][2 * i], fmaf(o[j][2 * i + 1], o[j][2 * i + 1], ss));
+        for (int j = 0; j < DV / 32; ++j) ss = fmaf(o[j][2 * i], o[j][2 * i], fmaf(o[j][2 * i + 1], o[j][2 * i + 1], ss));
         ss += __shfl_xor_sync(0xffffffffu, ss, 1);
         ss += __shfl_xor_sync(0xffffffffu, ss, 2);
-        if ((lane & 3) == 0) sums[half * GLA_CHUNK + block * 16 + (lane >> 2) + i * 8] = ss;
+        if ((lane & 3) == 0) sums[quarter * GLA_CHUNK + block * 16 + (lane >> 2) + i * 8] = ss;
     }
     __syncthreads();
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
         const int t = block * 16 + (lane >> 2) + i * 8;
         if (t >= n) continue;
-        const float ir = inv_rms(sums[t] + sums[GLA_CHUNK + t], g.vdim, g.eps);
-        const bf16* gate = row0 + (size_t)t * g.ld + g.gate_off() + h * g.vdim_pad;
-        bf16* out = g.out + ((size_t)(r0 + t) * g.heads + h) * g.vdim_pad;
+        const float ir = inv_rms((sums[t] + sums[GLA_CHUNK + t]) + (sums[2 * GLA_CHUNK + t] + sums[3 * GLA_CHUNK + t]), g.vdim, g.eps);
+        const bf16* gate = row0 + (size_t)t * g.ld + g.gate_off() + h * vdim_pad;
+        bf16* out = g.out + ((size_t)(r0 + t) * g.heads + h) * vdim_pad;
 #pragma unroll
-        for (int j = 0; j < DV / 16; ++j) {
-            const int v = (2 * (j >> 1) + half) * 16 + (j & 1) * 8 + (lane & 3) * 2;
-            if (v >= g.vdim_pad) continue;
+        for (int j = 0; j < DV / 32; ++j) {
+            const int v = (4 * (j >> 1) + quarter) * 16 + (j & 1) * 8 + (lane & 3) * 2;
+            if (v >= vdim_pad) continue;
             const float2 w = *reinterpret_cast<const float2*>(g.head_norm + v);
             const uint32_t z = *reinterpret_cast<const uint32_t*>(gate + v);
             const float z0 = __uint_as_float(z << 16), z1 = __uint_as_float(z & 0xffff0000u);
