@@ -112,7 +112,7 @@ typedef struct twm_dense_buffers {
     void* proj;                  /* [max_rows][widest w_in] */
     void* att;                   /* [max_rows][widest heads*vdim_pad] */
     void* act;                   /* [max_rows][widest ff_pad], routed: [max_rows * top][ff_pad] */
-    float* vec;                  /* decode: [widest w_in + widest heads*vdim_pad + widest act + widest experts], each up to a multiple of 16 */
+    float* vec;                  /* decode: [widest w_in + widest heads*vdim_pad + widest act (routed: top*ff_pad) + width_pad] */
     float* logits;               /* [max_want][vocab] */
     /* LATENT (NULL without): the tokens a step's queries can see, at most max_keys */
     int max_keys;

@@ -203,6 +203,11 @@ __device__ __forceinline__ uint4 lds128(const void* p) {
     return v;
 }
 
+__device__ __forceinline__ int ld_cg_s32(const int* p) {
+    int v;
+    asm volatile("ld.global.cg.s32 %0, [%1];" : "=r"(v) : "l"(p) : "memory");
+    return v;
+}
 __device__ __forceinline__ float ld_cg_f32(const float* p) {
     float v;
     asm volatile("ld.global.cg.f32 %0, [%1];" : "=f"(v) : "l"(p));

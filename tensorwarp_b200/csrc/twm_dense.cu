@@ -760,7 +760,7 @@ twm_status gemv(GemvArgs<T> g, int sms, int flags, void* stream)
         return invalid("cuTensorMapEncodeTiled refused a map of the decode product");
     const size_t row_bytes = (size_t)g.ldw * sizeof(T);
     const int parts = ROUTE == ROUTE_COLUMNS ? g.router.top : 1;
-    const size_t act = gemv_smem_bytes(row_bytes, parts, 0), limit = kSmemLimit - 16 * 1024;      // static shared memory beside it
+    const size_t act = gemv_smem_bytes(row_bytes, parts, 0), limit = kSmemLimit - 8 * 1024;      // static shared memory beside it
     if (act + 2 * GV_STAGE > limit) return invalid("an input row does not fit shared memory");
     g.stages = (int)std::min<size_t>(GV_MAX_STAGES, (limit - act) / GV_STAGE);
     return launch("gemv", gemv_kernel<T, PRO, EPI, ROUTE>, dim3(grid), GV_THREADS, gemv_smem_bytes(row_bytes, parts, g.stages), flags, stream, 0, g);
@@ -840,7 +840,7 @@ twm_status decode(const twm_dense_model* m, const twm_dense_buffers* b, int want
     float* proj = b->vec;
     float* att = proj + widest_in;
     float* act = att + widest_out;
-    float* router = act + widest_act;
+    float* h = act + widest_act;                         // a routed feed-forward's input row
     auto args = [&](const void* w, int N, int ldw, float* out) {
         GemvArgs<T> g = {};
         g.w = (const T*)w; g.N = N; g.ldw = ldw; g.out = out; g.meta = b->meta;
@@ -877,16 +877,15 @@ twm_status decode(const twm_dense_model* m, const twm_dense_buffers* b, int want
         y = b->y; y_norm = l.norm1;
         if (l.experts > 0) {
             const RouterArgs r = {l.experts, l.top, l.groups, l.keep};
-            g = with_residual(args(l.w_router, l.experts, wp, router), nullptr);
-            g.pre_norm = l.pre2;
-            if (l.pre2) TRY((gemv<T, PRO_NORM>(g, sms, flags, stream)));
-            else TRY((gemv<T, PRO_RESIDUAL>(g, sms, flags, stream)));
+            g = with_residual(args(nullptr, 0, wp, nullptr), nullptr);
+            RouterDecodeArgs<T> q;
+            q.src = g.src; q.x_out = g.x_out; q.h_out = h; q.pre_norm = l.pre2; q.w = (const T*)l.w_router; q.meta = b->meta; q.router = r;
+            q.ids = b->route; q.weights = b->route_weight;
+            TRY(launch("router_decode", router_decode_kernel<T>, dim3(RD_CTAS), RD_THREADS, router_decode_smem_bytes<T>(wp), flags, stream, RD_CTAS, q));
             g = args(l.w_gate_up, l.top * l.ff_pad, wp, act);
-            g.src.x_in = x; g.src.eps = m->eps; g.src.width = m->width; g.src.wp = wp;
-            g.pre_norm = l.pre2;
-            g.router = r; g.expert_rows = l.ff_pad; g.logits = router; g.ids = b->route; g.weights = b->route_weight;
-            if (l.pre2) TRY((gemv<T, PRO_NORM, TWM_EPI_RELU2, ROUTE_ROWS>(g, sms, flags, stream)));
-            else TRY((gemv<T, PRO_RESIDUAL, TWM_EPI_RELU2, ROUTE_ROWS>(g, sms, flags, stream)));
+            g.vec = h;
+            g.router = r; g.expert_rows = l.ff_pad; g.ids = b->route; g.weights = b->route_weight;
+            TRY((gemv<T, PRO_VEC, TWM_EPI_RELU2, ROUTE_ROWS>(g, sms, flags, stream)));
             GemvArgs<T> d = args(l.w_down, m->width, l.ff_pad, b->y);
             d.vec = act;
             d.router = r; d.expert_rows = m->width; d.ids = b->route; d.weights = b->route_weight;
@@ -904,9 +903,9 @@ twm_status decode(const twm_dense_model* m, const twm_dense_buffers* b, int want
         }
     }
     if (want_logits) {
-        GemvArgs<T> h = with_residual(args(m->head, m->vocab, wp, b->logits), nullptr);
-        h.pre_norm = m->final_norm;
-        TRY((gemv<T, PRO_NORM>(h, sms, flags, stream)));
+        GemvArgs<T> g = with_residual(args(m->head, m->vocab, wp, b->logits), nullptr);
+        g.pre_norm = m->final_norm;
+        TRY((gemv<T, PRO_NORM>(g, sms, flags, stream)));
     }
     return TWM_OK;
 }

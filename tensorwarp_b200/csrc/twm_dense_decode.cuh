@@ -18,9 +18,11 @@
 // but the attention.
 //
 // Routed products (experts) differ in where a row comes from.  ROUTE_ROWS (up): the `top` chosen experts' rows, one
-// expert after the other, are one long list of rows; the first warp makes the choice from the router's logits.
-// ROUTE_COLUMNS (down): a row is the chosen experts' rows side by side, and the input is their activations side by
-// side, each times its expert's weight; so the sum over experts is part of the product.
+// expert after the other, are one long list of rows.  ROUTE_COLUMNS (down): a row is the chosen experts' rows side by
+// side, and the input is their activations side by side, each times its expert's weight; so the sum over experts is
+// part of the product.  The choice is made by router_decode_kernel, two launches ahead of the down product: the up
+// product lets that one start only after its own wait for the router, so the down product takes the choice as soon
+// as it starts and streams its weights while the up product still runs.
 #pragma once
 
 #include "twm_dense_moe.cuh"
@@ -56,13 +58,12 @@ struct GemvArgs {
     float* shift_state;
     const float* pre_norm;      // PRO_NORM: the input row is rms_norm(residual row) * pre_norm
     const int* meta;
-    // routed: W is [experts][expert_rows][ldw].  ROUTE_ROWS: N = top * expert_rows, the choice is made from `logits` and left
-    // in ids and weights.  ROUTE_COLUMNS: N = expert_rows, vec is [top][ldw].
+    // routed: W is [experts][expert_rows][ldw].  ROUTE_ROWS: N = top * expert_rows.  ROUTE_COLUMNS: N = expert_rows, vec is
+    // [top][ldw].
     RouterArgs router;
     int expert_rows;
-    const float* logits;
-    int* ids;
-    float* weights;
+    const int* ids;
+    const float* weights;
     alignas(64) CUtensorMap w_map;      // W's rows as 64-bit words, boxes of 256 words x 4 rows
 };
 
@@ -79,7 +80,6 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
     using V = Vec<T>;
     constexpr bool GATED = EPI == TWM_EPI_GELU_GLU;
     extern __shared__ __align__(128) uint8_t gemv_smem[];
-    __shared__ float route_s[ROUTE == ROUTE_ROWS ? 2 * MOE_MAX_EXPERTS : 1];
     __shared__ int ids_s[ROUTE != ROUTE_NONE ? MOE_MAX_TOP : 1];
     uint8_t* ring = gemv_smem;
     T* as = reinterpret_cast<T*>(gemv_smem + (size_t)g.stages * GV_STAGE);
@@ -116,11 +116,18 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
         mbar_fence_init();
     }
     __syncthreads();
-    pdl_launch_dependents();
+    if (ROUTE != ROUTE_ROWS) pdl_launch_dependents();
 
     if (warp == GV_CONSUMERS / 32) {
         // ------------------------------------------------------------ producer --
-        if (ROUTE != ROUTE_NONE) named_bar_sync(2, 64);              // the choice is in ids_s
+        if (ROUTE == ROUTE_ROWS) {
+            pdl_wait_prior_grids();                                  // for the router's choice ...
+            pdl_launch_dependents();                                 // ... which the next launch relies on from its start
+        }
+        if (ROUTE != ROUTE_NONE) {
+            if (lane < g.router.top) ids_s[lane] = ld_cg_s32(g.ids + lane);
+            __syncwarp();
+        }
         if (elect_one()) {
             int slot = 0, c = 0, gi = 0, piece = 0, part = 0, first = 0, second_first = 0;
             uint32_t phase = 0;
@@ -156,25 +163,14 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
 
     // ------------------------------------------------------- prologue (256 threads) --
     pdl_wait_prior_grids();
-    if (ROUTE != ROUTE_NONE && warp == 0) {
-        int id = 0;
-        if (ROUTE == ROUTE_ROWS) {
-            float weight;
-            route_warp(g.logits, g.router, route_s, route_s + MOE_MAX_EXPERTS, lane, id, weight);
-            if (blockIdx.x == 0 && lane < g.router.top) { g.ids[lane] = id; g.weights[lane] = weight; }
-        } else if (lane < g.router.top) {
-            id = g.ids[lane];
-        }
-        if (lane < g.router.top) ids_s[lane] = id;
-        named_bar_sync(2, 64);
-    }
+    if (ROUTE == ROUTE_ROWS) pdl_launch_dependents();
     if (ROUTE == ROUTE_COLUMNS) {
-        for (int s = 0; s < g.router.top; ++s) {
-            const float ws = g.weights[s];
-            T* dst = as + (size_t)s * pieces * (GV_PIECE / sizeof(T));
-            for (int i = tid; i < (g.ldw >> 2); i += GV_CONSUMERS) {
+        for (int i = tid; i < (g.ldw >> 2); i += GV_CONSUMERS) {
+#pragma unroll 8
+            for (int s = 0; s < g.router.top; ++s) {
+                const float ws = g.weights[s];
                 const float4 v = reinterpret_cast<const float4*>(g.vec + (size_t)s * g.ldw)[i];
-                store4<T>(dst + i * 4, make_float4(v.x * ws, v.y * ws, v.z * ws, v.w * ws));
+                store4<T>(as + (size_t)s * pieces * (GV_PIECE / sizeof(T)) + i * 4, make_float4(v.x * ws, v.y * ws, v.z * ws, v.w * ws));
             }
         }
     } else if (PRO == PRO_VEC) {
@@ -309,6 +305,94 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
                                                                                   : epilogue_value<EPI>(sum(row + 4 * which));
             }
         }
+    }
+}
+
+// One token's router: one cluster of CTAs.  Every CTA makes the feed-forward's input row (the residual stream brought up to
+// date, normed) for itself, a warp takes the logits of every (8 * CTAs)-th expert, and the first CTA's first warp chooses.
+// Leaves the residual row, the input row in FP32, and the choice.
+constexpr int RD_THREADS = 256, RD_CTAS = 8;
+template <typename T>
+struct RouterDecodeArgs {
+    ResidualSource<T> src;
+    float* x_out;               // [wp]
+    float* h_out;               // [wp]
+    const float* pre_norm;      // [wp] or null
+    const T* w;                 // [experts][wp]
+    const int* meta;
+    RouterArgs router;
+    int* ids;
+    float* weights;
+};
+template <typename T>
+__host__ inline size_t router_decode_smem_bytes(int wp) { return sizeof(float) * 2 * (size_t)wp; }
+template <typename T>
+__global__ void __launch_bounds__(RD_THREADS)
+router_decode_kernel(const RouterDecodeArgs<T> g)
+{
+    using V = Vec<T>;
+    pdl_launch_dependents();
+    asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");      // waited for before the first push
+    extern __shared__ __align__(16) float rd_smem[];
+    __shared__ float logits[MOE_MAX_EXPERTS], scores[MOE_MAX_EXPERTS], group_scores[MOE_MAX_EXPERTS], red[32];
+    const int wp = g.src.wp, nvec = wp >> 2, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int first = blockIdx.x * (RD_THREADS / 32) + warp, stride = gridDim.x * (RD_THREADS / 32);
+    float4* hs = reinterpret_cast<float4*>(rd_smem);       // [wp]
+    float4* ys = hs + nvec;
+    for (int e = first; e < g.router.experts; e += stride)
+        if (lane == 0) l2_prefetch_bulk(g.w + (size_t)e * wp, (uint32_t)(wp * sizeof(T)));
+    pdl_wait_prior_grids();
+    const bool writer = blockIdx.x == 0, joined = g.src.y != nullptr, normed = joined && g.src.y_norm != nullptr;
+    const int tok = g.src.tokens != nullptr ? g.src.tokens[0] : 0, pos = g.meta[0];
+    ResidualSource<T> plain = g.src;                       // the row without what joins it
+    plain.y = nullptr;
+    float ss = 0.0f;
+    for (int i = tid; i < nvec; i += RD_THREADS) {         // every thread keeps to its own elements
+        const float4 y = joined ? reinterpret_cast<const float4*>(g.src.y)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+        hs[i] = plain.at(0, pos, tok, i, 1.0f);
+        ys[i] = y;
+        ss += ops::sumsq4(y);
+    }
+    const float ir = normed ? inv_rms(group_sum(ss, red, RD_THREADS, 1), g.src.width, g.src.eps) : 1.0f;
+    ss = 0.0f;
+    for (int i = tid; i < nvec; i += RD_THREADS) {
+        float4 x = hs[i], n = make_float4(1.f, 1.f, 1.f, 1.f);
+        if (normed) n = __ldg(reinterpret_cast<const float4*>(g.src.y_norm) + i);
+        const float4 y = scale4(ys[i], ir, n);
+        x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w;
+        hs[i] = x;
+        if (writer) reinterpret_cast<float4*>(g.x_out)[i] = x;
+        ss += ops::sumsq4(x);
+    }
+    const float fr = g.pre_norm != nullptr ? inv_rms(group_sum(ss, red, RD_THREADS, 1), g.src.width, g.src.eps) : 1.0f;
+    for (int i = tid; i < nvec; i += RD_THREADS) {
+        if (g.pre_norm != nullptr) hs[i] = scale4(hs[i], fr, __ldg(reinterpret_cast<const float4*>(g.pre_norm) + i));
+        if (writer) reinterpret_cast<float4*>(g.h_out)[i] = hs[i];
+    }
+    __syncthreads();
+    asm volatile("barrier.cluster.wait.aligned;" ::: "memory");    // every CTA of the cluster has started
+    for (int e = first; e < g.router.experts; e += stride) {
+        const uint4* w = reinterpret_cast<const uint4*>(g.w + (size_t)e * wp);
+        float s = 0.0f;
+#pragma unroll 4
+        for (int c = lane; c < wp / V::N; c += 32) {
+            float f[V::N];
+            V::unpack(__ldg(w + c), f);
+#pragma unroll
+            for (int k = 0; k < V::N; k += 4) {
+                const float4 h = hs[c * (V::N / 4) + k / 4];
+                s = fmaf(f[k], h.x, fmaf(f[k + 1], h.y, fmaf(f[k + 2], h.z, fmaf(f[k + 3], h.w, s))));
+            }
+        }
+        s = ops::warp_sum(s);
+        if (lane == 0) st_cluster_f32(mapa_shared(smem_u32(logits + e), 0), s);
+    }
+    cluster_sync_all();
+    if (writer && warp == 0) {
+        int id;
+        float weight;
+        route_warp(logits, g.router, scores, group_scores, lane, id, weight);
+        if (lane < g.router.top) { g.ids[lane] = id; g.weights[lane] = weight; }
     }
 }
 

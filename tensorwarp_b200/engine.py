@@ -77,7 +77,7 @@ class DenseEngine:
         self._buf = dict(meta=zeros(8, dtype=i32), tokens=zeros(rows, dtype=i32), want=zeros(self.max_want, dtype=i32),
                          x0=zeros(rows, wp, dtype=f32), x1=zeros(rows, wp, dtype=f32), y=zeros(rows, wp, dtype=f32),
                          a=zeros(rows, wp, dtype=dt), proj=zeros(rows, w_in, dtype=dt), att=zeros(rows, w_att, dtype=dt),
-                         act=zeros(rows * slots_per_row, w_ff, dtype=dt), vec=zeros(w_in + w_att + w_act + experts, dtype=f32),
+                         act=zeros(rows * slots_per_row, w_ff, dtype=dt), vec=zeros(w_in + w_att + w_act + wp, dtype=f32),
                          logits=zeros(self.max_want, self.vocab, dtype=f32))
         b = _dense.Buffers(max_rows=rows, max_want=self.max_want)
         latent = [x for x in lays if x.mixer == _dense.MIX_LATENT]
