@@ -673,8 +673,13 @@ twm_status prefill(const twm_dense_model* m, const twm_dense_buffers* b, int row
         // rows per CTA: enough CTAs to fill the machine several times; a shifted run computes one row more than it has
         const int rpc = next.shift ? (rows >= 4096 ? 8 : rows >= 1024 ? 4 : rows >= 256 ? 2 : 1) : 1;
         const int per = (wp / 4 + ROW_THREADS - 1) / ROW_THREADS;
-        auto kernel = per <= 1 ? residual_rows_kernel<T, 1> : per <= 2 ? residual_rows_kernel<T, 2> :
-                      per <= 4 ? residual_rows_kernel<T, 4> : per <= 8 ? residual_rows_kernel<T, 8> : residual_rows_kernel<T, 0>;
+        const bool full = next.pre_norm || next.step || next.n_clear || routed.rows;
+        auto pick = [&](auto f) {
+            constexpr bool F = decltype(f)::value;
+            return per <= 1 ? residual_rows_kernel<T, 1, F> : per <= 2 ? residual_rows_kernel<T, 2, F> : per <= 4 ? residual_rows_kernel<T, 4, F> :
+                   per <= 8 ? residual_rows_kernel<T, 8, F> : residual_rows_kernel<T, 0, F>;
+        };
+        auto kernel = full ? pick(std::true_type()) : pick(std::false_type());
         const twm_status st = launch("residual_rows", kernel, dim3((rows + rpc - 1) / rpc), ROW_THREADS,
                                      per <= 8 ? 0 : sizeof(float) * (size_t)wp, flags, stream, 0, source(next.step), x_next,
                                      want_a ? (T*)b->a : (T*)nullptr, next.shift, next.shift_state, next.pre_norm, b->meta, rows, rpc,

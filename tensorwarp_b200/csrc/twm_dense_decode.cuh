@@ -135,7 +135,11 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
                 if (it >= g.stages && !mbar_wait_bounded(&empty[slot], phase, abort_flag)) break;
                 uint8_t* dst = ring + (size_t)slot * GV_STAGE;
                 const int o0 = group_first(gi);
-                if (c == 0) { first = physical(o0); second_first = physical(stream + o0); }
+                if (ROUTE == ROUTE_NONE) {
+                    piece = c; first = o0; second_first = stream + o0;
+                } else if (c == 0) {
+                    first = physical(o0); second_first = physical(stream + o0);
+                }
                 const int matrix = ROUTE == ROUTE_COLUMNS ? ids_s[part] * g.expert_rows : 0;
                 // a full group's four rows lie together: an expert's rows are a multiple of 16.  Routed products have nothing to gain
                 // from row copies: by the time the choice is known the map has been fetched.
@@ -153,7 +157,7 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
                         bulk_g2s(dst + (r + OUT_ROWS) * GV_PIECE, src + (size_t)(matrix + physical(stream + o0 + r)) * row_bytes, (uint32_t)bytes,
                                  &full[slot]);
                 }
-                if (++piece == pieces) { piece = 0; ++part; }
+                if (ROUTE != ROUTE_NONE && ++piece == pieces) { piece = 0; ++part; }
                 if (++c == chunks) { c = 0; part = 0; ++gi; }
                 if (++slot == g.stages) { slot = 0; if (it >= g.stages) phase ^= 1u; }
             }
@@ -198,7 +202,9 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
             return st_before != nullptr ? reinterpret_cast<const float4*>(st_before)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
         };
         constexpr int PER = 4;
-        if (nvec <= PER * GV_CONSUMERS && g.src.tokens == nullptr) {
+        // without a norm of its own the input is taken this way only where nothing but a normed sublayer output joins
+        const bool plain = g.src.y != nullptr && g.src.y_norm != nullptr && g.src.step == nullptr;
+        if (nvec <= PER * GV_CONSUMERS && g.src.tokens == nullptr && (PRO == PRO_NORM || plain)) {
             // rows of up to 4096: everything is requested before the first use
             const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
             float4 x[PER], y[PER], before[PER];
@@ -206,12 +212,12 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
             for (int j = 0; j < PER; ++j) {
                 const int i = tid + j * GV_CONSUMERS;
                 const bool in = i < nvec;
-                y[j] = in && g.src.y != nullptr ? reinterpret_cast<const float4*>(g.src.y)[i] : zero;
+                y[j] = in && (PRO != PRO_NORM || g.src.y != nullptr) ? reinterpret_cast<const float4*>(g.src.y)[i] : zero;
                 x[j] = in ? reinterpret_cast<const float4*>(g.src.x_in)[i] : zero;
                 before[j] = PRO == PRO_SHIFT && in ? state_at(i) : zero;
             }
             float ss = 0.0f, ir = 1.0f;
-            const bool normed = g.src.y != nullptr && g.src.y_norm != nullptr;
+            const bool normed = PRO != PRO_NORM || (g.src.y != nullptr && g.src.y_norm != nullptr);
             if (normed) {
 #pragma unroll
                 for (int j = 0; j < PER; ++j) ss += ops::sumsq4(y[j]);
@@ -225,7 +231,7 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
                     float4 n = make_float4(1.f, 1.f, 1.f, 1.f);
                     if (normed) n = __ldg(reinterpret_cast<const float4*>(g.src.y_norm) + i);
                     x[j].x += y[j].x * ir * n.x; x[j].y += y[j].y * ir * n.y; x[j].z += y[j].z * ir * n.z; x[j].w += y[j].w * ir * n.w;
-                    if (g.src.step != nullptr) {
+                    if (PRO == PRO_NORM && g.src.step != nullptr) {
                         const float4 t = __ldg(reinterpret_cast<const float4*>(g.src.step) + i);
                         x[j].x += t.x; x[j].y += t.y; x[j].z += t.z; x[j].w += t.w;
                     }
@@ -259,8 +265,8 @@ gemv_kernel(const __grid_constant__ GemvArgs<T> g)
         int piece = 0;
         for (int c = 0; c < chunks; ++c) {
             ok = tc::wait_uniform(&full[slot], phase, abort_flag) && ok;
-            const bool in = piece * GV_PIECE + off < row_bytes;
-            if (++piece == pieces) piece = 0;
+            const bool in = (ROUTE == ROUTE_COLUMNS ? piece : c) * GV_PIECE + off < row_bytes;
+            if (ROUTE == ROUTE_COLUMNS && ++piece == pieces) piece = 0;
             if (ok && in) {
                 float af[V::N];
                 V::unpack(lds128(reinterpret_cast<const uint8_t*>(as) + (size_t)c * GV_PIECE + off), af);

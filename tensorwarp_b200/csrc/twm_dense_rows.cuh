@@ -119,8 +119,8 @@ __device__ __forceinline__ float4 scale4(const float4 x, float s, const float4 g
 // zero on the way (the expert counts of the routing that follows).  A CTA walks `rows_per_cta` consecutive rows and
 // keeps the row before; its first row's predecessor is computed again (or comes from the state).  PER > 0: a
 // thread's share of a row is PER vectors, held in registers, every load issued before the first use; PER = 0: rows
-// of any length, in shared memory.
-template <typename T, int PER>
+// of any length, in shared memory.  FULL = false: without pre_norm, step, routed outputs and clear.
+template <typename T, int PER, bool FULL>
 __global__ void __launch_bounds__(ROW_THREADS)
 residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __restrict__ a, const float* __restrict__ shift,
                      const float* __restrict__ shift_state, const float* __restrict__ pre_norm, const int* __restrict__ meta, int rows,
@@ -133,14 +133,14 @@ residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __rest
     const int wp = src.wp, nvec = wp >> 2;
     const int r0 = blockIdx.x * rows_per_cta, r1 = min(rows, r0 + rows_per_cta);
     const int pos0 = meta[0];
-    if (blockIdx.x == 0)
+    if (FULL && blockIdx.x == 0)
         for (int i = threadIdx.x; i < n_clear; i += ROW_THREADS) clear[i] = 0;
     const float* st = shift != nullptr && r0 == 0 && pos0 > 0
                           ? shift_state + ((size_t)meta[1] * 2 + ((pos0 - 1) & 1)) * wp : nullptr;
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     if constexpr (PER > 0) {
-        __shared__ int slot_row[MAX_TOP];
-        __shared__ float slot_weight[MAX_TOP];
+        __shared__ int slot_row[FULL ? MAX_TOP : 1];
+        __shared__ float slot_weight[FULL ? MAX_TOP : 1];
         float4 before[PER];
 #pragma unroll
         for (int j = 0; j < PER; ++j) {
@@ -149,7 +149,7 @@ residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __rest
         }
         for (int r = (shift != nullptr && r0 > 0) ? r0 - 1 : r0; r < r1; ++r) {
             float4 x[PER], y[PER];
-            if (src.routed.rows != nullptr) {               // the row's slots, known before the first of their loads
+            if (FULL && src.routed.rows != nullptr) {       // the row's slots, known before the first of their loads
                 __syncthreads();
                 if (threadIdx.x < src.routed.top) {
                     slot_row[threadIdx.x] = src.routed.row[(size_t)r * src.routed.top + threadIdx.x];
@@ -161,13 +161,14 @@ residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __rest
             ResidualSource<T> plain = src;                  // the row without what joins it
             plain.y = nullptr;
             plain.routed.rows = nullptr;
+            if (!FULL) plain.step = nullptr;
 #pragma unroll
             for (int j = 0; j < PER; ++j) {
                 const int i = threadIdx.x + j * ROW_THREADS;
                 y[j] = src.y != nullptr && i < nvec ? src.y_at(r, i) : zero;
                 x[j] = i < nvec ? plain.at(r, pos0 + r, tok, i, 1.0f) : zero;
             }
-            if (src.routed.rows != nullptr) {
+            if (FULL && src.routed.rows != nullptr) {
 #pragma unroll 4
                 for (int s = 0; s < src.routed.top; ++s) {
                     const T* row = src.routed.rows + (size_t)slot_row[s] * wp;
@@ -182,7 +183,7 @@ residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __rest
                 }
             }
             float ir = 1.0f;
-            if (src.has_y() && src.y_norm != nullptr) {
+            if ((src.y != nullptr || (FULL && src.routed.rows != nullptr)) && src.y_norm != nullptr) {
                 float ss = 0.0f;
 #pragma unroll
                 for (int j = 0; j < PER; ++j) ss += ops::sumsq4(y[j]);
@@ -196,9 +197,9 @@ residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __rest
                 float4 n = make_float4(1.f, 1.f, 1.f, 1.f);
                 if (src.y_norm != nullptr) n = __ldg(reinterpret_cast<const float4*>(src.y_norm) + i);
                 x[j].x += y[j].x * ir * n.x; x[j].y += y[j].y * ir * n.y; x[j].z += y[j].z * ir * n.z; x[j].w += y[j].w * ir * n.w;
-                xs += ops::sumsq4(x[j]);
+                if (FULL) xs += ops::sumsq4(x[j]);
             }
-            if (pre_norm != nullptr) pr = inv_rms(group_sum(xs, red, ROW_THREADS, 1), src.width, src.eps);
+            if (FULL && pre_norm != nullptr) pr = inv_rms(group_sum(xs, red, ROW_THREADS, 1), src.width, src.eps);
 #pragma unroll
             for (int j = 0; j < PER; ++j) {
                 const int i = threadIdx.x + j * ROW_THREADS;
@@ -207,7 +208,7 @@ residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __rest
                     reinterpret_cast<float4*>(x_out + (size_t)r * wp)[i] = x[j];
                     float4 h = x[j];
                     if (shift != nullptr) h = shift4(x[j], before[j], __ldg(reinterpret_cast<const float4*>(shift) + i));
-                    if (pre_norm != nullptr) h = scale4(x[j], pr, __ldg(reinterpret_cast<const float4*>(pre_norm) + i));
+                    if (FULL && pre_norm != nullptr) h = scale4(x[j], pr, __ldg(reinterpret_cast<const float4*>(pre_norm) + i));
                     if (a != nullptr) store4<T>(a + (size_t)r * wp + i * 4, h);
                 }
                 before[j] = x[j];
@@ -230,7 +231,7 @@ residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __rest
             const int tok = src.tokens != nullptr ? src.tokens[r] : 0;
             const float ir = src.row_inv_rms(r, red, ROW_THREADS, 1);
             float pr = 1.0f;
-            if (pre_norm != nullptr) {
+            if (FULL && pre_norm != nullptr) {
                 float xs = 0.0f;
                 for (int i = threadIdx.x; i < nvec; i += ROW_THREADS) xs += ops::sumsq4(src.at(r, pos0 + r, tok, i, ir));
                 pr = inv_rms(group_sum(xs, red, ROW_THREADS, 1), src.width, src.eps);
@@ -245,7 +246,7 @@ residual_rows_kernel(ResidualSource<T> src, float* __restrict__ x_out, T* __rest
                     h = shift4(x, *before, __ldg(reinterpret_cast<const float4*>(shift) + i));
                     *before = x;
                 }
-                if (pre_norm != nullptr) h = scale4(x, pr, __ldg(reinterpret_cast<const float4*>(pre_norm) + i));
+                if (FULL && pre_norm != nullptr) h = scale4(x, pr, __ldg(reinterpret_cast<const float4*>(pre_norm) + i));
                 if (a != nullptr) store4<T>(a + (size_t)r * wp + i * 4, h);
             }
         }

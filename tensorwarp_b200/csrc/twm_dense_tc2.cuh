@@ -178,7 +178,6 @@ gemm_tc2_kernel(const __grid_constant__ TcArgs g)
         tc::tc_fence_after();
         asm volatile("tcgen05.dealloc.cta_group::2.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(2u * T2_BN) : "memory");
     }
-    cluster_sync_all();                                      // the next kernel's CTA may ask for tensor memory as soon as this one is gone
 }
 
 }  // namespace dense

@@ -44,7 +44,7 @@ def engine(case, dtype, **options):
     return DenseEngine(cases.model(cfg, cases.weights(cfg, 7, rank), rank, dtype), **options)
 
 
-def close(got, want, dtype, case="tiles"):
+def close(got, want, dtype, case="tiles", tol=None):
     """In 16 bits a choice of experts that is nearly a tie may go either way: where the model chooses, most rows are compared.
     Where all experts are used, rounding the norms alone to 16 bits in the oracle moves single rows by 0.06, half of them
     by less than 0.015."""
@@ -54,7 +54,7 @@ def close(got, want, dtype, case="tiles"):
         assert np.quantile(err, q) < TOL[dtype] and np.isfinite(err).all(), float(np.quantile(err, q))
         assert case != "tiles" or err.max() < 0.2, (int(err.argmax()), float(err.max()))
     else:
-        assert err.max() < TOL[dtype], (int(err.argmax()), float(err.max()))
+        assert err.max() < (tol or TOL[dtype]), (int(err.argmax()), float(err.max()))
     assert _dense.device_error() == 0
 
 
@@ -167,6 +167,34 @@ def test_long_decoding_far_from_the_first_tokens(case, dtype):
     eng.step(seq, toks[:100])
     rows = [eng.step(seq, [t], [0]).clone() for t in toks[100:]]
     close(torch.cat(rows), logits[100:], dtype, case)
+
+
+@BOTH
+def test_long_prompt(dtype):
+    """More tokens than the kernels' grids hold at once; every window has passed many times.  Over thousands of tokens the
+    32-bit rounding of slow decays (next to 1) adds up in the state."""
+    n = 2200
+    toks, logits, _ = oracle("tiles", n, 5)
+    eng = engine("tiles", dtype, max_tokens=n, portion=n)
+    want = [0, 1, 63, 64, 65, 1023, 1024, 2047, 2048, 2049] + list(range(2150, n))
+    for _ in range(3):
+        seq = eng.open()
+        close(eng.step(seq, toks, want), logits[want], dtype, tol=1e-4)
+        eng.close(seq)
+
+
+@BOTH
+@pytest.mark.parametrize("width,ff,top", [(80, 1200, 3), (2400, 40, 3), (1300, 1210, 2)])
+def test_experts_larger_than_one_pass_of_the_decode_products(width, ff, top, dtype):
+    cfg = cases.config(width, 61, [cases.layer(cases.linear(2, 16, 16), cases.experts(top, top, ff)),
+                                   cases.layer(cases.latent(2, 16, 8, 16, 16, 5), cases.experts(top, top, ff))])
+    t = cases.weights(cfg, 3, 4)
+    toks = cases.tokens(cfg, 14, 3)
+    want = ref.forward(cfg, cases.as_float64(t), toks)
+    eng = DenseEngine(cases.model(cfg, t, 4, dtype), max_tokens=32)
+    seq = eng.open()
+    close(torch.cat([eng.step(seq, [x], [0]).clone() for x in toks]), want, dtype)
+    close(eng.step(eng.open(), toks, list(range(14))), want, dtype)
 
 
 def test_a_sequence_ends_at_its_slot():
@@ -342,7 +370,7 @@ def test_router(n, top, groups, keep):
 
 
 @pytest.mark.parametrize("counts,n,k", [((3, 0, 130, 1), 64, 48), ((0, 0, 5), 200, 80), ((128, 128), 130, 256), ((1,) * 40, 48, 16),
-                                        ((257, 0, 300, 64, 2, 500), 320, 192), ((7, 900, 0), 1030, 64)])
+                                        ((257, 0, 300, 64, 2, 500), 320, 192), ((7, 900, 0), 1030, 64), ((1500, 0, 900, 3), 2048, 96)])
 @pytest.mark.parametrize("dtype,kernel", [(torch.float32, 1), (torch.bfloat16, 1), (torch.bfloat16, 64), (torch.bfloat16, 128), (torch.bfloat16, 256),
                                           (torch.bfloat16, 0)])
 @pytest.mark.parametrize("epi", [_dense.EPI_STORE, _dense.EPI_STORE_F32, _dense.EPI_RELU2])
