@@ -75,7 +75,7 @@ twm_status launch(const char* what, void (*kernel)(KArgs...), dim3 grid, int thr
                   int cluster, Args&&... args)
 {
     if (smem > kSmemLimit) return invalid("a row does not fit shared memory");
-    if (smem > 48 * 1024) {
+    if (smem > 32 * 1024) {                              // 48 KB without asking, static shared memory included
         const cudaError_t r = cudaFuncSetAttribute((const void*)kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (r != cudaSuccess) return fail(what, r);
     }

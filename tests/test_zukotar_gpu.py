@@ -184,7 +184,7 @@ def test_long_prompt(dtype):
 
 
 @BOTH
-@pytest.mark.parametrize("width,ff,top", [(80, 1200, 3), (2400, 40, 3), (1300, 1210, 2)])
+@pytest.mark.parametrize("width,ff,top", [(80, 1200, 3), (2400, 40, 3), (1300, 1210, 2), (5000, 16, 2)])
 def test_experts_larger_than_one_pass_of_the_decode_products(width, ff, top, dtype):
     cfg = cases.config(width, 61, [cases.layer(cases.linear(2, 16, 16), cases.experts(top, top, ff)),
                                    cases.layer(cases.latent(2, 16, 8, 16, 16, 5), cases.experts(top, top, ff))])
